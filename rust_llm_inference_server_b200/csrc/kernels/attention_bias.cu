@@ -17,6 +17,9 @@
 // keys and values as they are read.  `gate_cols` > 1: the gate has one logit a channel of every head (gate[t, h *
 // dv + c]) instead of one a head.
 //
+// row_norm_store: queries and keys RMS-normed over their whole projections (all heads together, one weight an entry), before
+// they are split into heads.
+//
 // `bias` is a float32 table [n_dist, n_heads] by distance (the host turns bucket rules into it; all
 // distances from n_dist - 1 on share the last row).  Norms, scores, softmax, value sums, the mixing and
 // the gate are float32 whatever the element type.
@@ -252,6 +255,74 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_vec_kernel(
     }
 }
 
+// Queries and keys normed over all their heads together: q = q / sqrt(mean over the nh d entries of q^2 + eps) * q_w, k the
+// same over its nkv d entries (q_w, k_w one number an entry; null: no norm), values as projected.  One CTA a token; VN
+// elements a load (d and dv are multiples of VN).
+template <typename T, int VN>
+__global__ __launch_bounds__(256) void qk_row_norm_store_kernel(
+    const T* __restrict__ proj, long long stride, int q_off, int k_off, int v_off, const float* __restrict__ q_w,
+    const float* __restrict__ k_w, float eps, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+    const int* __restrict__ slots, int nh, int nkv, int d, int dv, int page_size) {
+    pdl_wait_and_trigger();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    const T* row = proj + (size_t)t * stride;
+    auto load = [](const T* p, float* v) {
+        if constexpr (VN == 1) v[0] = to_f<T>(*p);
+        else load16<T>(p, v);
+    };
+    auto store = [](T* p, const float* v) {
+        if constexpr (VN == 1) *p = from_f<T>(v[0]);
+        else {
+            alignas(16) T o[VN];
+#pragma unroll
+            for (int i = 0; i < VN; ++i) o[i] = from_f<T>(v[i]);
+            *reinterpret_cast<uint4*>(p) = *reinterpret_cast<const uint4*>(o);
+        }
+    };
+    float v[VN], sq = 0.f, sk = 0.f;
+    if (q_w != nullptr)
+        for (int c = threadIdx.x * VN; c < nh * d; c += blockDim.x * VN) {
+            load(row + q_off + c, v);
+#pragma unroll
+            for (int i = 0; i < VN; ++i) sq = fmaf(v[i], v[i], sq);
+        }
+    if (k_w != nullptr)
+        for (int c = threadIdx.x * VN; c < nkv * d; c += blockDim.x * VN) {
+            load(row + k_off + c, v);
+#pragma unroll
+            for (int i = 0; i < VN; ++i) sk = fmaf(v[i], v[i], sk);
+        }
+    sq = block_sum(sq, scratch);
+    sk = block_sum(sk, scratch);
+    const float rq = 1.0f / sqrtf(sq / (float)(nh * d) + eps), rk = 1.0f / sqrtf(sk / (float)(nkv * d) + eps);
+    for (int c = threadIdx.x * VN; c < nh * d; c += blockDim.x * VN) {
+        load(row + q_off + c, v);
+        if (q_w != nullptr) {
+#pragma unroll
+            for (int i = 0; i < VN; ++i) v[i] = v[i] * rq * q_w[c + i];
+        }
+        store(q_out + (size_t)t * nh * d + c, v);
+    }
+    const int slot = slots != nullptr ? slots[t] : -1;
+    if (slot < 0) return;
+    const long long r0 = (long long)(slot / page_size) * nkv * page_size + slot % page_size;
+    for (int c = threadIdx.x * VN; c < nkv * d; c += blockDim.x * VN) {
+        load(row + k_off + c, v);
+        if (k_w != nullptr) {
+#pragma unroll
+            for (int i = 0; i < VN; ++i) v[i] = v[i] * rk * k_w[c + i];
+        }
+        const int g = c / d;
+        store(k_cache + (r0 + (long long)g * page_size) * d + (c - g * d), v);
+    }
+    for (int c = threadIdx.x * VN; c < nkv * dv; c += blockDim.x * VN) {
+        load(row + v_off + c, v);
+        const int g = c / dv;
+        store(v_cache + (r0 + (long long)g * page_size) * dv + (c - g * dv), v);
+    }
+}
+
 template <typename T>
 __global__ __launch_bounds__(WARPS * 32) void attn_bias_kernel(
     const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ out,
@@ -409,6 +480,25 @@ extern "C" int rlis_qk_norm_store(const void* proj, long long stride, int q_off,
                     q_temp_coef, q_temp_every, rot_half, proj_bias);
     else
         return RLIS_ERR_UNSUPPORTED;
+    return RLIS_LAUNCH_CHECK();
+}
+
+// q_w float32 [nh d], k_w float32 [nkv d] (null: no norm); the rest as rlis_qk_norm_store.
+extern "C" int rlis_qk_row_norm_store(const void* proj, long long stride, int q_off, int k_off, int v_off, const float* q_w,
+                                      const float* k_w, float eps, void* q_out, void* k_cache, void* v_cache, const int* slots,
+                                      int n_tokens, int nh, int nkv, int d, int dv, int page_size, int dtype, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (d <= 0 || dv <= 0 || nh <= 0 || nkv <= 0) return RLIS_ERR_UNSUPPORTED;
+    const int vn = dtype == RLIS_F32 ? 4 : 8;
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_out) |
+                           reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache);
+    const bool vec = d % vn == 0 && dv % vn == 0 && (ptrs & 15) == 0 && stride % vn == 0 && q_off % vn == 0 &&
+                     k_off % vn == 0 && v_off % vn == 0;
+#define RLIS_RNS(T, VN) rlis_launch(qk_row_norm_store_kernel<T, VN>, n_tokens, 256, 0, stream, (const T*)proj, stride, q_off, k_off,                                     v_off, q_w, k_w, eps, (T*)q_out, (T*)k_cache, (T*)v_cache, slots, nh, nkv, d, dv, page_size)
+    if (dtype == RLIS_F32) { if (vec) RLIS_RNS(float, 4); else RLIS_RNS(float, 1); }
+    else if (dtype == RLIS_BF16) { if (vec) RLIS_RNS(bf16, 8); else RLIS_RNS(bf16, 1); }
+    else return RLIS_ERR_UNSUPPORTED;
+#undef RLIS_RNS
     return RLIS_LAUNCH_CHECK();
 }
 

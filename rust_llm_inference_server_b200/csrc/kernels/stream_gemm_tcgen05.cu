@@ -64,6 +64,12 @@
 //     its sums by 1 / sqrt(sum of the token's partials in the order of the tiles / dim + eps).
 // Both are deterministic and depend on the token's own values only.
 //
+// A bias (float32, one a feature) may be added to the sums of every epilogue.  And a third way on to the next sublayer, for
+// residual streams side by side whose norm needs no statistics (see stream_mix.cu):
+//   * "streams" (the last product of a mixer or feed-forward): the finisher takes y = bf16(sum) + bias, updates the token's
+//     streams in place, x_t <- sum_s mix[s, t] x_s + out[t] y, weighs them, u = sum_t in[t] x_t, and writes h = bf16(tanh(
+//     alpha u) w + b), the rows of the product that follows: no partial sums, no scale left to apply, no norm kernel.
+//
 // Every mbarrier wait is bounded (a fifth of a second); a wait that runs out sets an error word
 // (rlis_stream_gemm_error), every role runs to its end without further waits, and the CTA frees
 // its tensor memory before it returns.
@@ -85,9 +91,10 @@ template <int NT> __host__ __device__ constexpr int stages_of() { return NT <= 1
 constexpr int W_STAGE_BYTES = SF * SK * 2;
 constexpr int S_THREADS = 128;
 constexpr int MAX_SPLITS = 16;          // the largest cluster (above 8 is opt-in)
+constexpr int MAX_STREAMS = 8;          // streams epilogue
 
 template <int NT> constexpr size_t stream_smem_bytes(int n_stages = stages_of<NT>()) {
-    return (size_t)n_stages * (W_STAGE_BYTES + NT * SK * 2) + 1024 /* alignment */ + 768 /* SCtrl */;
+    return (size_t)n_stages * (W_STAGE_BYTES + NT * SK * 2) + 1024 /* alignment */ + 1152 /* SCtrl */;
 }
 
 // A timeline for measurements, compiled in only with -DRLIS_TIMELINE (the build adds it when the
@@ -118,6 +125,7 @@ struct SCtrl {
     uint32_t tmem_base;
     int abort;
     float red[4];           // sink epilogue: the warps' sums of squares
+    float coef[MAX_STREAMS * MAX_STREAMS + 2 * MAX_STREAMS];   // streams epilogue: mix, out, in
     float rstd[128];        // scaled rows: the norm's scale of every token
 };
 
@@ -132,6 +140,16 @@ struct NormFuse {
     bf16* xn;                   // sink: [M, N] = bf16(resid * norm_w)
     float* out_partials;        // sink: [tiles, M]
     float gate_slope;           // gated epilogue: g sigmoid(slope g) * u (1: silu; +inf: max(g, 0))
+    const float* bias;          // [N] added to the sums, or null
+    // streams (epilogue 3): what x_s are read from (row stride, stream stride; 0: one row is every stream) and written to
+    // ([M, S, N]), their coefficients, and the dynamic tanh that follows (norm_w its weight, xn its result)
+    const float* s_in;
+    long long s_row, s_stream;
+    int n_streams;
+    const float *mix, *out_c, *in_c;
+    float* s_out;
+    float alpha;
+    const float* norm_b;
 };
 
 // A float into the shared memory of the cluster's CTA `rank` (at the offset of `local`), counted
@@ -173,10 +191,10 @@ __device__ __forceinline__ void store_token(OutT* __restrict__ y, float v, int t
 // the thread's feature f of resid += bf16(v); xn = bf16(resid * w); the CTA's sum of resid^2 to
 // partials[tile][t].  `live` false: the barriers only.
 __device__ __forceinline__ void sink_token(const NormFuse& nf, float* red, float v, int t, int f, int tile, int M,
-                                           int N, bool live, float r_old, float w) {
+                                           int N, bool live, float r_old, float w, float bias) {
     float r = 0.f;
     if (live && f < N) {
-        r = r_old + __bfloat162float(__float2bfloat16_rn(v));
+        r = r_old + (__bfloat162float(__float2bfloat16_rn(v)) + bias);
         nf.resid[(size_t)t * N + f] = r;
         nf.xn[(size_t)t * N + f] = __float2bfloat16_rn(r * w);
     }
@@ -185,6 +203,30 @@ __device__ __forceinline__ void sink_token(const NormFuse& nf, float* red, float
     __syncthreads();
     if (threadIdx.x == 0 && live) nf.out_partials[(size_t)tile * M + t] = (red[0] + red[1]) + (red[2] + red[3]);
     __syncthreads();
+}
+
+// Streams epilogue for token t and the thread's feature f (see the head of the file); x: the old streams.
+__device__ __forceinline__ void load_streams(const NormFuse& nf, float (&x)[MAX_STREAMS], int t, int f) {
+#pragma unroll
+    for (int s = 0; s < MAX_STREAMS; ++s) x[s] = s < nf.n_streams ? nf.s_in[t * nf.s_row + s * nf.s_stream + f] : 0.f;
+}
+__device__ __forceinline__ void streams_token(const NormFuse& nf, const float* coef, const float (&x)[MAX_STREAMS], float v,
+                                              float bias, float w, float b, int t, int f, int N) {
+    const float y = __bfloat162float(__float2bfloat16_rn(v)) + bias;
+    const float *mix = coef, *out_c = coef + MAX_STREAMS * MAX_STREAMS, *in_c = out_c + MAX_STREAMS;
+    float u = 0.f;
+#pragma unroll
+    for (int to = 0; to < MAX_STREAMS; ++to) {
+        if (to >= nf.n_streams) break;
+        float a = 0.f;
+#pragma unroll
+        for (int s = 0; s < MAX_STREAMS; ++s)
+            if (s < nf.n_streams) a = fmaf(mix[s * MAX_STREAMS + to], x[s], a);
+        a = fmaf(out_c[to], y, a);
+        u = fmaf(in_c[to], a, u);
+        nf.s_out[((size_t)t * nf.n_streams + to) * N + f] = a;
+    }
+    nf.xn[(size_t)t * N + f] = __float2bfloat16_rn(fmaf(tanhf(nf.alpha * u), w, b));
 }
 
 template <int NT, int EPI, typename OutT>
@@ -295,7 +337,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
 #ifdef RLIS_TIMELINE
     if (tl_on) g_timeline[tl_slot][8] = *reinterpret_cast<volatile unsigned long long*>(&g_timeline_last_end);
 #endif
-    const bool scaled = EPI != 2 && nf.in_partials != nullptr;
+    const bool scaled = EPI < 2 && nf.in_partials != nullptr;
     if (scaled && (int)threadIdx.x < M) {
         // this token's scale: the partial sums in the order of the tiles (RMSNorm: 1 / sqrt(mean + eps))
         float ss = 0.f;
@@ -304,7 +346,25 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
     }
     // sink: what the first token this thread finishes needs from memory, requested before the sums arrive
     const int f = n0 + warp * 32 + lane;
-    float sink_w = 0.f, sink_r0 = 0.f;
+    float sink_w = 0.f, sink_r0 = 0.f, st_b = 0.f;
+    float st_x[EPI == 3 ? MAX_STREAMS : 1];
+    const float bias = nf.bias != nullptr && f < N ? nf.bias[f] : 0.f;
+    if constexpr (EPI == 3) {
+        if (threadIdx.x < MAX_STREAMS * MAX_STREAMS) {
+            const int s = threadIdx.x / MAX_STREAMS, to = threadIdx.x % MAX_STREAMS, S = nf.n_streams;
+            ctrl->coef[threadIdx.x] = s < S && to < S ? nf.mix[s * S + to] : 0.f;
+            if (threadIdx.x < S) {
+                ctrl->coef[MAX_STREAMS * MAX_STREAMS + threadIdx.x] = nf.out_c[threadIdx.x];
+                ctrl->coef[MAX_STREAMS * MAX_STREAMS + MAX_STREAMS + threadIdx.x] = nf.in_c != nullptr ? nf.in_c[threadIdx.x] : 1.f;
+            }
+        }
+        const int t0 = splits == 1 ? 0 : split;
+        if (f < N) {
+            sink_w = nf.norm_w[f];
+            st_b = nf.norm_b[f];
+            if (t0 < M) load_streams(nf, st_x, t0, f);
+        }
+    }
     if (EPI == 2 && f < N) {
         sink_w = nf.norm_w[f];
         const int t0 = splits == 1 ? 0 : split;
@@ -329,16 +389,26 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                     const int t = c * 16 + j;
                     if (t >= M) continue;           // the same for all threads
                     const float r_old = t == 0 ? sink_r0 : (ok && f < N ? nf.resid[(size_t)t * N + f] : 0.f);
-                    sink_token(nf, ctrl->red, __uint_as_float(r[j]), t, f, tile, M, N, ok, r_old, sink_w);
+                    sink_token(nf, ctrl->red, __uint_as_float(r[j]), t, f, tile, M, N, ok, r_old, sink_w, bias);
                 }
                 continue;
             }
             if (!ok) continue;
+            if constexpr (EPI == 3) {
 #pragma unroll
-            for (int j = 0; j < 16; ++j)
-                if (c * 16 + j < M)
-                    store_token<EPI, OutT>(y, __uint_as_float(r[j]) * (scaled ? ctrl->rstd[c * 16 + j] : 1.0f),
-                                           c * 16 + j, f, lane, N, nf.gate_slope);
+                for (int j = 0; j < 16; ++j) {
+                    const int t = c * 16 + j;
+                    if (t >= M || f >= N) continue;
+                    if (t > 0) load_streams(nf, st_x, t, f);
+                    streams_token(nf, ctrl->coef, st_x, __uint_as_float(r[j]), bias, sink_w, st_b, t, f, N);
+                }
+            } else {
+#pragma unroll
+                for (int j = 0; j < 16; ++j)
+                    if (c * 16 + j < M)
+                        store_token<EPI, OutT>(y, __uint_as_float(r[j]) * (scaled ? ctrl->rstd[c * 16 + j] : 1.0f) + bias,
+                                               c * 16 + j, f, lane, N, nf.gate_slope);
+            }
         }
     } else {
         // Once every CTA of the cluster is done with its products, the stages are free everywhere:
@@ -378,6 +448,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
 #pragma unroll 1
             for (int c2 = split, slot = 0; c2 < N_CHUNKS; c2 += splits, ++slot) {
                 const int fo = n0 + c2 * CHUNK_F + fi;
+                const float fbias = nf.bias != nullptr && fo < N ? nf.bias[fo] : 0.f;
 #pragma unroll 1
                 for (int t = tg; t < ((M + 15) & ~15); t += S_THREADS / CHUNK_F) {
                     const float* src = part + (slot * splits) * (CHUNK_F * NT) + (t / 4) * (CHUNK_F * 4) + fi * 4 + (t & 3);
@@ -386,12 +457,12 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                     const float sc = scaled && t < M ? ctrl->rstd[t] : 1.0f;
                     if (EPI == 1) {
                         // (every lane takes part in the exchange of the gated epilogue; rows past M are not stored)
-                        const float g = v * sc;
+                        const float g = v * sc + fbias;
                         const float other = __shfl_xor_sync(0xffffffffu, g, 4);
                         if (ok && t < M && (fi & 4) == 0 && fo + 4 < N)
                             y[(size_t)t * (N >> 1) + ((fo >> 3) << 2) + (fo & 3)] = from_f<OutT>(glu_gate(g, nf.gate_slope) * other);
                     } else if (ok && t < M && fo < N) {
-                        y[(size_t)t * N + fo] = from_f<OutT>(v * sc);
+                        y[(size_t)t * N + fo] = from_f<OutT>(v * sc + fbias);
                     }
                 }
             }
@@ -425,9 +496,14 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                 for (int s = 0; s < splits; ++s) v += part[(slot * splits + s) * SF + (int)threadIdx.x];
                 if (EPI == 2) {
                     const float r_old = slot == 0 ? sink_r0 : (good && f < N ? nf.resid[(size_t)t * N + f] : 0.f);
-                    sink_token(nf, ctrl->red, v, t, f, tile, M, N, good, r_old, sink_w);
+                    sink_token(nf, ctrl->red, v, t, f, tile, M, N, good, r_old, sink_w, bias);
+                } else if constexpr (EPI == 3) {
+                    if (good && f < N) {
+                        if (slot > 0) load_streams(nf, st_x, t, f);
+                        streams_token(nf, ctrl->coef, st_x, v, bias, sink_w, st_b, t, f, N);
+                    }
                 } else if (good) {
-                    store_token<EPI, OutT>(y, v * (scaled ? ctrl->rstd[t] : 1.0f), t, f, lane, N, nf.gate_slope);
+                    store_token<EPI, OutT>(y, v * (scaled ? ctrl->rstd[t] : 1.0f) + bias, t, f, lane, N, nf.gate_slope);
                 }
             }
         }
@@ -449,9 +525,10 @@ int g_target_ctas = 0;      // 0: twice the number of SMs
 int g_min_stages = -1;      // stages a CTA is given at least (measurements; -1: by the rows, see launch_stream)
 
 template <int NT, int EPI, typename OutT>
-int launch_stream(const void* x, const void* W, void* y, int M, int N, int K, const NormFuse& nf, cudaStream_t stream) {
+int launch_stream(const void* x, long long ldx, const void* W, void* y, int M, int N, int K, const NormFuse& nf,
+                  cudaStream_t stream) {
     CUtensorMap map_w, map_x;
-    if (!make_map(&map_w, W, N, K, SF) || !make_map(&map_x, x, M, K, NT)) return RLIS_ERR_UNSUPPORTED;
+    if (!make_map(&map_w, W, N, K, SF) || !make_map(&map_x, x, M, K, NT, ldx)) return RLIS_ERR_UNSUPPORTED;
     static bool attr_done = false;
     if (!attr_done) {
         cudaFuncSetAttribute(stream_gemm_kernel<NT, EPI, OutT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -499,11 +576,11 @@ int launch_stream(const void* x, const void* W, void* y, int M, int N, int K, co
 }
 
 template <int NT>
-int dispatch_stream(const void* x, const void* W, void* y, int M, int N, int K, int out_dtype, int epilogue,
+int dispatch_stream(const void* x, long long ldx, const void* W, void* y, int M, int N, int K, int out_dtype, int epilogue,
                     const NormFuse& nf, cudaStream_t stream) {
-    if (epilogue == 0 && out_dtype == RLIS_BF16) return launch_stream<NT, 0, bf16>(x, W, y, M, N, K, nf, stream);
-    if (epilogue == 0 && out_dtype == RLIS_F32) return launch_stream<NT, 0, float>(x, W, y, M, N, K, nf, stream);
-    if (epilogue == 1 && out_dtype == RLIS_BF16) return launch_stream<NT, 1, bf16>(x, W, y, M, N, K, nf, stream);
+    if (epilogue == 0 && out_dtype == RLIS_BF16) return launch_stream<NT, 0, bf16>(x, ldx, W, y, M, N, K, nf, stream);
+    if (epilogue == 0 && out_dtype == RLIS_F32) return launch_stream<NT, 0, float>(x, ldx, W, y, M, N, K, nf, stream);
+    if (epilogue == 1 && out_dtype == RLIS_BF16) return launch_stream<NT, 1, bf16>(x, ldx, W, y, M, N, K, nf, stream);
     return RLIS_ERR_UNSUPPORTED;
 }
 }  // namespace
@@ -542,24 +619,27 @@ extern "C" void rlis_stream_gemm_set_min_stages(int n) { g_min_stages = n; }
 
 // out_dtype: RLIS_BF16 or RLIS_F32.  epilogue 0: y [M, N]; 1 (gated unit, rows of W interleaved
 // gate/up in blocks of 4, N a multiple of 8): y [M, N / 2] = g sigmoid(gate_slope g) u (slope 1: SwiGLU; +inf: relu).  M up to 128; K a multiple of 8;
-// x and W 16-byte aligned.
+// x and W 16-byte aligned; x's rows lie ldx elements apart (a multiple of 8).  bias float32 [N] in the order of W's rows
+// (null: none) is added to the (scaled) sums.
 //
 // Scaled rows (epilogues 0 and 1; in_partials not null): x is bf16(resid * norm weight) and
 // in_partials [n_partials, M] the sums of squares that a sink product left; y is multiplied by
 // 1 / sqrt(sum / norm_dim + eps) of its row.
-// Sink (epilogue 2, M up to 16; y unused): resid [M, N] float32 += bf16(x W^T) in place,
+// Sink (epilogue 2, M up to 16; y unused): resid [M, N] float32 += bf16(x W^T) + bias in place,
 // xn [M, N] bf16 = resid * norm_w, out_partials [ceil(N / 128), M] = sums of resid^2 by 128 features.
-extern "C" int rlis_stream_gemm_fused(const void* x, const void* W, void* y, int M, int N, int K, int out_dtype,
-                                      int epilogue, const float* in_partials, int n_partials, int norm_dim, float eps,
-                                      float* resid, const float* norm_w, void* xn, float* out_partials,
+static bool stream_takes(const void* x, long long ldx, const void* W, int M, int K) {
+    return M <= 128 && K > 0 && (K & 7) == 0 && ldx >= K && (ldx & 7) == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 &&
+           (reinterpret_cast<uintptr_t>(x) & 15) == 0;
+}
+extern "C" int rlis_stream_gemm_fused(const void* x, long long ldx, const void* W, void* y, int M, int N, int K, int out_dtype,
+                                      int epilogue, const float* bias, const float* in_partials, int n_partials, int norm_dim,
+                                      float eps, float* resid, const float* norm_w, void* xn, float* out_partials,
                                       float gate_slope, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (M > 128 || K <= 0 || (K & 7) != 0) return RLIS_ERR_UNSUPPORTED;
-    if (epilogue == 1 && (N & 7) != 0) return RLIS_ERR_UNSUPPORTED;
-    if ((reinterpret_cast<uintptr_t>(W) & 15) != 0 || (reinterpret_cast<uintptr_t>(x) & 15) != 0)
-        return RLIS_ERR_UNSUPPORTED;
+    if (!stream_takes(x, ldx, W, M, K) || (epilogue == 1 && (N & 7) != 0)) return RLIS_ERR_UNSUPPORTED;
     NormFuse nf{};
     nf.gate_slope = gate_slope;
+    nf.bias = bias;
     if (in_partials != nullptr) {
         if (epilogue == 2 || n_partials <= 0 || norm_dim <= 0) return RLIS_ERR_UNSUPPORTED;
         nf.in_partials = in_partials;
@@ -574,17 +654,38 @@ extern "C" int rlis_stream_gemm_fused(const void* x, const void* W, void* y, int
         nf.norm_w = norm_w;
         nf.xn = reinterpret_cast<bf16*>(xn);
         nf.out_partials = out_partials;
-        return launch_stream<16, 2, bf16>(x, W, nullptr, M, N, K, nf, stream);
+        return launch_stream<16, 2, bf16>(x, ldx, W, nullptr, M, N, K, nf, stream);
     }
-    if (M <= 16) return dispatch_stream<16>(x, W, y, M, N, K, out_dtype, epilogue, nf, stream);
-    if (M <= 32) return dispatch_stream<32>(x, W, y, M, N, K, out_dtype, epilogue, nf, stream);
-    if (M <= 64) return dispatch_stream<64>(x, W, y, M, N, K, out_dtype, epilogue, nf, stream);
-    return dispatch_stream<128>(x, W, y, M, N, K, out_dtype, epilogue, nf, stream);
+    if (M <= 16) return dispatch_stream<16>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
+    if (M <= 32) return dispatch_stream<32>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
+    if (M <= 64) return dispatch_stream<64>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
+    return dispatch_stream<128>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
 }
 
-extern "C" int rlis_stream_gemm_bf16(const void* x, const void* W, void* y, int M, int N, int K,
-                                     int out_dtype, int epilogue, float gate_slope, cudaStream_t stream) {
-    if (epilogue == 2) return RLIS_ERR_UNSUPPORTED;
-    return rlis_stream_gemm_fused(x, W, y, M, N, K, out_dtype, epilogue, nullptr, 0, 0, 0.f, nullptr, nullptr, nullptr,
-                                  nullptr, gate_slope, stream);
+// Streams (M up to 16): y = bf16(x W^T) + bias joins the residual streams, and h = bf16(tanh(alpha u) w + b) of their
+// weighed sum is the input of the product that follows.  s_in float32, token rows s_row and streams s_stream floats apart
+// (0: one row is every stream); mix [S, S] (from, to), out_c [S], in_c [S] (null: ones); s_out [M, S, N] (may be s_in).
+extern "C" int rlis_stream_gemm_streams(const void* x, long long ldx, const void* W, int M, int N, int K, const float* bias,
+                                        const float* s_in, long long s_row, long long s_stream, int n_streams, const float* mix,
+                                        const float* out_c, const float* in_c, float* s_out, float alpha, const float* w,
+                                        const float* b, void* h, cudaStream_t stream) {
+    if (M <= 0 || N <= 0) return 0;
+    if (!stream_takes(x, ldx, W, M, K) || M > 16 || n_streams < 1 || n_streams > MAX_STREAMS || s_in == nullptr ||
+        mix == nullptr || out_c == nullptr || s_out == nullptr || w == nullptr || b == nullptr || h == nullptr)
+        return RLIS_ERR_UNSUPPORTED;
+    NormFuse nf{};
+    nf.bias = bias;
+    nf.s_in = s_in;
+    nf.s_row = s_row;
+    nf.s_stream = s_stream;
+    nf.n_streams = n_streams;
+    nf.mix = mix;
+    nf.out_c = out_c;
+    nf.in_c = in_c;
+    nf.s_out = s_out;
+    nf.alpha = alpha;
+    nf.norm_w = w;
+    nf.norm_b = b;
+    nf.xn = reinterpret_cast<bf16*>(h);
+    return launch_stream<16, 3, bf16>(x, ldx, W, nullptr, M, N, K, nf, stream);
 }

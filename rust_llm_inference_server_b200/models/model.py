@@ -152,6 +152,8 @@ class Model:
         float32 logits [len(rows), vocab] (crates/model/src/llama.rs:272-285)."""
         if isinstance(delta, ScaledRows):       # the last block left the final norm to the head's product
             return self.lm_head.forward(delta, step)
+        if hasattr(delta, "normed_rows"):       # residual streams side by side: the final norm reads their sum
+            return self.lm_head.forward(delta.normed_rows(self.final_norm, step, rows, self.dtype), step)
         h = self.final_norm.forward_rows(resid, delta, step, rows)
         return self.lm_head.forward(h, step)
 
@@ -171,6 +173,11 @@ class _Tail:
             return None
         sink = getattr(self.final_norm, "sink", None)
         return sink(resid, step) if sink is not None else None
+
+    def entry_streams(self, step, n_streams: int):
+        """The same for residual streams side by side (`parts.block.HyperBlock`): their plain sum under the final norm, when
+        the step wants the logits of all its rows in order."""
+        return (None, self.final_norm) if getattr(step, "wants_every_row", False) else None
 
 
 def build_model(config_json: dict, dtype, device="cuda") -> Model:

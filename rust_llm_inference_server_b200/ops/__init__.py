@@ -335,9 +335,32 @@ def head_norm_gate(x: torch.Tensor, weight: torch.Tensor | None, eps: float, out
     return out
 
 
-def gated_delta_state_floats(n_heads: int, n_qk_heads: int, d: int, dv: int, taps: int) -> int:
-    """float32 entries of a request's state for `gated_delta`: S of every head, then the convolution's tail."""
-    return n_heads * dv * d + (taps - 1) * (2 * n_qk_heads * d + n_heads * dv)
+def gate_group_norm(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                    groups: int) -> torch.Tensor:
+    """g = x silu(gate), then each of `groups` equal parts of a row divided by its own root mean square (eps under the
+    root), times `weight` (float32 [W]).  x float32 [T, W]; gate [T, W] in out's type (may be a column slice of wider rows)."""
+    T, W = x.shape
+    _req(x, "x", torch.float32)
+    _req(weight, "weight", torch.float32, (W,))
+    _req(out, "out", None, (T, W))
+    if gate.dtype != out.dtype or tuple(gate.shape) != (T, W) or gate.stride(1) != 1 or not gate.is_cuda:
+        raise KernelError("gate_group_norm: the gate must be [T, W] rows with unit stride in out's type")
+    if groups < 1 or W % groups:
+        raise KernelError(f"gate_group_norm: {groups} parts do not divide rows of {W}")
+    check(lib().rlis_gate_group_norm(x.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(), out.data_ptr(), T, W,
+                                     int(groups), float(eps), _code(out.dtype), _stream()), "gate_group_norm")
+    _count("gate_group_norm")
+    return out
+
+
+def conv_recurrence_state_floats(n_heads: int, n_qk_heads: int, d: int, dv: int, taps: int) -> int:
+    """float32 entries of a request's state for the recurrences behind short convolutions (`gated_delta`, `channel_delta`,
+    `state_space`): S of every head, then the convolution's tail, rounded up to whole 16-byte vectors."""
+    n = n_heads * dv * d + (taps - 1) * (2 * n_qk_heads * d + n_heads * dv)
+    return -(-n // 4) * 4
+
+
+gated_delta_state_floats = conv_recurrence_state_floats
 
 
 # Portions of this many tokens a request (on average over the step) go through the recurrence 16 tokens at a time,
@@ -352,45 +375,180 @@ def _sm_count(device) -> int:
     return torch.cuda.get_device_properties(device).multi_processor_count
 
 
-def gated_delta(proj: torch.Tensor, qkv_off: int, b_off: int, a_off: int, conv_w: torch.Tensor, a_log: torch.Tensor,
-                dt_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step, n_heads: int, n_qk_heads: int,
-                d: int, dv: int, taps: int, unit_eps: float, q_scale: float, chunks: bool | None = None) -> torch.Tensor:
-    """The gated delta rule over the step's tokens (csrc/kernels/gated_delta.cu): from the rows of a stacked
-    projection `proj` [T, N] (q | k | v from column qkv_off: n_qk_heads heads of d twice, then n_heads of dv; one
-    logit a head of beta from b_off and of the decay from a_off), a causal convolution of `taps` taps per channel
-    (conv_w float32 [C, taps]) and silu, unit vectors q (times q_scale) and k, then per head S <- g S, u = beta
-    (v - S^T k), S <- S + k u^T, o = S^T q.  `state` float32 [slots, gated_delta_state_floats(...)] holds S and
-    the convolution's tail between steps; out float32 [T, nh dv].
+def _recurrence_in_chunks(step, n_tokens: int, n_heads: int, dv: int, device) -> bool:
+    return n_tokens >= GATED_DELTA_CHUNKS_FROM * step.n_seqs and \
+        step.n_seqs * n_heads * -(-dv // 16) <= 3 * _sm_count(device)
 
-    A step of long portions of few requests (GATED_DELTA_CHUNKS_FROM) goes through the kernels that take 16 tokens
-    of a request at a time; other steps walk token by token (`chunks` says which, for any step)."""
+
+def _recurrence_operands(name: str, proj, off: int, logits_off: int, conv_w, a_log, dt_bias, state, out, n_heads: int,
+                         n_qk_heads: int, d: int, dv: int, taps: int, n_dt: int) -> int:
+    """Checks what the three recurrences share; returns the number of convolved channels."""
     T, N = proj.shape
     C = 2 * n_qk_heads * d + n_heads * dv
     _req(proj, "proj")
     _req(conv_w, "conv_w", torch.float32, (C, taps))
     _req(a_log, "a_log", torch.float32, (n_heads,))
-    _req(dt_bias, "dt_bias", torch.float32, (n_heads,))
+    _req(dt_bias, "dt_bias", torch.float32, (n_dt,))
     _req(out, "out", torch.float32, (T, n_heads * dv))
-    _req(state, "state", torch.float32, (None, gated_delta_state_floats(n_heads, n_qk_heads, d, dv, taps)))
-    if qkv_off + C > N or b_off + n_heads > N or a_off + n_heads > N:
+    _req(state, "state", torch.float32, (None, conv_recurrence_state_floats(n_heads, n_qk_heads, d, dv, taps)))
+    if off + C > N or logits_off + n_heads > N:
+        raise KernelError(f"{name}: the column offsets reach beyond the projection's rows")
+    return C
+
+
+def _step_pointers(step) -> tuple:
+    return (step.cu_seqlens.data_ptr(), step.ctx_lens.data_ptr(), step.state_slots.data_ptr(), step.seq_of_token.data_ptr())
+
+
+def _count_recurrence(name: str, chunks: bool, solves: bool) -> None:
+    _count(name + ".prepare")
+    if chunks:
+        _count(name + ".gram")
+        if solves:
+            _count(name + ".solve")
+    _count(name + (".chunks" if chunks else ".scan"))
+
+
+def gated_delta(proj: torch.Tensor, qkv_off: int, b_off: int, a_off: int, conv_w: torch.Tensor, a_log: torch.Tensor,
+                dt_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step, n_heads: int, n_qk_heads: int,
+                d: int, dv: int, taps: int, unit_eps: float, q_scale: float, chunks: bool | None = None) -> torch.Tensor:
+    """The gated delta rule over the step's tokens (csrc/kernels/conv_recurrence.cuh): from the rows of a stacked
+    projection `proj` [T, N] (q | k | v from column qkv_off: n_qk_heads heads of d twice, then n_heads of dv; one
+    logit a head of beta from b_off and of the decay from a_off), a causal convolution of `taps` taps per channel
+    (conv_w float32 [C, taps]) and silu, unit vectors q (times q_scale) and k, then per head S <- g S, u = beta
+    (v - S^T k), S <- S + k u^T, o = S^T q.  `state` float32 [slots, conv_recurrence_state_floats(...)] holds S and
+    the convolution's tail between steps; out float32 [T, nh dv].
+
+    A step of long portions of few requests (GATED_DELTA_CHUNKS_FROM) goes through the kernels that take 16 tokens
+    of a request at a time; other steps walk token by token (`chunks` says which, for any step)."""
+    T, N = proj.shape
+    C = _recurrence_operands("gated_delta", proj, qkv_off, b_off, conv_w, a_log, dt_bias, state, out, n_heads, n_qk_heads,
+                             d, dv, taps, n_heads)
+    if a_off + n_heads > N:
         raise KernelError("gated_delta: the column offsets reach beyond the projection's rows")
-    act = step.buffer("gated_delta_act", (T, C + 2 * n_heads), torch.float32)
+    act = step.buffer("recurrence_act", (T, C + 2 * n_heads), torch.float32)
     if chunks is None:
-        chunks = T >= GATED_DELTA_CHUNKS_FROM * step.n_seqs and \
-            step.n_seqs * n_heads * -(-dv // 16) <= 3 * _sm_count(proj.device)
-    gram = step.buffer("gated_delta_gram", (T, n_qk_heads * 32 + n_heads * 16), torch.float32).data_ptr() if chunks else 0
+        chunks = _recurrence_in_chunks(step, T, n_heads, dv, proj.device)
+    gram = step.buffer("recurrence_gram", (T, n_qk_heads * 32 + n_heads * 16), torch.float32).data_ptr() if chunks else 0
     check(lib().rlis_gated_delta(proj.data_ptr(), proj.stride(0), int(qkv_off), int(b_off), int(a_off), conv_w.data_ptr(),
                                  a_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), state.stride(0),
-                                 step.cu_seqlens.data_ptr(), step.ctx_lens.data_ptr(), step.state_slots.data_ptr(),
-                                 step.seq_of_token.data_ptr(), act.data_ptr(), gram, out.data_ptr(), T, step.n_seqs, n_heads,
+                                 *_step_pointers(step), act.data_ptr(), gram, out.data_ptr(), T, step.n_seqs, n_heads,
                                  n_qk_heads, d, dv, taps, float(unit_eps), float(q_scale), _code(proj.dtype), _stream()),
           "gated_delta")
-    _count("gated_delta.prepare")
-    if chunks:
-        _count("gated_delta.gram")
-        _count("gated_delta.solve")
-    _count("gated_delta.chunks" if chunks else "gated_delta.scan")
+    _count_recurrence("gated_delta", chunks, True)
     return out
+
+
+def channel_delta(proj: torch.Tensor, qkv_off: int, b_off: int, decay: torch.Tensor, conv_w: torch.Tensor,
+                  a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step, n_heads: int,
+                  n_qk_heads: int, d: int, dv: int, taps: int, unit_eps: float, q_scale: float,
+                  chunks: bool | None = None) -> torch.Tensor:
+    """`gated_delta` with one decay a head and key channel: `decay` [T, n_heads d] holds the decay logits in proj's type
+    (may be a column slice of wider rows), g = exp(-exp(a_log_h) softplus(decay + dt_bias)) with dt_bias float32
+    [n_heads d], and S <- diag(g) S."""
+    T = proj.shape[0]
+    C = _recurrence_operands("channel_delta", proj, qkv_off, b_off, conv_w, a_log, dt_bias, state, out, n_heads,
+                             n_qk_heads, d, dv, taps, n_heads * d)
+    if decay.dtype != proj.dtype or tuple(decay.shape) != (T, n_heads * d) or decay.stride(1) != 1 or not decay.is_cuda:
+        raise KernelError("channel_delta: the decay logits must be [T, nh d] rows with unit stride in the projection's type")
+    act = step.buffer("recurrence_act", (T, C + n_heads + n_heads * d), torch.float32)
+    if chunks is None:
+        chunks = _recurrence_in_chunks(step, T, n_heads, dv, proj.device)
+    gram = scaled = 0
+    if chunks:
+        gram = step.buffer("recurrence_gram", (T, n_heads * 48), torch.float32).data_ptr()
+        scaled = step.buffer("recurrence_scaled", (T, n_heads * 4 * d), torch.float32).data_ptr()
+    check(lib().rlis_channel_delta(proj.data_ptr(), proj.stride(0), int(qkv_off), int(b_off), decay.data_ptr(),
+                                   decay.stride(0), 0, conv_w.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(),
+                                   state.data_ptr(), state.stride(0), *_step_pointers(step), act.data_ptr(), gram, scaled,
+                                   out.data_ptr(), T, step.n_seqs, n_heads, n_qk_heads, d, dv, taps, float(unit_eps),
+                                   float(q_scale), _code(proj.dtype), _stream()), "channel_delta")
+    _count_recurrence("channel_delta", chunks, True)
+    return out
+
+
+def state_space(proj: torch.Tensor, conv_off: int, dt_off: int, conv_w: torch.Tensor, conv_b: torch.Tensor | None,
+                a_log: torch.Tensor, dt_bias: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, out: torch.Tensor, step,
+                n_heads: int, n_groups: int, n_state: int, dv: int, taps: int, chunks: bool | None = None) -> torch.Tensor:
+    """The state-space recurrence of Mamba-2 over the step's tokens: from the rows of `proj` [T, N] (x | B | C from column
+    conv_off: n_heads heads of dv, then n_groups groups of n_state twice; one logit a head of the step size from dt_off), a
+    causal convolution of `taps` taps per channel (conv_w float32 [channels, taps], conv_b float32 [channels] or None) and
+    silu; dt = softplus(logit + dt_bias); per head S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C + skip x.  Head h reads
+    group h / (n_heads / n_groups).  `state` float32 [slots, conv_recurrence_state_floats(n_heads, n_groups, n_state, dv,
+    taps)]; out float32 [T, nh dv].  `chunks` as for `gated_delta`."""
+    T = proj.shape[0]
+    C = _recurrence_operands("state_space", proj, conv_off, dt_off, conv_w, a_log, dt_bias, state, out, n_heads, n_groups,
+                             n_state, dv, taps, n_heads)
+    _req(skip, "skip", torch.float32, (n_heads,))
+    if conv_b is not None:
+        _req(conv_b, "conv_b", torch.float32, (C,))
+    act = step.buffer("recurrence_act", (T, C + 2 * n_heads), torch.float32)
+    if chunks is None:
+        chunks = _recurrence_in_chunks(step, T, n_heads, dv, proj.device)
+    gram = step.buffer("recurrence_gram", (T, n_groups * 32), torch.float32).data_ptr() if chunks else 0
+    check(lib().rlis_state_space(proj.data_ptr(), proj.stride(0), int(conv_off), int(dt_off), conv_w.data_ptr(),
+                                 conv_b.data_ptr() if conv_b is not None else None, a_log.data_ptr(), dt_bias.data_ptr(),
+                                 skip.data_ptr(), state.data_ptr(), state.stride(0), *_step_pointers(step), act.data_ptr(),
+                                 gram, out.data_ptr(), T, step.n_seqs, n_heads, n_groups, n_state, dv, taps,
+                                 _code(proj.dtype), _stream()), "state_space")
+    _count_recurrence("state_space", chunks, False)
+    return out
+
+
+STREAM_NORMS = {"none": 0, "dynamic_tanh": 1, "rmsnorm": 2}
+MAX_STREAMS = 8
+
+
+class StreamNorm:
+    """The norm that `stream_mix` applies: kind "none", "dynamic_tanh" (tanh(alpha u) w + b) or "rmsnorm" (u / sqrt(mean
+    u^2 + eps) w); w, b float32 vectors."""
+
+    def __init__(self, kind: str = "none", w=None, b=None, alpha: float = 1.0, eps: float = 0.0):
+        if kind not in STREAM_NORMS:
+            raise KernelError(f"unknown norm {kind!r}; known: {sorted(STREAM_NORMS)}")
+        self.kind, self.w, self.b, self.alpha, self.eps = kind, w, b, float(alpha), float(eps)
+
+
+def stream_mix(x: torch.Tensor, n_streams: int, y: torch.Tensor | None = None, y_bias: torch.Tensor | None = None,
+               mix: torch.Tensor | None = None, out_coef: torch.Tensor | None = None, x_out: torch.Tensor | None = None,
+               in_coef: torch.Tensor | None = None, norm: StreamNorm | None = None, h: torch.Tensor | None = None,
+               u_out: torch.Tensor | None = None, rows: torch.Tensor | None = None):
+    """Residual streams side by side: with y, x_t <- sum_s mix[s, t] x_s + out_coef[t] (y + y_bias), all streams at once
+    from the old ones, into `x_out` (float32 [T, S, W]; None: not kept); then u = sum_t in_coef[t] x_t, h = norm(u) in h's
+    type and u_out = u in float32 (each only where given).  x float32 [T, S, W], or [T, W]: one row is every stream.  mix
+    float32 [S, S] (from, to; None: the streams stay themselves), out_coef and in_coef float32 [S] (None: ones).  `rows`
+    (int32 [R]): h and u_out are made for these rows, and the streams stay as they are."""
+    T, W, S = x.shape[0], x.shape[-1], int(n_streams)
+    _req(x, "x", torch.float32, (T, W) if x.dim() == 2 else (T, S, W))
+    if not 1 <= S <= MAX_STREAMS:
+        raise KernelError(f"stream_mix: one to {MAX_STREAMS} streams, got {S}")
+    n = T
+    if rows is not None:
+        _req(rows, "rows", torch.int32, (None,))
+        n = rows.shape[0]
+    dtype = y.dtype if y is not None else h.dtype if h is not None else torch.float32
+    if y is not None:
+        _req(y, "y", None, (T, W))
+    if x_out is not None:
+        _req(x_out, "x_out", torch.float32, (T, S, W))
+    for v, nm, shape in ((y_bias, "y_bias", (W,)), (mix, "mix", (S, S)), (out_coef, "out_coef", (S,)), (in_coef, "in_coef", (S,))):
+        if v is not None:
+            _req(v, nm, torch.float32, shape)
+    norm = norm or StreamNorm()
+    for v in (norm.w, norm.b):
+        if v is not None:
+            _req(v, "norm vector", torch.float32, (W,))
+    if h is not None:
+        _req(h, "h", dtype, (n, W))
+    if u_out is not None:
+        _req(u_out, "u_out", torch.float32, (n, W))
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    check(lib().rlis_stream_mix(x.data_ptr(), x.stride(0), 0 if x.dim() == 2 else W, S, ptr(y), ptr(y_bias), ptr(mix),
+                                ptr(out_coef), ptr(x_out), ptr(in_coef), STREAM_NORMS[norm.kind], norm.alpha, norm.eps,
+                                ptr(norm.w), ptr(norm.b), ptr(h), ptr(u_out), ptr(rows), n, W, _code(dtype), _stream()),
+          "stream_mix")
+    _count("stream_mix" + (".update" if y is not None else "") + (".rows" if rows is not None else ""))
+    return h if h is not None else u_out
 
 
 BIAS_ACTIVATIONS = {"none": 0, "relu2": 1}
@@ -724,67 +882,105 @@ class ResidualSink:
         self.resid, self.weight, self.eps = resid, weight, float(eps)
 
 
-def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = False, sink: ResidualSink | None = None,
-                slope: float = 1.0):
-    """y = x @ w^T for at most 128 rows of bfloat16 x: the decode step's weight-streaming product on
-    the tcgen05 tensor cores (TMA-fed, weights as the M side, k split over CTAs).  `swiglu4`: w is a
-    gate|up matrix interleaved in blocks of 4 rows and the result is silu(gate) * up, [M, N / 2]; with a `slope`,
-    gate sigmoid(slope gate) * up (+inf: max(gate, 0) * up).  `x` may be ScaledRows: the rows' scale is applied to the result.  `sink` (up to 16 rows): the
-    result, rounded to bfloat16, is added to sink.resid in place and the ScaledRows of the norm that
-    follows are returned instead of y."""
+class StreamsSink:
+    """The same for residual streams side by side and a norm without statistics (see `stream_mix`): the last product of a
+    part updates the streams `x` (float32 [T, S, W], or [T, W] for one row that is every stream) into `x_out` and hands on
+    the finished rows of the dynamic tanh that follows (`norm`, a StreamNorm), in bfloat16."""
+
+    def __init__(self, x, x_out, n_streams: int, mix, out_coef, in_coef, norm: StreamNorm):
+        if norm.kind != "dynamic_tanh":
+            raise KernelError("a sink over streams takes a norm without statistics")
+        self.x, self.x_out, self.n_streams, self.mix, self.out_coef, self.in_coef, self.norm = \
+            x, x_out, int(n_streams), mix, out_coef, in_coef, norm
+
+
+def _stream_rows(x: torch.Tensor, name: str) -> int:
+    """Elements between the rows of x ([M, K] bfloat16, unit stride, 16-byte rows)."""
+    if x.dtype != torch.bfloat16 or not x.is_cuda or x.dim() != 2 or x.stride(1) != 1 or x.stride(0) % 8 or x.data_ptr() % 16:
+        raise KernelError(f"{name}: expected bfloat16 rows on the device with unit stride, 16-byte aligned")
+    return x.stride(0)
+
+
+def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = False, sink=None, slope: float = 1.0,
+                bias: torch.Tensor | None = None):
+    """y = x @ w^T (+ bias, float32 [N]) for at most 128 rows of bfloat16 x: the decode step's weight-streaming product on
+    the tcgen05 tensor cores (TMA-fed, weights as the M side, k split over CTAs).  x may be a column slice of wider rows.
+    `swiglu4`: w is a gate|up matrix interleaved in blocks of 4 rows (bias in the same order) and the result is silu(gate)
+    * up, [M, N / 2]; with a `slope`, gate sigmoid(slope gate) * up (+inf: max(gate, 0) * up).  `x` may be ScaledRows: the
+    rows' scale is applied to the result.  `sink` (up to 16 rows), a ResidualSink: the
+    result, rounded to bfloat16 (+ bias), is added to sink.resid in place and the ScaledRows of the norm that
+    follows are returned instead of y; a StreamsSink: the streams are updated and the normed rows are returned."""
     scaled = x if isinstance(x, ScaledRows) else None
     if scaled is not None:
         x = scaled.x
     M, K = x.shape
     N = w.shape[0]
-    _req(x, "x", torch.bfloat16)
+    ldx = _stream_rows(x, "stream_gemm")
     _req(w, "w", torch.bfloat16, (N, K))
+    if bias is not None:
+        _req(bias, "bias", torch.float32, (N,))
+    bp = bias.data_ptr() if bias is not None else None
     if M > STREAM_MAX_ROWS or K % 8 or (swiglu4 and N % 8):
         raise KernelError(f"stream_gemm: takes up to {STREAM_MAX_ROWS} rows and K a multiple of 8, got M={M}, K={K}")
-    if scaled is None and sink is None:
-        out = torch.empty((M, N // 2 if swiglu4 else N), dtype=out_dtype, device=x.device)
-        check(lib().rlis_stream_gemm_bf16(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, _code(out_dtype),
-                                          1 if swiglu4 else 0, float(slope), _stream()), "stream_gemm")
-        _count("stream_gemm.swiglu" if swiglu4 else "stream_gemm")
-        return out
-    in_p, n_p, dim, eps = 0, 0, 0, 0.0
-    if scaled is not None:
-        if sink is not None:
-            raise KernelError("stream_gemm: scaled rows into a sink are not supported")
-        n_p = scaled.partials.shape[0]
-        _req(scaled.partials, "partials", torch.float32, (n_p, M))
-        if scaled.dim != K:
-            raise KernelError(f"stream_gemm: scaled rows of width {scaled.dim} for a product over {K}")
-        in_p, dim, eps = scaled.partials.data_ptr(), scaled.dim, scaled.eps
+    if sink is not None and (scaled is not None or swiglu4 or M > DECODE_GEMM_ROWS):
+        raise KernelError(f"stream_gemm: a sink takes a plain product of up to {DECODE_GEMM_ROWS} unscaled rows")
     if sink is None:
+        in_p, n_p, dim, eps = None, 0, 0, 0.0
+        if scaled is not None:
+            n_p = scaled.partials.shape[0]
+            _req(scaled.partials, "partials", torch.float32, (n_p, M))
+            if scaled.dim != K:
+                raise KernelError(f"stream_gemm: scaled rows of width {scaled.dim} for a product over {K}")
+            in_p, dim, eps = scaled.partials.data_ptr(), scaled.dim, scaled.eps
         out = torch.empty((M, N // 2 if swiglu4 else N), dtype=out_dtype, device=x.device)
-        check(lib().rlis_stream_gemm_fused(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, _code(out_dtype),
-                                           1 if swiglu4 else 0, in_p, n_p, dim, eps, 0, 0, 0, 0, float(slope), _stream()),
-              "stream_gemm")
-        _count("stream_gemm.scaled.swiglu" if swiglu4 else "stream_gemm.scaled")
+        check(lib().rlis_stream_gemm_fused(x.data_ptr(), ldx, w.data_ptr(), out.data_ptr(), M, N, K, _code(out_dtype),
+                                           1 if swiglu4 else 0, bp, in_p, n_p, dim, eps, None, None, None, None, float(slope),
+                                           _stream()), "stream_gemm")
+        _count("stream_gemm" + (".scaled" if scaled is not None else "") + (".swiglu" if swiglu4 else ""))
         return out
-    if swiglu4 or M > DECODE_GEMM_ROWS:
-        raise KernelError(f"stream_gemm: a sink takes a plain product of up to {DECODE_GEMM_ROWS} rows")
+    if isinstance(sink, StreamsSink):
+        S, nm = sink.n_streams, sink.norm
+        _req(sink.x, "sink.x", torch.float32, (M, N) if sink.x.dim() == 2 else (M, S, N))
+        _req(sink.x_out, "sink.x_out", torch.float32, (M, S, N))
+        for v, what, shape in ((sink.mix, "mix", (S, S)), (sink.out_coef, "out_coef", (S,)), (nm.w, "norm weight", (N,)),
+                               (nm.b, "norm bias", (N,))):
+            _req(v, "sink " + what, torch.float32, shape)
+        if sink.in_coef is not None:
+            _req(sink.in_coef, "sink in_coef", torch.float32, (S,))
+        h = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
+        check(lib().rlis_stream_gemm_streams(x.data_ptr(), ldx, w.data_ptr(), M, N, K, bp, sink.x.data_ptr(), sink.x.stride(0),
+                                             0 if sink.x.dim() == 2 else N, S, sink.mix.data_ptr(), sink.out_coef.data_ptr(),
+                                             sink.in_coef.data_ptr() if sink.in_coef is not None else None,
+                                             sink.x_out.data_ptr(), nm.alpha, nm.w.data_ptr(), nm.b.data_ptr(), h.data_ptr(),
+                                             _stream()), "stream_gemm")
+        _count("stream_gemm.streams")
+        return h
     _req(sink.resid, "sink.resid", torch.float32, (M, N))
     _req(sink.weight, "sink.weight", torch.float32, (N,))
     xn = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
     partials = torch.empty(((N + 127) // 128, M), dtype=torch.float32, device=x.device)
-    check(lib().rlis_stream_gemm_fused(x.data_ptr(), w.data_ptr(), 0, M, N, K, _code(torch.bfloat16), 2, 0, 0, 0, 0.0,
-                                       sink.resid.data_ptr(), sink.weight.data_ptr(), xn.data_ptr(),
+    check(lib().rlis_stream_gemm_fused(x.data_ptr(), ldx, w.data_ptr(), None, M, N, K, _code(torch.bfloat16), 2, bp, None, 0, 0,
+                                       0.0, sink.resid.data_ptr(), sink.weight.data_ptr(), xn.data_ptr(),
                                        partials.data_ptr(), 1.0, _stream()), "stream_gemm")
     _count("stream_gemm.sink")
     return ScaledRows(xn, partials, N, sink.eps)
 
 
-def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu: tuple | None = None) -> torch.Tensor:
+def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu: tuple | None = None,
+                 bias: torch.Tensor | None = None) -> torch.Tensor:
     """y = x @ w^T on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory), bfloat16
     operands.  epilogue "plain": bf16 [M, N]; "float32": float32 [M, N]; "swiglu4": w is a gate|up
     matrix interleaved in blocks of 4 rows and the result is silu(gate) * up, bf16 [M, N / 2]; "glu4":
-    the same layout with the gating of `glu` = (slope, limit or None, up_shift), see `glu_act`."""
+    the same layout with the gating of `glu` = (slope, limit or None, up_shift), see `glu_act`, after `bias` (float32 [N]
+    in the order of w's rows; this epilogue only) is added."""
     M, K = x.shape
     N = w.shape[0]
     _req(x, "x", torch.bfloat16)
     _req(w, "w", torch.bfloat16, (N, K))
+    if bias is not None:
+        _req(bias, "bias", torch.float32, (N,))
+        if epilogue != "glu4":
+            raise KernelError("gemm_tcgen05: the glu4 epilogue is the one that takes a bias")
     code = {"plain": 0, "swiglu4": 1, "float32": 2, "glu4": 3}[epilogue]
     gated = code in (1, 3)
     if M < 128 or N < 256 or K % 8 or N % (16 if gated else 8):
@@ -795,8 +991,8 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu:
     if code == 3:
         slope, limit, shift = glu
         check(lib().rlis_gemm_tcgen05_glu(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, float(slope),
-                                          float("inf") if limit is None else float(limit), float(shift), _stream()),
-              "gemm_tcgen05")
+                                          float("inf") if limit is None else float(limit), float(shift),
+                                          bias.data_ptr() if bias is not None else None, _stream()), "gemm_tcgen05")
     else:
         check(lib().rlis_gemm_tcgen05(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, code, _stream()),
               "gemm_tcgen05")
@@ -862,22 +1058,29 @@ def fuses_norms(n_rows: int, dtype, *widths: int) -> bool:
             and all(w % 8 == 0 for w in widths))
 
 
-def linear(x, w: torch.Tensor, out_dtype=None, sink: ResidualSink | None = None):
-    """y = x @ w^T for w stored (out, in).  float32: this package's FFMA kernel.  bfloat16: up to
-    16 rows go to this package's weight-streaming tcgen05 kernel, more to the library GEMM; both
+def linear(x, w: torch.Tensor, out_dtype=None, sink=None, bias: torch.Tensor | None = None):
+    """y = x @ w^T for w stored (out, in); x may be a column slice of wider rows.  float32: this package's FFMA kernel.
+    bfloat16: up to 16 rows go to this package's weight-streaming tcgen05 kernel, more to the library GEMM; both
     accumulate in float32, and `out_dtype=torch.float32` keeps that precision (used for logits).
-    ScaledRows as x and a `sink` are for the streaming kernel only (see `fuses_norms`)."""
+    ScaledRows as x and a `sink` (with an optional `bias` of the product) are for the streaming kernel only (see
+    `fuses_norms`)."""
     if isinstance(x, ScaledRows) or sink is not None:
         if not fuses_norms(x.shape[0], x.dtype, x.shape[1]):
             raise KernelError("linear: scaled rows or a sink with a product that does not take them")
-        return stream_gemm(x, w, out_dtype or torch.bfloat16, sink=sink)
+        return stream_gemm(x, w, out_dtype or torch.bfloat16, sink=sink, bias=bias)
+    if bias is not None:
+        raise KernelError("linear: a bias is taken with a sink")
     if x.dtype == torch.float32:
+        if not x.is_contiguous() and x.dim() == 2 and x.stride(1) == 1:
+            out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
+            gemm_f32_batched(x.unsqueeze(1), w.unsqueeze(0), out.unsqueeze(1))
+            return out
         return gemm_f32(x, w)
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError(f"linear: expected matching float32 or bfloat16 operands, got {x.dtype}, {w.dtype}")
     if not x.is_cuda:
         raise KernelError("linear: expected CUDA tensors; there is no CPU path")
-    if x.shape[1] % 8 == 0 and x.is_contiguous() and (
+    if x.shape[1] % 8 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0 and x.data_ptr() % 16 == 0 and (
             x.shape[0] <= STREAM_GEMM_ROWS or (x.shape[0] <= STREAM_MAX_ROWS and w.shape[0] >= 256 * num_sms())):
         # few rows, or up to 128 rows over a matrix so tall that the streaming kernel does not split k
         # (two tiles of 128 features an SM and more: an LM head).  Measured at 128256 x 2048: 48 rows
@@ -1176,18 +1379,21 @@ def attention(q, k_cache, v_cache, out, step, group: int, n_heads: int, n_kv_hea
 
 
 def glu_act(gate_up: torch.Tensor, out: torch.Tensor, slope: float = 1.0, limit: float | None = None,
-            up_shift: float = 0.0, interleave: int = 0) -> torch.Tensor:
+            up_shift: float = 0.0, interleave: int = 0, bias: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, i] = g sigmoid(slope g) (u + up_shift) with g = gate_up[t, i] and u = gate_up[t, I + i], both in
     float32 (slope +inf: max(g, 0) (u + up_shift)); with a `limit`, g is cut at limit from above and u clipped to [-limit, limit] first.
-    interleave B > 0: blocks of B gate columns each followed by their B columns of u."""
+    interleave B > 0: blocks of B gate columns each followed by their B columns of u.  `bias` (float32 [2 I] in the order
+    of gate_up's columns) is added to g and u before anything else."""
     T, I2 = gate_up.shape
     if I2 % 2:
         raise KernelError(f"glu_act: the stacked gate|up width must be even, got {I2}")
     _req(gate_up, "gate_up")
     _req(out, "out", gate_up.dtype, (T, I2 // 2))
+    if bias is not None:
+        _req(bias, "bias", torch.float32, (I2,))
     check(lib().rlis_glu_act(gate_up.data_ptr(), out.data_ptr(), T, I2 // 2, float(slope),
                              float("inf") if limit is None else float(limit), float(up_shift), int(interleave),
-                             _code(out.dtype), _stream()), "glu_act")
+                             bias.data_ptr() if bias is not None else None, _code(out.dtype), _stream()), "glu_act")
     _count("glu_act")
     return out
 
@@ -1248,6 +1454,32 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w, k
                                    1 if rot_half else 0, proj_bias.data_ptr() if proj_bias is not None else None,
                                    _code(proj.dtype), _stream()), "qk_norm_store")
     _count("qk_norm_store" + (".mix" if v_other is not None else "") + (".rot" if rot_dims else ""))
+    return q_out
+
+
+def qk_row_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w, k_w, eps: float, q_out: torch.Tensor,
+                      k_cache: torch.Tensor, v_cache: torch.Tensor, slots, n_heads: int, n_kv_heads: int, dim: int, v_dim: int,
+                      page_size: int) -> torch.Tensor:
+    """As `qk_norm_store` without its options, with queries and keys RMS-normed over all their heads together: q_w float32
+    [n_heads dim], k_w float32 [n_kv_heads dim] (None: no norm)."""
+    T, N = proj.shape
+    _req(proj, "proj")
+    _req(q_out, "q_out", proj.dtype, (T, n_heads * dim))
+    for w, nm, n in ((q_w, "q_w", n_heads * dim), (k_w, "k_w", n_kv_heads * dim)):
+        if w is not None:
+            _req(w, nm, torch.float32, (n,))
+    if v_off + n_kv_heads * v_dim > N or k_off + n_kv_heads * dim > N or q_off + n_heads * dim > N:
+        raise KernelError("qk_row_norm_store: the column offsets reach beyond the projection's rows")
+    if slots is not None:
+        _req(slots, "slots", torch.int32, (T,))
+        _req(k_cache, "k_cache", proj.dtype, (None, n_kv_heads, page_size, dim))
+        _req(v_cache, "v_cache", proj.dtype, (None, n_kv_heads, page_size, v_dim))
+    ptr = lambda t: t.data_ptr() if t is not None else None
+    check(lib().rlis_qk_row_norm_store(proj.data_ptr(), N, int(q_off), int(k_off), int(v_off), ptr(q_w), ptr(k_w), float(eps),
+                                       q_out.data_ptr(), k_cache.data_ptr() if slots is not None else None,
+                                       v_cache.data_ptr() if slots is not None else None, ptr(slots), T, n_heads, n_kv_heads,
+                                       dim, v_dim, page_size, _code(proj.dtype), _stream()), "qk_row_norm_store")
+    _count("qk_row_norm_store")
     return q_out
 
 

@@ -33,7 +33,11 @@ SIGNATURES = {
     "rlis_sum_norm": [P, P, F, P, P, F, P, F, P, P, I, I, F, F, I, P],
     "rlis_head_norm_gate": [P, P, P, LL, P, I, I, I, F, I, I, P],
     "rlis_gated_delta": [P, LL, I, I, I, P, P, P, P, LL, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, I, P],
-    "rlis_gated_delta_state_floats": [I, I, I, I, I],
+    "rlis_channel_delta": [P, LL, I, I, P, LL, I, P, P, P, P, LL, P, P, P, P, P, P, P, P, I, I, I, I, I, I, I, F, F, I, P],
+    "rlis_state_space": [P, LL, I, I, P, P, P, P, P, P, LL, P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, P],
+    "rlis_conv_recurrence_state_floats": [I, I, I, I, I],
+    "rlis_stream_mix": [P, LL, LL, I, P, P, P, P, P, P, I, F, F, P, P, P, P, P, I, I, I, P],
+    "rlis_gate_group_norm": [P, P, LL, P, P, I, I, I, F, I, P],
     "rlis_act_norm": [P, LL, I, P, P, LL, P, LL, I, I, F, I, P],
     "rlis_bias_act": [P, P, P, LL, I, I, I, P],
     "rlis_latent_kv_store": [P, LL, P, P, P, P, P, I, I, I, I, F, F, I, P, P, P, I, P],
@@ -47,6 +51,7 @@ SIGNATURES = {
     "rlis_recurrence_scan_rows": [P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, P, I, F, P, P, I, P],
     "rlis_recurrence_scan": [P, LL, I, I, I, I, P, P, P, P, P, P, I, I, I, I, I, P],
     "rlis_qk_norm_store": [P, LL, I, I, I, P, P, F, P, LL, F, P, P, P, P, I, I, I, I, I, I, P, I, F, P, F, I, I, P, I, P],
+    "rlis_qk_row_norm_store": [P, LL, I, I, I, P, P, F, P, P, P, P, I, I, I, I, I, I, I, P],
     "rlis_attention_bias": [P, P, P, P, P, I, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, I, I, P],
     "rlis_attention_bias_mma_takes": [I, I],
     "rlis_attention_bias_prefill": [P, P, P, P, P, I, P, LL, P, I, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P],
@@ -59,7 +64,7 @@ SIGNATURES = {
     "rlis_moe_gemm_mma": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, P],
     "rlis_moe_mma_takes_tile": [I],
     "rlis_moe_combine": [P, P, P, P, P, P, I, I, I, P, P, I, I, P],
-    "rlis_glu_act": [P, P, I, I, F, F, F, I, I, P],
+    "rlis_glu_act": [P, P, I, I, F, F, F, I, P, I, P],
     "rlis_rope_cache": [P, P, P, P, P, P, P, I, I, I, I, I, I, P],
     "rlis_attention_generic": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P],
     "rlis_attention_decode": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
@@ -73,9 +78,9 @@ SIGNATURES = {
     "rlis_sample_filtered": [P, P, P, I, I, LL, P],
     "rlis_nll_rows": [P, P, P, I, I, LL, P],
     "rlis_gemm_tcgen05": [P, P, P, I, I, I, I, P],
-    "rlis_gemm_tcgen05_glu": [P, P, P, I, I, I, F, F, F, P],
-    "rlis_stream_gemm_bf16": [P, P, P, I, I, I, I, I, F, P],
-    "rlis_stream_gemm_fused": [P, P, P, I, I, I, I, I, P, I, I, F, P, P, P, P, F, P],
+    "rlis_gemm_tcgen05_glu": [P, P, P, I, I, I, F, F, F, P, P],
+    "rlis_stream_gemm_fused": [P, LL, P, P, I, I, I, I, I, P, P, I, I, F, P, P, P, P, F, P],
+    "rlis_stream_gemm_streams": [P, LL, P, I, I, I, P, P, LL, LL, I, P, P, P, P, F, P, P, P, P],
     "rlis_take_errors": [P, P],
     "rlis_stream_gemm_timeline": [I],
     "rlis_stream_gemm_timeline_read": [P, P],

@@ -1,7 +1,8 @@
 """Causal grouped-query attention with per-head RMS norms of queries and keys, a learned bias by
 distance, values of their own width that a layer may mix with another layer's, and a gate on every head's
 output; optionally a rotation of part of every head before the norms, keys that double as values, a query
-temperature by position, a penalty linear in the distance, a window, and a sink in the softmax."""
+temperature by position, a penalty linear in the distance, a window, a sink in the softmax, and norms over the whole
+projections."""
 
 from __future__ import annotations
 
@@ -103,6 +104,16 @@ class BiasedAttention(Mixer):
             raise ValueError("a head's output is gated as a whole or channel by channel, not both")
         self.gate_cols = spec.n_heads * spec.v_dim if spec.out_gate is not None else spec.n_heads
         self.proj_bias = None
+        if spec.sink_score is not None:
+            if spec.sink is not None:
+                raise ValueError("a sink's score is one number for all heads or a tensor, not both")
+            self.sinks = torch.full((spec.n_heads,), float(spec.sink_score), dtype=torch.float32, device=device)
+        if spec.norm_over not in ("head", "projection"):
+            raise ValueError(f"queries and keys are normed over a 'head' or the 'projection', not {spec.norm_over!r}")
+        self.row_norm = spec.norm_over == "projection"
+        if self.row_norm and (spec.unit_norm or spec.rotation is not None or spec.q_temp is not None or spec.value_mix is not None
+                              or spec.v_proj is None or spec.q_bias is not None or spec.k_bias is not None or spec.v_bias is not None):
+            raise ValueError("a norm over the whole projection takes no rotation, temperature, bias or shared values")
 
     def tensors(self) -> dict:
         s = self.spec
@@ -113,9 +124,9 @@ class BiasedAttention(Mixer):
         if s.sink is not None:
             out[s.sink] = (s.n_heads,)
         if s.q_norm is not None:
-            out[s.q_norm] = (s.dim,)
+            out[s.q_norm] = (s.n_heads * s.dim if self.row_norm else s.dim,)
         if s.k_norm is not None:
-            out[s.k_norm] = (s.dim,)
+            out[s.k_norm] = (s.n_kv_heads * s.dim if self.row_norm else s.dim,)
         if s.bias is not None:
             out[s.bias.table] = (s.bias.rows, s.n_heads)
         if s.head_gate is not None:
@@ -180,7 +191,11 @@ class BiasedAttention(Mixer):
         s = self.spec
         return ops.biased_decode_pieces(step.n_decode, s.n_kv_heads, step.max_decode_ctx)
 
-    def forward(self, x, step, cache, state, writes_cache=True):
+    def fuses_norms(self, step) -> bool:
+        s = self.spec
+        return ops.fuses_norms(step.n_tokens, self.dtype, s.hidden, s.n_heads * s.v_dim)
+
+    def forward(self, x, step, cache, state, writes_cache=True, sink=None):
         s = self.spec
         T = x.shape[0]
         with span("q|k|v|gate proj"):
@@ -194,11 +209,15 @@ class BiasedAttention(Mixer):
                 raise RuntimeError("a layer mixes in another layer's values, and no layer of this step has left any")
         q = step.buffer("attn_q", (T, s.n_heads * s.dim), self.dtype)
         with span("q, k norms + value mix + kv write"):
-            ops.qk_norm_store(proj, self.q_off, self.k_off, self.v_off, self.q_w, self.k_w, self.eps, other, self.lam, q,
-                              cache.k, cache.v, step.slots[cache.group] if writes_cache else None, s.n_heads,
-                              s.n_kv_heads, s.dim, s.v_dim, cache.page_size, rotation=self.rotation,
-                              positions=step.positions, q_temp=self.q_temp, rot_half=self.rot_half,
-                              proj_bias=self.proj_bias)
+            slots = step.slots[cache.group] if writes_cache else None
+            if self.row_norm:
+                ops.qk_row_norm_store(proj, self.q_off, self.k_off, self.v_off, self.q_w, self.k_w, self.eps, q, cache.k,
+                                      cache.v, slots, s.n_heads, s.n_kv_heads, s.dim, s.v_dim, cache.page_size)
+            else:
+                ops.qk_norm_store(proj, self.q_off, self.k_off, self.v_off, self.q_w, self.k_w, self.eps, other, self.lam, q,
+                                  cache.k, cache.v, slots, s.n_heads, s.n_kv_heads, s.dim, s.v_dim, cache.page_size,
+                                  rotation=self.rotation, positions=step.positions, q_temp=self.q_temp,
+                                  rot_half=self.rot_half, proj_bias=self.proj_bias)
         o = step.buffer("attn_o", (T, s.n_heads * s.v_dim), self.dtype)
         gate = proj[:, self.g_off:self.g_off + self.gate_cols] if (s.head_gate is not None or s.out_gate is not None) else None
         with span("attention"):
@@ -206,7 +225,7 @@ class BiasedAttention(Mixer):
                                  s.dim, s.v_dim, cache.page_size, self.scale, self.window, sinks=self.sinks,
                                  slopes=self.slopes)
         with span("o proj"):
-            return ops.linear(o, self.w_o)
+            return ops.linear(o, self.w_o, sink=sink)
 
 
 register_mixer("biased_attention", BiasedAttention)

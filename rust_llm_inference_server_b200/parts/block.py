@@ -16,6 +16,7 @@ from __future__ import annotations
 import torch
 
 from .. import ops
+from ..ops.profile import span
 from .base import (Part, build_feed_forward, build_mixer, build_norm, register_arrangement)
 
 
@@ -226,6 +227,153 @@ class PostNormBlock:
         return resid, (StreamRows(h) if chained else None)
 
 
+class HyperBlock:
+    """Pre-norm sublayers over S residual streams (hyper-connections).  A sublayer reads norm(sum_s read[s] x_s); its
+    result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, all streams at once.  The streams are float32: one
+    kernel updates them with a sublayer's result and makes the normed input of the sublayer that follows, also when that
+    is the first sublayer of the next block of this kind (a block returns `Streams` with that update pending).  The
+    streams start equal, so the first kernel reads the embedding's row as every stream.  In steps of a few rows, where
+    the norm that follows needs no statistics, the part's last product does the update and the norm in its epilogue
+    (`ops.StreamsSink`).  After the last block the final norm reads the sum of the streams; a block of another
+    arrangement that follows gets that sum as its residual stream."""
+
+    chains_norms = True      # `forward` takes `next_block`
+
+    def __init__(self, spec, dtype, device):
+        self.dtype = dtype
+        self.hidden = spec.norm1.dim
+        self.norm1 = build_norm(spec.norm1, dtype, device)
+        self.mixer = build_mixer(spec.mixer, dtype, device)
+        self.feed_forward = build_feed_forward(spec.feed_forward, dtype, device) if spec.feed_forward is not None else None
+        self.norm2 = build_norm(spec.norm2, dtype, device) if self.feed_forward is not None else None
+        if spec.hyper1 is None or (self.feed_forward is not None and spec.hyper2 is None):
+            raise ValueError("the hyper arrangement takes the coefficients of every sublayer (HyperSpec)")
+        self.streams = int(spec.hyper1.streams)
+        if not 1 <= self.streams <= ops.MAX_STREAMS:
+            raise ValueError(f"one to {ops.MAX_STREAMS} residual streams, got {self.streams}")
+        if self.feed_forward is not None and int(spec.hyper2.streams) != self.streams:
+            raise ValueError("both sublayers of a block run over the same streams")
+        self.hyper1 = _HyperTensors(spec.hyper1)
+        self.hyper2 = _HyperTensors(spec.hyper2) if self.feed_forward is not None else None
+        for n in (self.norm1, self.norm2):
+            if n is not None and not hasattr(n, "stream_norm"):
+                raise ValueError("the hyper arrangement takes norms that `ops.stream_mix` knows")
+
+    def entry_sink(self, resid, step):
+        return None          # nothing of an ordinary residual stream is left to the product before this block
+
+    def entry_streams(self, step, n_streams: int):
+        """For the part that runs before this block over the same streams: what it would have to read them with."""
+        return (self.hyper1.read, self.norm1) if n_streams == self.streams else None
+
+    def parts(self):
+        return tuple(p for p in (self.hyper1, self.norm1, self.mixer, self.hyper2, self.norm2, self.feed_forward)
+                     if p is not None)
+
+    def _join(self, part, run, streams, hyper, step, follows, bias=None):
+        """Runs a sublayer and hands its result to the streams: in its last product where that can, else pending."""
+        if follows is not None and part.fuses_norms(step):
+            sink = streams.sink(hyper, follows, step, self.dtype)
+            if sink is not None:
+                return streams.normed_by(run(sink=sink), sink)
+        return streams.pending(run() if bias is None else run(defer_bias=True), bias, hyper)
+
+    def forward(self, resid, pending, step, cache, state, writes_cache=True, next_block=None):
+        if isinstance(pending, Streams):
+            streams = pending
+        else:
+            if pending is not None:      # a block of another arrangement has left its last addition
+                ops.stream_mix(resid, 1, y=pending, x_out=resid.unsqueeze(1))
+            streams = Streams(resid, self.streams)
+        ask = getattr(next_block, "entry_streams", None)
+        after = ask(step, self.streams) if ask is not None else None
+        h = streams.read((self.hyper1.read, self.norm1), step, self.dtype)
+        mid = (self.hyper2.read, self.norm2) if self.feed_forward is not None else after
+        streams = self._join(self.mixer, lambda **k: self.mixer.forward(h, step, cache, state, writes_cache, **k), streams,
+                             self.hyper1, step, mid)
+        if self.feed_forward is not None:
+            h2 = streams.read(mid, step, self.dtype)
+            streams = self._join(self.feed_forward, lambda **k: self.feed_forward.forward(h2, step, **k), streams,
+                                 self.hyper2, step, after, getattr(self.feed_forward, "b_down", None))
+        if ask is None:                  # whoever comes next knows nothing of streams
+            streams.total(out=resid)
+            return resid, None
+        return resid, streams
+
+
+class Streams:
+    """The residual streams of a step between two sublayers: `x` float32 [T, S, W] (or [T, W]: one row that is every
+    stream), perhaps with a sublayer's result still to be joined, or with the next sublayer's normed input already made."""
+
+    def __init__(self, x, n: int, y=None, bias=None, hyper=None, rows=None):
+        self.x, self.n, self.y, self.bias, self.hyper, self.rows = x, n, y, bias, hyper, rows
+
+    def _update(self) -> dict:
+        if self.y is None:
+            return {}
+        return {"y": self.y, "y_bias": self.bias, "mix": self.hyper.mix, "out_coef": self.hyper.write}
+
+    def _home(self, step):
+        return step.buffer("streams", (self.x.shape[0], self.n, self.x.shape[-1]), torch.float32)
+
+    def pending(self, y, bias, hyper) -> "Streams":
+        return Streams(self.x, self.n, y, bias, hyper)
+
+    def normed_by(self, rows, sink) -> "Streams":
+        return Streams(sink.x_out, self.n, rows=rows)
+
+    def read(self, how, step, dtype):
+        """The normed input of the sublayer that reads the streams by `how` = (coefficients, norm)."""
+        if self.rows is not None:
+            return self.rows
+        coef, norm = how
+        h = step.buffer("norm_out", (self.x.shape[0], self.x.shape[-1]), dtype)
+        update = self._update()
+        x_out = self._home(step) if update else None
+        with span("streams + norm"):
+            ops.stream_mix(self.x, self.n, x_out=x_out, in_coef=coef, norm=norm.stream_norm(), h=h, **update)
+        if update:
+            self.x, self.y = x_out, None
+        return h
+
+    def sink(self, hyper, follows, step, dtype):
+        coef, norm = follows
+        sn = norm.stream_norm()
+        if sn.kind != "dynamic_tanh" or self.y is not None or not ops.fuses_norms(self.x.shape[0], dtype, self.x.shape[-1]):
+            return None
+        return ops.StreamsSink(self.x, self._home(step), self.n, hyper.mix, hyper.write, coef, sn)
+
+    def normed_rows(self, norm, step, rows, dtype):
+        """The rows `rows` of the streams' sum after `norm` (what the LM head reads)."""
+        if self.rows is not None:        # made by the last product, for all rows of the step in order
+            return self.rows
+        out = step.buffer("norm_rows_out", (rows.shape[0], self.x.shape[-1]), dtype)
+        with span("streams + norm"):
+            return ops.stream_mix(self.x, self.n, norm=norm.stream_norm(), h=out, rows=rows, **self._update())
+
+    def total(self, out=None):
+        """The sum of the streams, float32 [T, W]."""
+        out = out if out is not None else torch.empty((self.x.shape[0], self.x.shape[-1]), dtype=torch.float32, device=self.x.device)
+        return ops.stream_mix(self.x, self.n, u_out=out, **self._update())
+
+
+class _HyperTensors(Part):
+    """The coefficients of one sublayer's hyper-connection."""
+
+    graph_safe = True
+
+    def __init__(self, spec):
+        self.spec = spec
+
+    def tensors(self) -> dict:
+        s = self.spec
+        return {s.read: (s.streams,), s.write: (s.streams,), s.mix: (s.streams, s.streams)}
+
+    def load(self, src) -> None:
+        s = self.spec
+        self.read, self.write, self.mix = (src.get(n, "vector").contiguous() for n in (s.read, s.write, s.mix))
+
+
 class StreamRows:
     """What an outnorm block hands the next one: `x`, the (complete) residual stream in the compute type."""
 
@@ -264,3 +412,4 @@ register_arrangement("prenorm", PreNormBlock)
 register_arrangement("sandwich", SandwichBlock)
 register_arrangement("outnorm", OutNormBlock)
 register_arrangement("postnorm", PostNormBlock)
+register_arrangement("hyper", HyperBlock)

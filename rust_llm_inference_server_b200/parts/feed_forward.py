@@ -25,15 +25,27 @@ class SwiGLU(FeedForward):
         # one); a clipping limit or a shifted linear branch go through the gating kernel that takes them as parameters
         self.slope = float(getattr(spec, "slope", 1.0))
         self.plain = getattr(spec, "limit", None) is None and float(getattr(spec, "up_shift", 0.0)) == 0.0
+        self.b_gate_up = self.b_down = None
+        if (getattr(spec, "gate_bias", None) is None) != (getattr(spec, "up_bias", None) is None):
+            raise ValueError("a gated unit has biases on both of its first projections or on neither")
 
     def tensors(self) -> dict:
         s = self.spec
-        return {s.gate_proj: (s.intermediate, s.hidden), s.up_proj: (s.intermediate, s.hidden),
-                s.down_proj: (s.hidden, s.intermediate)}
+        out = {s.gate_proj: (s.intermediate, s.hidden), s.up_proj: (s.intermediate, s.hidden),
+               s.down_proj: (s.hidden, s.intermediate)}
+        for name, n in ((s.gate_bias, s.intermediate), (s.up_bias, s.intermediate), (s.down_bias, s.hidden)):
+            if name is not None:
+                out[name] = (n,)
+        return out
 
     def load(self, src) -> None:
         s = self.spec
         g, u = src.get(s.gate_proj), src.get(s.up_proj)
+        if s.gate_bias is not None:      # in the order of the stacked matrix's rows
+            bg, bu = src.get(s.gate_bias, "vector"), src.get(s.up_bias, "vector")
+            self.b_gate_up = torch.stack([bg.view(-1, 4), bu.view(-1, 4)], dim=1).reshape(-1).contiguous() \
+                if s.intermediate % 4 == 0 else torch.cat([bg, bu]).contiguous()
+        self.b_down = src.get(s.down_bias, "vector").contiguous() if s.down_bias is not None else None
         self.interleave = 4 if s.intermediate % 4 == 0 else 0
         if self.interleave:
             self.w_gate_up = torch.stack([g.view(-1, 4, s.hidden), u.view(-1, 4, s.hidden)], dim=1) \
@@ -45,41 +57,37 @@ class SwiGLU(FeedForward):
     def fuses_norms(self, step) -> bool:
         return self.plain and ops.fuses_norms(step.n_tokens, self.dtype, self.spec.hidden, self.spec.intermediate)
 
-    def forward(self, x, step, sink=None):
-        if not self.plain:
-            s = self.spec
-            if (self.dtype == torch.bfloat16 and self.interleave == 4 and s.hidden % 8 == 0 and x.shape[0] >= 128
-                    and s.intermediate % 128 == 0):
-                # prefill: the tcgen05 product with the clipped gating in its epilogue
-                with span("mlp gate+up, clipped gating"):
-                    act = ops.gemm_tcgen05(x, self.w_gate_up, "glu4", glu=(s.slope, s.limit, s.up_shift))
-            else:
-                with span("mlp gate+up"):
-                    gu = ops.linear(x, self.w_gate_up)
-                with span("clipped gating"):
-                    act = step.buffer("ffn_act", (x.shape[0], s.intermediate), self.dtype)
-                    ops.glu_act(gu, act, s.slope, s.limit, s.up_shift, self.interleave)
-            with span("mlp down proj"):
-                return ops.linear(act, self.w_down)
-        fusable = self.dtype == torch.bfloat16 and self.interleave == 4 and self.spec.hidden % 8 == 0
-        silu = self.slope == 1.0
-        with span("mlp gate+up, silu*up" if silu else "mlp gate+up, gate*up"):
-            if fusable and x.shape[0] <= ops.STREAM_GEMM_ROWS:
-                act = ops.stream_gemm(x, self.w_gate_up, swiglu4=True, slope=self.slope)   # product and gating in one kernel
-            elif fusable and x.shape[0] >= 128 and self.spec.intermediate % 128 == 0:
-                # prefill: the tcgen05 product with the gating in its epilogue (the gate|up activations
-                # never reach HBM)
-                act = ops.gemm_tcgen05(x, self.w_gate_up, "swiglu4") if silu \
-                    else ops.gemm_tcgen05(x, self.w_gate_up, "glu4", glu=(self.slope, None, 0.0))
-            else:
-                gu = ops.linear(x, self.w_gate_up)
-                act = step.buffer("ffn_act", (x.shape[0], self.spec.intermediate), self.dtype)
-                if silu:
-                    ops.swiglu(gu, act, self.interleave)
-                else:
-                    ops.glu_act(gu, act, self.slope, None, 0.0, self.interleave)
+    def _activation(self, x, step):
+        """The gated activations [T, intermediate] of the first product."""
+        s = self.spec
+        T = x.shape[0]
+        limit, shift = getattr(s, "limit", None), float(getattr(s, "up_shift", 0.0))
+        fusable = self.dtype == torch.bfloat16 and self.interleave == 4 and s.hidden % 8 == 0
+        silu = self.plain and self.slope == 1.0 and self.b_gate_up is None
+        if fusable and self.plain and T <= ops.STREAM_GEMM_ROWS:
+            # product and gating in one kernel
+            return ops.stream_gemm(x, self.w_gate_up, swiglu4=True, slope=self.slope, bias=self.b_gate_up)
+        if fusable and T >= 128 and s.intermediate % 128 == 0:
+            # prefill: the tcgen05 product with the gating in its epilogue (the gate|up activations never reach HBM)
+            return ops.gemm_tcgen05(x, self.w_gate_up, "swiglu4") if silu \
+                else ops.gemm_tcgen05(x, self.w_gate_up, "glu4", glu=(self.slope, limit, shift), bias=self.b_gate_up)
+        gu = ops.linear(x, self.w_gate_up)
+        act = step.buffer("ffn_act", (T, s.intermediate), self.dtype)
+        if silu:
+            return ops.swiglu(gu, act, self.interleave)
+        return ops.glu_act(gu, act, self.slope, limit, shift, self.interleave, bias=self.b_gate_up)
+
+    def forward(self, x, step, sink=None, defer_bias: bool = False):
+        """With `defer_bias` the caller adds `self.b_down` itself (in float32, while it joins the result)."""
+        with span("mlp gate+up, gating"):
+            act = self._activation(x, step)
         with span("mlp down proj"):
-            return ops.linear(act, self.w_down, sink=sink)
+            if sink is not None:
+                return ops.linear(act, self.w_down, sink=sink, bias=self.b_down)
+            y = ops.linear(act, self.w_down)
+            if self.b_down is not None and not defer_bias:
+                y = ops.bias_act(y, self.b_down, step.buffer("ffn_out", tuple(y.shape), self.dtype), "none")
+            return y
 
 
 class DenseFF(FeedForward):

@@ -1,4 +1,4 @@
-"""RMSNorm over the float32 residual stream (crates/model/src/layers.rs:103-146)."""
+"""Norms over the float32 residual stream: RMSNorm (crates/model/src/layers.rs:103-146) and the dynamic tanh."""
 
 from __future__ import annotations
 
@@ -49,4 +49,46 @@ class RMSNorm(Norm):
         return ops.ResidualSink(resid, self.weight, self.eps)
 
 
+    def stream_norm(self):
+        """This norm as `ops.stream_mix` takes it."""
+        return ops.StreamNorm("rmsnorm", self.weight, eps=self.eps)
+
+
+class DynamicTanh(Norm):
+    """y = tanh(alpha x) * w + b, in float32: no mean and no variance, so nothing of a row has to be known before its
+    entries can be written (and a product's epilogue can apply it, see `ops.StreamsSink`)."""
+
+    graph_safe = True
+
+    def __init__(self, spec, dtype, device):
+        self.dim = spec.dim
+        self.spec = spec
+        self.dtype = dtype
+
+    def tensors(self) -> dict:
+        s = self.spec
+        return {s.weight: (s.dim,), s.bias: (s.dim,), s.alpha: ()}
+
+    def load(self, src) -> None:
+        s = self.spec
+        self.weight = src.get(s.weight, "vector").contiguous()
+        self.bias = src.get(s.bias, "vector").contiguous()
+        self.alpha = float(src.get(s.alpha, "vector").reshape(-1)[0].item())
+
+    def stream_norm(self):
+        return ops.StreamNorm("dynamic_tanh", self.weight, self.bias, self.alpha)
+
+    def forward(self, resid, delta, step):
+        out = step.buffer("norm_out", (resid.shape[0], self.dim), self.dtype)
+        with span("residual add + dynamic tanh"):
+            return ops.stream_mix(resid, 1, y=delta, x_out=resid.unsqueeze(1) if delta is not None else None,
+                                  norm=self.stream_norm(), h=out)
+
+    def forward_rows(self, resid, delta, step, rows):
+        out = step.buffer("norm_rows_out", (rows.shape[0], self.dim), self.dtype)
+        with span("residual add + dynamic tanh"):
+            return ops.stream_mix(resid, 1, y=delta, norm=self.stream_norm(), h=out, rows=rows)
+
+
 register_norm("rmsnorm", RMSNorm)
+register_norm("dynamic_tanh", DynamicTanh)

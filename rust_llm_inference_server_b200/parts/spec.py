@@ -25,6 +25,17 @@ class RMSNormSpec:
 
 
 @dataclass(frozen=True)
+class DynamicTanhSpec:
+    """y = tanh(alpha x) * w + b: a norm that computes no mean or variance.  `alpha` names a scalar tensor, `weight` and
+    `bias` vectors of shape (dim,)."""
+    dim: int
+    weight: str
+    bias: str
+    alpha: str
+    kind: str = "dynamic_tanh"
+
+
+@dataclass(frozen=True)
 class RopeSpec:
     """Rotate-half rotary encoding; `scaling` as in config.RopeScaling (llama3) or None.  `head_dim` is the number
     of entries that turn (entry i with entry i + head_dim / 2): a mixer that rotates itself may apply it to the
@@ -111,7 +122,10 @@ class BiasedAttentionSpec:
     `sink` (n_heads,): exp(sink_h) joins the denominator of head h's softmax, without a key or a value.
     `rotation` may also be a rotate-half spec (`RopeSpec`, or a yarn spec with pairing "half").  `q_bias`, `k_bias`,
     `v_bias`: biases of the three projections.  `out_gate` (n_heads * v_dim, hidden): every channel of every head's
-    output is multiplied by sigmoid of its row applied to the mixer's input (instead of `head_gate`)."""
+    output is multiplied by sigmoid of its row applied to the mixer's input (instead of `head_gate`).  `norm_over`
+    "projection": queries (and keys) are normed over all their heads together before they are split into heads; `q_norm` is
+    then (n_heads * dim,) and `k_norm` (n_kv_heads * dim,).  `sink_score`: a number, exp of which joins the denominator of
+    every head's softmax (instead of `sink`)."""
     hidden: int
     n_heads: int
     n_kv_heads: int
@@ -139,6 +153,8 @@ class BiasedAttentionSpec:
     k_bias: Optional[str] = None     # (n_kv_heads * dim,)
     v_bias: Optional[str] = None     # (n_kv_heads * v_dim,)
     out_gate: Optional[str] = None   # (n_heads * v_dim, hidden)
+    norm_over: str = "head"          # "head" or "projection"
+    sink_score: Optional[float] = None
     kind: str = "biased_attention"
 
 
@@ -246,7 +262,11 @@ class GatedDeltaSpec:
     last tap on the current token) and silu; q and k become unit vectors per head (x / sqrt(sum x^2 + unit_eps)),
     q times dim^(-1/2); beta = sigmoid(W_b h) and decay g = exp(-exp(a_log) softplus(W_a h + dt_bias)), one a
     head; per head S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q (float32 state per request); out =
-    W_o (rmsnorm_per_head(o) * out_norm * silu(W_g h)).  Head h reads q and k of head h / (n_heads / n_qk_heads)."""
+    W_o (rmsnorm_per_head(o) * out_norm * silu(W_g h)).  Head h reads q and k of head h / (n_heads / n_qk_heads).
+
+    `channel_decay`: one decay a head and key channel; W_a and dt_bias then have n_heads * dim rows, and S <- diag(g) S.
+    `decay_down` / `gate_down` (rank, hidden): the decay logits are W_a (W_a_down h), the gate's W_g (W_g_down h), so W_a and
+    W_g have `rank` columns (the checkpoint says how many).  `gate_act`: "silu" or "sigmoid"."""
     hidden: int
     n_heads: int
     n_qk_heads: int
@@ -268,7 +288,37 @@ class GatedDeltaSpec:
     out_norm: str                    # (v_dim,)
     o_proj: str                      # (hidden, n_heads * v_dim)
     unit_eps: float = 1e-6
+    channel_decay: bool = False
+    decay_down: Optional[str] = None  # (rank, hidden)
+    gate_down: Optional[str] = None   # (rank, hidden)
+    gate_act: str = "silu"
     kind: str = "gated_delta"
+
+
+@dataclass(frozen=True)
+class StateSpaceSpec:
+    """The state-space mixer of Mamba-2.  One projection makes z | x | B | C | dt (n_heads * v_dim twice, n_groups * n_state
+    twice, n_heads); x, B and C pass a causal convolution over time per channel (`conv` taps and a bias) and silu; dt =
+    softplus(dt + dt_bias); per head (group h / (n_heads / n_groups)) S <- exp(-exp(a_log) dt) S + dt B x^T, y = S^T C +
+    skip x (float32 state per request); out = W_o (norm(y silu(z)) * out_norm), the norm an RMS norm of each of
+    `norm_groups` equal parts."""
+    hidden: int
+    n_heads: int
+    n_groups: int
+    n_state: int
+    v_dim: int
+    conv: int
+    norm_groups: int
+    eps: float
+    in_proj: str                     # (2 n_heads v_dim + 2 n_groups n_state + n_heads, hidden)
+    conv_weight: str                 # (n_heads v_dim + 2 n_groups n_state, conv)
+    conv_bias: Optional[str]         # (n_heads v_dim + 2 n_groups n_state,)
+    a_log: str                       # (n_heads,)
+    dt_bias: str                     # (n_heads,)
+    skip: str                        # (n_heads,)
+    out_norm: str                    # (n_heads v_dim,)
+    o_proj: str                      # (hidden, n_heads v_dim)
+    kind: str = "state_space"
 
 
 @dataclass(frozen=True)
@@ -303,7 +353,8 @@ class DenseFFSpec:
 class SwiGLUSpec:
     """W_down (g sigmoid(slope g) (u + up_shift)) with g = W_gate h and u = W_up h; with a `limit`, g is
     cut at limit from above and u clipped to [-limit, limit] first.  The defaults are SwiGLU.  A `slope` of
-    +infinity is the limit max(g, 0) (u + up_shift): a unit gated by relu."""
+    +infinity is the limit max(g, 0) (u + up_shift): a unit gated by relu.  `gate_bias`, `up_bias` (both or neither) are
+    added to g and u before anything else, `down_bias` to the result."""
     hidden: int
     intermediate: int
     gate_proj: str                   # (intermediate, hidden)
@@ -312,6 +363,9 @@ class SwiGLUSpec:
     slope: float = 1.0
     limit: Optional[float] = None
     up_shift: float = 0.0
+    gate_bias: Optional[str] = None  # (intermediate,)
+    up_bias: Optional[str] = None    # (intermediate,)
+    down_bias: Optional[str] = None  # (hidden,)
     kind: str = "swiglu"
 
 
@@ -381,6 +435,16 @@ class LMHeadSpec:
 
 
 @dataclass(frozen=True)
+class HyperSpec:
+    """The coefficients of one sublayer's hyper-connection over S residual streams: the sublayer reads u = sum_s read[s]
+    x_s and its result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, all streams at once."""
+    streams: int
+    read: str                        # (streams,)
+    write: str                       # (streams,)
+    mix: str                         # (streams, streams), [from, to]
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One block.  arrangement "prenorm": x += mixer(norm1(x)); x += feed_forward(norm2(x))
     (crates/model/src/llama.rs:264-271; `feed_forward` None leaves the second line out, norm2 is then None too).
@@ -391,7 +455,9 @@ class LayerSpec:
     stream itself and only their results are normed, x += residual_mult * norm1(mixer(x)), then x +=
     residual_mult * norm2(feed_forward(x)), the second line only with a feed-forward.  arrangement "postnorm": the
     sum is normed, x = norm1(stream_mult * x + mixer(x)), then x = norm2(stream_mult * x + feed_forward(x)), the
-    sublayers reading x itself and the second line only with a feed-forward."""
+    sublayers reading x itself and the second line only with a feed-forward.  arrangement "hyper": pre-norm sublayers over
+    several residual streams, joined as `hyper1` and `hyper2` (HyperSpec) say; the streams start equal, and the layers that
+    follow (or the final norm) read their sum."""
     norm1: Any
     mixer: Any
     norm2: Any
@@ -403,6 +469,8 @@ class LayerSpec:
     scale2: Optional[str] = None
     residual_mult: float = 1.0
     stream_mult: float = 1.0
+    hyper1: Optional[HyperSpec] = None
+    hyper2: Optional[HyperSpec] = None
 
 
 @dataclass(frozen=True)
