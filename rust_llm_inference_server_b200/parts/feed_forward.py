@@ -79,7 +79,7 @@ class SwiGLU(FeedForward):
 
     def forward(self, x, step, sink=None, defer_bias: bool = False):
         """With `defer_bias` the caller adds `self.b_down` itself (in float32, while it joins the result)."""
-        with span("mlp gate+up, gating"):
+        with span("mlp gate+up, silu*up" if self.plain and self.slope == 1.0 else "mlp gate+up, gate*up"):
             act = self._activation(x, step)
         with span("mlp down proj"):
             if sink is not None:
