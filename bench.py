@@ -1009,12 +1009,157 @@ def workload_rumedra(args, torch, np) -> dict:
     four Lanirax layers (the closest model: a parallel mixer of window attention and a recurrence, routed feed-forwards)
     and four Llama layers of the same width, random bfloat16 weights; then the stages of one step by CUDA-event spans
     (eager launches), and the kernels alone, replayed from CUDA graphs, against their rooflines."""
+    return layers_workload("rumedra", (("rumedra", rumedra_config), ("lanirax", lanirax_config), ("llama", llama_config_like)),
+                           rumedra_kernel_rooflines, args, torch, np)
+
+
+def papulix_config(width: int, vocab: int = 32000) -> dict:
+    """Four Papulix layers at a real model's proportions over four residual streams.  Attention: heads of 64 in groups of
+    four with values as wide as keys.  Delta rule with a decay a channel: heads of 128 x 128, four taps, ranks of 128.
+    State space: twice the width in heads of 64 with 128 states, eight groups, four taps.  Gated units of 8/3 widths."""
+    H, R = width // 64, width // 128
+    attn = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 64, "scale": 0.125}
+    delta = {"heads": R, "kv_heads": R, "dim": 128, "vdim": 128, "conv": 4}
+    ssd = {"heads": 2 * H, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}
+    mlp = {"kind": "dense", "ff": width * 8 // 3 // 128 * 128}
+    return {"architecture": "Papulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 4.0},
+            "logit_scale": 0.5, "streams": 4,
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in
+                       (("attention", attn), ("channel_delta", delta), ("mamba2", ssd), ("channel_delta", delta))]}
+
+
+def papulix_kernel_rooflines(width: int, B: int, ctx: int, T: int, pk: dict, torch, np) -> dict:
+    """The kernels that Papulix adds or extends, alone, at the sizes of `papulix_config(width)`, each beside the like kernel
+    of the closest models: {name: {"us", "ideal_us", "frac"}}.  Ideal: bytes that must move over the measured copy
+    bandwidth (single tokens, norms, streams), FLOPs over the measured bfloat16 GEMM rate (attention and gated units over
+    prompts), or float32 FMAs over the FFMA rate of the SMs at their maximum clock (the recurrences over prompts, float32
+    by design)."""
+    from rust_llm_inference_server_b200 import ops
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    sms = torch.cuda.get_device_properties(0).multi_processor_count
+    ffma = sms * 128 * 2 * pk.get("sm_max_mhz", 1965.0) * 1e6
+    page, nh, nkv, hd = 16, width // 64, max(1, width // 256), 64
+    rh, rd, taps, S = width // 128, 128, 4, 4
+    mh, mg, mn, mv = width // 32, 8, 128, 64
+    bf, out = torch.bfloat16, {}
+    rnd = lambda *shape: torch.randn(*shape, device="cuda") * 0.3
+
+    def row(name, us, ideal_s):
+        out[name] = {"us": round(us, 1), "ideal_us": round(ideal_s * 1e6, 1), "frac": round(ideal_s * 1e6 / us, 3)}
+
+    for kind, reqs in (("decode", [(ctx - 1, 1)] * B), ("prefill", [(0, T)])):
+        st = _KernelStep(reqs, page, torch, np)
+        st.n_prefill_tokens = st.n_prefill_tokens if kind == "prefill" else 0
+        n = st.n_tokens
+        dec = kind == "decode"
+        keys = B * ctx if dec else T * (T + 1) // 2
+        # attention with one in the denominator and a gate a channel, beside the slope attention over all keys
+        kc, vc, q = rnd(st.n_pages, nkv, page, hd).to(bf), rnd(st.n_pages, nkv, page, hd).to(bf), rnd(n, nh * hd).to(bf)
+        gate, o, zeros = rnd(n, nh * hd + 8).to(bf)[:, :nh * hd], torch.empty_like(q), torch.zeros(nh, device="cuda")
+        slopes = torch.tensor([2.0 ** (-8.0 * (h + 1) / nh) for h in range(nh)], device="cuda")
+        attn = keys * nkv * hd * 2 * 2 / hbm if dec else 2 * nh * keys * 2 * hd / tf
+        us = _graph_time_us(lambda: ops.attention_biased(q, kc, vc, o, None, gate, st, 0, nh, nkv, hd, hd, page, 0.125, 0,
+                                                         sinks=zeros), torch)
+        row(f"sink_gate_attention_{kind}", us, attn)
+        us = _graph_time_us(lambda: ops.attention_biased(q, kc, vc, o, None, None, st, 0, nh, nkv, hd, hd, page, 0.125, 0,
+                                                         slopes=slopes), torch)
+        row(f"slope_attention_{kind}", us, attn)
+        # norms over the whole projections and the paged write, beside norms a head
+        N = (nh + 2 * nkv) * hd
+        proj, qw, kw = rnd(n, N).to(bf), torch.ones(nh * hd, device="cuda"), torch.ones(nkv * hd, device="cuda")
+        slots = torch.arange(n, device="cuda", dtype=torch.int32)
+        moved = n * (N * 2 + (nh + 2 * nkv) * hd * 2) / hbm
+        us = _graph_time_us(lambda: ops.qk_row_norm_store(proj, 0, nh * hd, (nh + nkv) * hd, qw, kw, 1e-5, q, kc, vc, slots, nh, nkv,
+                                                          hd, hd, page), torch)
+        row(f"row_norm_store_{kind}", us, moved)
+        us = _graph_time_us(lambda: ops.qk_norm_store(proj, 0, nh * hd, (nh + nkv) * hd, qw[:hd], kw[:hd], 1e-5, None, 0.0, q, kc, vc,
+                                                      slots, nh, nkv, hd, hd, page), torch)
+        row(f"head_norm_store_{kind}", us, moved)
+        # the recurrences: a decay a channel beside a decay a head, at the same heads; the state-space walk beside the decayed
+        # linear attention at the same heads
+        C = 3 * rh * rd
+        proj = rnd(n, C + 2 * rh + (-(2 * rh) % 8)).to(bf)
+        low = rnd(n, 2 * rh * rd).to(bf)
+        conv_w, a_log = rnd(C, taps).contiguous(), rnd(rh).contiguous()
+        dtb, dtb1 = rnd(rh * rd).contiguous(), rnd(rh).contiguous()
+        state = torch.zeros(len(reqs), ops.conv_recurrence_state_floats(rh, rh, rd, rd, taps), device="cuda")
+        o3 = torch.empty(n, rh * rd, device="cuda")
+        args = (state, o3, st, rh, rh, rd, rd, taps, 1e-6, rd ** -0.5)
+        ideal = B * rh * rd * rd * 4 * 2 / hbm if dec else 3 * 2 * T * rh * rd * rd / ffma
+        us = _graph_time_us(lambda: ops.channel_delta(proj, 0, C, low[:, :rh * rd], conv_w, a_log, dtb, *args), torch)
+        row(f"channel_delta_{kind}", us, ideal)
+        us = _graph_time_us(lambda: ops.gated_delta(proj, 0, C, C + rh, conv_w, a_log, dtb1, *args), torch)
+        row(f"gated_delta_{kind}", us, ideal)
+        inner = mh * mv
+        C = inner + 2 * mg * mn
+        proj = rnd(n, inner + C + mh + (-mh % 8)).to(bf)
+        conv_w, conv_b = rnd(C, taps).contiguous(), rnd(C).contiguous()
+        a_log, dtb, skip = rnd(mh).contiguous(), rnd(mh).contiguous(), rnd(mh).contiguous()
+        state = torch.zeros(len(reqs), ops.conv_recurrence_state_floats(mh, mg, mn, mv, taps), device="cuda")
+        y3 = torch.empty(n, inner, device="cuda")
+        ideal = B * mh * mn * mv * 4 * 2 / hbm if dec else 2 * 2 * T * mh * mn * mv / ffma
+        us = _graph_time_us(lambda: ops.state_space(proj, inner, inner + C, conv_w, conv_b, a_log, dtb, skip, state, y3, st, mh, mg,
+                                                    mn, mv, taps), torch)
+        row(f"state_space_{kind}", us, ideal)
+        proj2 = rnd(n, 2 * mh * mn + inner).to(bf)
+        state2, decay = torch.zeros(len(reqs), mh, mv, mn, device="cuda"), torch.full((mh,), 0.97, device="cuda")
+        us = _graph_time_us(lambda: ops.lightning_scan(proj2, 0, mh * mn, 2 * mh * mn, y3, state2, decay, st, mh, mn, mv), torch)
+        row(f"decayed_linear_attention_{kind}", us, ideal)
+        # the gate before a norm in parts, beside a norm a head before its gate
+        z, w, yb = proj[:, :inner], torch.ones(inner, device="cuda"), torch.empty(n, inner, dtype=bf, device="cuda")
+        moved = n * inner * (4 + 2 + 2) / hbm
+        row(f"gate_group_norm_{kind}", _graph_time_us(lambda: ops.gate_group_norm(y3, z, w, 1e-5, yb, mg), torch), moved)
+        row(f"head_norm_gate_{kind}", _graph_time_us(lambda: ops.head_norm_gate(y3, w[:mv], 1e-5, yb, mh, gate=z), torch), moved)
+        # the streams' update and norm, beside the residual addition and RMS norm of one stream
+        x, a, h = rnd(n, S, width).contiguous(), rnd(n, width).to(bf), torch.empty(n, width, dtype=bf, device="cuda")
+        mix, co, wv, bv = rnd(S, S).contiguous(), rnd(S).contiguous(), torch.ones(width, device="cuda"), torch.zeros(width, device="cuda")
+        norm = ops.StreamNorm("dynamic_tanh", wv, bv, 0.7)
+        us = _graph_time_us(lambda: ops.stream_mix(x, S, y=a, y_bias=bv, mix=mix, out_coef=co, x_out=x, in_coef=co, norm=norm, h=h), torch)
+        row(f"stream_mix_{kind}", us, n * width * (S * 8 + 4) / hbm)
+        resid = rnd(n, width).contiguous()
+        row(f"residual_rmsnorm_{kind}", _graph_time_us(lambda: ops.rmsnorm(resid, wv, 1e-5, h, a), torch), n * width * (8 + 4) / hbm)
+        # the gated unit with biases beside the plain one
+        I = width * 8 // 3 // 128 * 128
+        wgu = torch.stack([rnd(I // 4, 4, width), rnd(I // 4, 4, width)], dim=1).reshape(2 * I, width).to(bf).contiguous()
+        wdn, bgu = rnd(width, I).to(bf), rnd(2 * I).contiguous()
+
+        def unit(bias):
+            if n <= ops.STREAM_GEMM_ROWS:
+                return ops.linear(ops.stream_gemm(a, wgu, swiglu4=True, bias=bias), wdn)
+            return ops.linear(ops.gemm_tcgen05(a, wgu, "swiglu4") if bias is None else
+                              ops.gemm_tcgen05(a, wgu, "glu4", glu=(1.0, None, 0.0), bias=bias), wdn)
+        ideal = 3 * I * width * 2 / hbm if dec else 2.0 * n * 3 * I * width / tf
+        row(f"biased_gated_ff_{kind}", _graph_time_us(lambda: unit(bgu), torch), ideal)
+        row(f"silu_gated_ff_{kind}", _graph_time_us(lambda: unit(None), torch), ideal)
+        if dec:
+            # the last product with the streams' update and norm in its epilogue, beside the one with the residual addition
+            act = rnd(n, I).to(bf)
+            sink = ops.StreamsSink(x, x, S, mix, co, co, norm)
+            row("down_proj_streams_decode", _graph_time_us(lambda: ops.stream_gemm(act, wdn, sink=sink, bias=bv), torch), I * width * 2 / hbm)
+            rs = ops.ResidualSink(resid, wv, 1e-5)
+            row("down_proj_residual_decode", _graph_time_us(lambda: ops.stream_gemm(act, wdn, sink=rs), torch), I * width * 2 / hbm)
+    return out
+
+
+def workload_papulix(args, torch, np) -> dict:
+    """Prefill (one 2,048-token prompt) and decode (batch 8, context 4,096) of four Papulix layers at two widths beside
+    four Lanirax layers (the closest model: a gated delta rule and attention with a sink) and four Llama layers of the same
+    width, random bfloat16 weights; then the stages of one step by CUDA-event spans (eager launches), and the kernels
+    alone, replayed from CUDA graphs, against their rooflines."""
+    return layers_workload("papulix", (("papulix", papulix_config), ("lanirax", lanirax_config), ("llama", llama_config_like)),
+                           papulix_kernel_rooflines, args, torch, np)
+
+
+def layers_workload(head: str, models, rooflines, args, torch, np) -> dict:
+    """Prefill, decode and stages of four layers of every one of `models` (name, configuration by width) at two widths, and
+    the kernels of the first alone."""
     from rust_llm_inference_server_b200 import LLM
     from rust_llm_inference_server_b200.ops import profile
     pk, pk_src = peaks()
     B, ctx, page, T = args.batch, args.context, 16, PREFILL_TOKENS
     steps = min(args.steps, 64)
-    out = {"workload": "rumedra", "metric": "prefill and decode tokens/s of four layers, Rumedra beside Lanirax and Llama at equal width",
+    names = [n.capitalize() for n, _ in models]
+    out = {"workload": head, "metric": f"prefill and decode tokens/s of four layers, {names[0]} beside {' and '.join(names[1:])} at equal width",
            "unit": "tokens/s", "impl": "ours", "dtype": "bf16", "n_gpus": 1, "steps": steps, "warmup": args.warmup,
            "data": "synthetic: uniform-random token ids, random-init weights (device generator)",
            "config": {"global_batch": B, "seq_len": ctx, "prefill_tokens": T, "page_size": page, "layers": 4},
@@ -1023,8 +1168,8 @@ def workload_rumedra(args, torch, np) -> dict:
     clocks.start()
     for width in (1024, 2048):
         row = {}
-        for name, cfg in (("rumedra", rumedra_config(width)), ("lanirax", lanirax_config(width)), ("llama", llama_config_like(width))):
-            llm = LLM.from_random(cfg, 8, dtype="bfloat16", on_device=True, max_seq_len=ctx + page,
+        for name, cfg in models:
+            llm = LLM.from_random(cfg(width), 8, dtype="bfloat16", on_device=True, max_seq_len=ctx + page,
                                   num_blocks=B * (ctx + page) // page + 64, block_size=page, max_num_seqs=B,
                                   max_batched_tokens=max(2048, B), prefix_caching=False)
             pre = prefill_run(llm, T, 5, 3, torch, np)
@@ -1044,13 +1189,13 @@ def workload_rumedra(args, torch, np) -> dict:
                          "prefill_stage_us": pre_stages, "decode_stage_us": dec_stages}
             del llm
             torch.cuda.empty_cache()
-        row["rooflines"] = rumedra_kernel_rooflines(width, B, ctx, T, pk, torch, np)
+        row["rooflines"] = rooflines(width, B, ctx, T, pk, torch, np)
         out["sizes"][f"width{width}"] = row
     out["clocks"] = clocks.stop()
-    head = out["sizes"]["width2048"]["rumedra"]
-    out["value"] = head["decode_tokens_per_s"]
-    out["ms_per_step"] = head["decode_ms_per_step"]
-    out["gpu_launches"] = int(round(head["launches_per_decode_step"] * steps))
+    first = out["sizes"]["width2048"][head]
+    out["value"] = first["decode_tokens_per_s"]
+    out["ms_per_step"] = first["decode_ms_per_step"]
+    out["gpu_launches"] = int(round(first["launches_per_decode_step"] * steps))
     return out
 
 
@@ -1084,7 +1229,7 @@ def print_timeline(records: list) -> None:
 
 
 WORKLOADS = {"3b": workload_3b, "8b": workload_8b, "1b-fp32": workload_1b_fp32, "lasapel": workload_lasapel,
-             "gavodra": workload_gavodra, "lanirax": workload_lanirax, "rumedra": workload_rumedra}
+             "gavodra": workload_gavodra, "lanirax": workload_lanirax, "rumedra": workload_rumedra, "papulix": workload_papulix}
 
 
 def main() -> int:

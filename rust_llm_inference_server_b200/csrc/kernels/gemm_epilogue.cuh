@@ -7,11 +7,20 @@ namespace tc {
 
 // Parameters of the gated epilogue with clipping (EPI 3): g' sigmoid(slope g') (u' + shift) with g' = min(g,
 // limit) and u' = clamp(u, -limit, limit); limit +inf clips nothing; slope +inf: max(g', 0) (u' + shift).  bias (float32, one
-// a column, 16-byte aligned; null: none) is added to g and u first.
+// a column; null: none) is added to g and u first.
 struct GluParams {
     float slope, limit, shift;
     const float* bias;
 };
+
+// The bias of 32 columns, one a lane (requested before the sums are read), and its addition to every lane's row of sums.
+__device__ __forceinline__ float bias_of_lane(const GluParams& gp, int col, int lane, int N) {
+    return gp.bias != nullptr && col + lane < N ? gp.bias[col + lane] : 0.f;
+}
+__device__ __forceinline__ void add_bias32(uint32_t (&r)[32], float bias) {
+#pragma unroll
+    for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) + __shfl_sync(0xffffffffu, bias, i));
+}
 
 // EPI 0: bf16 y [M, N].  EPI 1: SwiGLU over a gate|up matrix whose rows are interleaved in blocks of
 // 4 (columns 8 t .. 8 t + 3 gate, 8 t + 4 .. 8 t + 7 up), y [M, N / 2] bf16.  EPI 2: float32 y [M, N].
@@ -36,19 +45,10 @@ __device__ __forceinline__ void store_sums32(const uint32_t (&r)[32], void* __re
         bf16* o = reinterpret_cast<bf16*>(y) + (size_t)row * (N >> 1) + (col >> 1);
         float res[16];
 #pragma unroll
-        for (int tt = 0; tt < 4; ++tt) {
-            float4 bg = make_float4(0.f, 0.f, 0.f, 0.f), bu = bg;
-            if (EPI == 3 && gp.bias != nullptr && col + tt * 8 < N) {
-                bg = *reinterpret_cast<const float4*>(gp.bias + col + tt * 8);
-                bu = *reinterpret_cast<const float4*>(gp.bias + col + tt * 8 + 4);
-            }
+        for (int tt = 0; tt < 4; ++tt)
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
-                float gt = __uint_as_float(r[tt * 8 + j]), up = __uint_as_float(r[tt * 8 + 4 + j]);
-                if (EPI == 3) {
-                    gt += j == 0 ? bg.x : j == 1 ? bg.y : j == 2 ? bg.z : bg.w;
-                    up += j == 0 ? bu.x : j == 1 ? bu.y : j == 2 ? bu.z : bu.w;
-                }
+                const float gt = __uint_as_float(r[tt * 8 + j]), up = __uint_as_float(r[tt * 8 + 4 + j]);
                 if (EPI == 1) {
                     res[tt * 4 + j] = gt / (1.0f + expf(-gt)) * up;
                 } else {
@@ -56,7 +56,6 @@ __device__ __forceinline__ void store_sums32(const uint32_t (&r)[32], void* __re
                     res[tt * 4 + j] = glu_gate(g, gp.slope) * (u + gp.shift);
                 }
             }
-        }
 #pragma unroll
         for (int v = 0; v < 2; ++v) {
             if (col + v * 16 >= N) break;

@@ -157,9 +157,11 @@ __global__ __launch_bounds__(GT_THREADS) void gemm_tcgen05_kernel(const __grid_c
             const int row = m0 + q * 32 + lane;
             const uint32_t tmem_acc = tmem_base + (uint32_t)(buf * BN) + ((uint32_t)(q * 32) << 16);
             for (int cb = 0; cb < BN / 32; ++cb) {
+                const int col = n0 + cb * 32;
+                const float bias = EPI == 3 ? bias_of_lane(gp, col, lane, N) : 0.f;
                 uint32_t r[32];
                 tmem_ld32(tmem_acc + (uint32_t)(cb * 32), r);
-                const int col = n0 + cb * 32;
+                if (EPI == 3 && gp.bias != nullptr) add_bias32(r, bias);
                 if (!ok || row >= M || col >= N) continue;
                 store_sums32<EPI>(r, y, row, col, N, gp);
             }
@@ -273,9 +275,8 @@ extern "C" int rlis_gemm_tcgen05(const void* x, const void* W, void* y, int M, i
 
 // The gate|up product with the clipped gating in its epilogue: W's rows interleaved gate/up in blocks of 4,
 // y [M, N / 2] bf16 = g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).  bias float32
-// [N] in the order of W's rows, 16-byte aligned (null: none): added to g and u first.
+// [N] in the order of W's rows (null: none): added to g and u first.
 extern "C" int rlis_gemm_tcgen05_glu(const void* x, const void* W, void* y, int M, int N, int K, float slope,
                                      float limit, float shift, const float* bias, cudaStream_t stream) {
-    if ((reinterpret_cast<uintptr_t>(bias) & 15) != 0) return RLIS_ERR_UNSUPPORTED;
     return gemm_tcgen05_impl(x, W, y, M, N, K, 3, GluParams{slope, limit, shift, bias}, stream);
 }

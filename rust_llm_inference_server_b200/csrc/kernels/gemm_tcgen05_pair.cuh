@@ -192,9 +192,11 @@ __global__ __launch_bounds__(GP_THREADS) void gemm_tcgen05_pair_kernel(const __g
             const int row = m0 + q * 32 + lane;
             const uint32_t tmem_acc = tmem_base + (uint32_t)(buf * PN) + ((uint32_t)(q * 32) << 16);
             for (int cb = 0; cb < PN / 32; ++cb) {
+                const int col = n0 + cb * 32;
+                const float bias = EPI == 3 ? bias_of_lane(gp, col, lane, N) : 0.f;
                 uint32_t r[32];
                 tmem_ld32(tmem_acc + (uint32_t)(cb * 32), r);
-                const int col = n0 + cb * 32;
+                if (EPI == 3 && gp.bias != nullptr) add_bias32(r, bias);
                 if (!ok || row >= M || col >= N) continue;
                 store_sums32<EPI>(r, y, row, col, N, gp);
             }

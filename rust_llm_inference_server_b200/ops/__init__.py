@@ -915,13 +915,13 @@ def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = Fa
         x = scaled.x
     M, K = x.shape
     N = w.shape[0]
+    if M > STREAM_MAX_ROWS or K % 8 or (swiglu4 and N % 8):
+        raise KernelError(f"stream_gemm: takes up to {STREAM_MAX_ROWS} rows and K a multiple of 8, got M={M}, K={K}")
     ldx = _stream_rows(x, "stream_gemm")
     _req(w, "w", torch.bfloat16, (N, K))
     if bias is not None:
         _req(bias, "bias", torch.float32, (N,))
     bp = bias.data_ptr() if bias is not None else None
-    if M > STREAM_MAX_ROWS or K % 8 or (swiglu4 and N % 8):
-        raise KernelError(f"stream_gemm: takes up to {STREAM_MAX_ROWS} rows and K a multiple of 8, got M={M}, K={K}")
     if sink is not None and (scaled is not None or swiglu4 or M > DECODE_GEMM_ROWS):
         raise KernelError(f"stream_gemm: a sink takes a plain product of up to {DECODE_GEMM_ROWS} unscaled rows")
     if sink is None:

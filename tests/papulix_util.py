@@ -83,7 +83,7 @@ CONFIGS = {
         mamba2(12, 64, 128, 1, 3, 4),
     ], (1, 2, 2)),
 }
-SEEDS = {"A": 3, "B": 5, "C": 8, "D": 13, "E": 21, "F": 34}
+SEEDS = {"A": 3, "B": 5, "C": 8, "D": 15, "E": 21, "F": 34}
 RANKS = {"A": (12, 16), "B": (1, 3), "C": (16, 8), "D": (5, 11), "E": (32, 24), "F": (24, 40)}
 
 
@@ -149,7 +149,7 @@ def draw_weights(cfg: dict, seed: int, ranks=(8, 8)) -> dict:
         elif last == "D":
             x = 0.7 + 0.3 * z
         elif last == "alpha":
-            x = rng.uniform(0.4, 0.9, shape)
+            x = rng.uniform(0.4, 0.9, shape) / cfg["streams"]      # some entries saturate, most do not
         elif last == "conv":
             x = 0.3 + 0.6 * z
         elif last == "mix" and len(shape) == 2 and "hc" in name:
@@ -161,9 +161,7 @@ def draw_weights(cfg: dict, seed: int, ranks=(8, 8)) -> dict:
         elif last == "b" and len(shape) == 1:
             x = 0.4 * z                                    # biases of norms, projections and convolutions
         elif len(shape) == 2:
-            x = z * (1.0 if last == "embed" else 1.3) / np.sqrt(shape[1] if last != "embed" else 1)
-            if last == "embed":
-                x = z * 0.7
+            x = z * 0.7 if last == "embed" else z / np.sqrt(shape[1])
         else:
             x = 1.0 + 0.2 * z                              # norm weights
         out[name] = torch.from_numpy(np.asarray(x, dtype=np.float32).reshape(shape)).to(torch.bfloat16)

