@@ -1,7 +1,7 @@
 // Residual streams side by side (hyper-connections), and norms without statistics.  One pass over a token's row joins a
 // sublayer's result to the streams and makes the input of the sublayer that follows:
 //
-//   x_t <- sum_s mix[s, t] x_s + out[t] (y + y_bias)     all S streams at once from the old ones (only when y is given)
+//   x_t <- sum_s mix[s, t] x_s + out[t] (y + y_bias)     with the old x_s on the right (only when y is given)
 //   u    = sum_t in[t] x_t                               (in null: the plain sum)
 //   h    = norm(u)                                       rounded once to the activation type
 //
@@ -151,7 +151,7 @@ __global__ __launch_bounds__(THREADS) void stream_mix_kernel(
     }
 }
 
-// out[t, part] = g / sqrt(mean over the part of g^2 + eps) * w with g = x silu(z): the gate comes before the norm, each of
+// out[t, part] = g / sqrt(mean over the part of g^2 + eps) * w with g = x silu(z): first gated, then normed, each of
 // gridDim.y equal parts of a row has a root mean square of its own.  One CTA a (token, part).
 template <typename T, int VN>
 __global__ __launch_bounds__(THREADS) void gate_group_norm_kernel(

@@ -513,8 +513,8 @@ def stream_mix(x: torch.Tensor, n_streams: int, y: torch.Tensor | None = None, y
                mix: torch.Tensor | None = None, out_coef: torch.Tensor | None = None, x_out: torch.Tensor | None = None,
                in_coef: torch.Tensor | None = None, norm: StreamNorm | None = None, h: torch.Tensor | None = None,
                u_out: torch.Tensor | None = None, rows: torch.Tensor | None = None):
-    """Residual streams side by side: with y, x_t <- sum_s mix[s, t] x_s + out_coef[t] (y + y_bias), all streams at once
-    from the old ones, into `x_out` (float32 [T, S, W]; None: not kept); then u = sum_t in_coef[t] x_t, h = norm(u) in h's
+    """Residual streams side by side: with y, x_t <- sum_s mix[s, t] x_s + out_coef[t] (y + y_bias), old streams on
+    the right, into `x_out` (float32 [T, S, W]; None: not kept); then u = sum_t in_coef[t] x_t, h = norm(u) in h's
     type and u_out = u in float32 (each only where given).  x float32 [T, S, W], or [T, W]: one row is every stream.  mix
     float32 [S, S] (from, to; None: the streams stay themselves), out_coef and in_coef float32 [S] (None: ones).  `rows`
     (int32 [R]): h and u_out are made for these rows, and the streams stay as they are."""

@@ -229,7 +229,7 @@ class PostNormBlock:
 
 class HyperBlock:
     """Pre-norm sublayers over S residual streams (hyper-connections).  A sublayer reads norm(sum_s read[s] x_s); its
-    result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, all streams at once.  The streams are float32: one
+    result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, old streams on the right.  The streams are float32: one
     kernel updates them with a sublayer's result and makes the normed input of the sublayer that follows, also when that
     is the first sublayer of the next block of this kind (a block returns `Streams` with that update pending).  The
     streams start equal, so the first kernel reads the embedding's row as every stream.  In steps of a few rows, where

@@ -26,7 +26,7 @@ class RMSNormSpec:
 
 @dataclass(frozen=True)
 class DynamicTanhSpec:
-    """y = tanh(alpha x) * w + b: a norm that computes no mean or variance.  `alpha` names a scalar tensor, `weight` and
+    """y = tanh(alpha x) * w + b: a norm without statistics of the row.  `alpha` names a scalar tensor, `weight` and
     `bias` vectors of shape (dim,)."""
     dim: int
     weight: str
@@ -437,7 +437,7 @@ class LMHeadSpec:
 @dataclass(frozen=True)
 class HyperSpec:
     """The coefficients of one sublayer's hyper-connection over S residual streams: the sublayer reads u = sum_s read[s]
-    x_s and its result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, all streams at once."""
+    x_s and its result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, old streams on the right."""
     streams: int
     read: str                        # (streams,)
     write: str                       # (streams,)

@@ -71,7 +71,7 @@ def stream_input(streams, coef):
 
 
 def stream_update(streams, mix, out, y):
-    """x_t <- sum_s mix[s, t] x_s + out[t] y, all at once (mix is indexed [from, to])."""
+    """x_t <- sum_s mix[s, t] x_s + out[t] y, with the old x_s on the right (rows of mix are sources, columns targets)."""
     return np.einsum("st,sjw->tjw", mix, streams) + out[:, None, None] * y[None]
 
 

@@ -142,7 +142,7 @@ def test_plain_mechanisms_against_closed_forms():
     assert np.allclose(P.softmax_plus_one(np.array([-800.0, 800.0])), [0.0, 1.0])
     p = P.softmax_plus_one(np.array([0.3, -1.0]))
     assert np.allclose(p, np.exp([0.3, -1.0]) / (1 + np.exp([0.3, -1.0]).sum()))
-    # streams: all at once from the old ones, the matrix indexed [from, to]
+    # streams: every new one from the old ones; rows of the matrix are sources, columns targets
     st = rng.standard_normal((2, 1, 3))
     mix, out, y = np.array([[0.5, 2.0], [3.0, 0.1]]), np.array([1.0, -1.0]), rng.standard_normal((1, 3))
     new = P.stream_update(st, mix, out, y)
