@@ -85,9 +85,12 @@ __device__ __forceinline__ float rope_second(float a, float b, float c, float s)
     return __fmaf_rn(b, c, __fmul_rn(a, s));
 }
 
-// The gate of a gated unit: g sigmoid(slope g); slope 1 is silu, slope +inf its limit max(g, 0).
-__device__ __forceinline__ float glu_gate(float g, float slope) {
-    return slope == __int_as_float(0x7f800000) ? fmaxf(g, 0.f) : g / (1.0f + expf(-slope * g));
+// The gate of a gated unit: g sigmoid(slope (g + cubic g^3)).  Slope 1 is silu, slope +inf its limit max(g, 0); slope
+// 2 sqrt(2 / pi) with cubic 0.044715 is the tanh form of gelu (0.5 (1 + tanh(u)) is sigmoid(2 u)).
+__device__ __forceinline__ float glu_gate(float g, float slope, float cubic = 0.f) {
+    if (slope == __int_as_float(0x7f800000)) return fmaxf(g, 0.f);
+    const float z = cubic != 0.f ? fmaf(cubic * g * g, g, g) : g;
+    return g / (1.0f + expf(-slope * z));
 }
 
 #define RLIS_LAUNCH_CHECK() ((int)cudaGetLastError())

@@ -6,11 +6,13 @@
 namespace tc {
 
 // Parameters of the gated epilogue with clipping (EPI 3): g' sigmoid(slope g') (u' + shift) with g' = min(g,
-// limit) and u' = clamp(u, -limit, limit); limit +inf clips nothing; slope +inf: max(g', 0) (u' + shift).  bias (float32, one
+// limit) and u' = clamp(u, -limit, limit); limit +inf clips nothing; slope +inf: max(g', 0) (u' + shift); the gate's
+// argument is g' + cubic g'^3.  bias (float32, one
 // a column; null: none) is added to g and u first.
 struct GluParams {
     float slope, limit, shift;
     const float* bias;
+    float cubic;
 };
 
 // The bias of 32 columns, one a lane (requested before the sums are read), and its addition to every lane's row of sums.
@@ -53,7 +55,7 @@ __device__ __forceinline__ void store_sums32(const uint32_t (&r)[32], void* __re
                     res[tt * 4 + j] = gt / (1.0f + expf(-gt)) * up;
                 } else {
                     const float g = fminf(gt, gp.limit), u = fminf(fmaxf(up, -gp.limit), gp.limit);
-                    res[tt * 4 + j] = glu_gate(g, gp.slope) * (u + gp.shift);
+                    res[tt * 4 + j] = glu_gate(g, gp.slope, gp.cubic) * (u + gp.shift);
                 }
             }
 #pragma unroll

@@ -254,7 +254,7 @@ extern "C" int rlis_gemm_tcgen05_grouped(const void* x, const void* W, void* y, 
     int dev = 0, sms = 148;
     if (cudaGetDevice(&dev) == cudaSuccess) cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     const unsigned grid = (unsigned)(num_tiles < sms ? num_tiles : sms);
-    const GluParams gp{slope, limit, shift, nullptr};
+    const GluParams gp{slope, limit, shift, nullptr, 0.0f};
     if (epilogue == 0)
         rlis_launch(gemm_tcgen05_kernel<0>, grid, GT_THREADS, GT_SMEM, stream, map_x, map_w, y, M, N, K, m_tiles, num_tiles, gp,
                     tile_expert, N);
@@ -270,13 +270,13 @@ extern "C" int rlis_gemm_tcgen05_grouped(const void* x, const void* W, void* y, 
 extern "C" int rlis_gemm_tcgen05(const void* x, const void* W, void* y, int M, int N, int K, int epilogue,
                                  cudaStream_t stream) {
     if (epilogue < 0 || epilogue > 2) return RLIS_ERR_UNSUPPORTED;
-    return gemm_tcgen05_impl(x, W, y, M, N, K, epilogue, GluParams{1.0f, INFINITY, 0.0f, nullptr}, stream);
+    return gemm_tcgen05_impl(x, W, y, M, N, K, epilogue, GluParams{1.0f, INFINITY, 0.0f, nullptr, 0.0f}, stream);
 }
 
 // The gate|up product with the clipped gating in its epilogue: W's rows interleaved gate/up in blocks of 4,
-// y [M, N / 2] bf16 = g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).  bias float32
+// y [M, N / 2] bf16 = g' sigmoid(slope (g' + cubic g'^3)) (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).  bias float32
 // [N] in the order of W's rows (null: none): added to g and u first.
 extern "C" int rlis_gemm_tcgen05_glu(const void* x, const void* W, void* y, int M, int N, int K, float slope,
-                                     float limit, float shift, const float* bias, cudaStream_t stream) {
-    return gemm_tcgen05_impl(x, W, y, M, N, K, 3, GluParams{slope, limit, shift, bias}, stream);
+                                     float limit, float shift, float cubic, const float* bias, cudaStream_t stream) {
+    return gemm_tcgen05_impl(x, W, y, M, N, K, 3, GluParams{slope, limit, shift, bias, cubic}, stream);
 }

@@ -361,7 +361,7 @@ __global__ __launch_bounds__(256) void moe_combine_kernel(
 // columns followed by their B columns of the linear branch (the layout the products' gated epilogues want).
 template <typename T>
 __global__ void glu_act_kernel(const T* __restrict__ gu, T* __restrict__ out, int inter, size_t total,
-                               float slope, float limit, float shift, int interleave, const float* __restrict__ bias) {
+                               float slope, float limit, float shift, float cubic, int interleave, const float* __restrict__ bias) {
     pdl_wait_and_trigger();
     const size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= total) return;
@@ -371,7 +371,7 @@ __global__ void glu_act_kernel(const T* __restrict__ gu, T* __restrict__ out, in
     const size_t ui = interleave > 0 ? gi + interleave : (size_t)inter + i;
     const float g = fminf(to_f<T>(gu[t * 2 * inter + gi]) + (bias != nullptr ? bias[gi] : 0.f), limit);
     const float u = fminf(fmaxf(to_f<T>(gu[t * 2 * inter + ui]) + (bias != nullptr ? bias[ui] : 0.f), -limit), limit);
-    out[idx] = from_f<T>(glu_gate(g, slope) * (u + shift));
+    out[idx] = from_f<T>(glu_gate(g, slope, cubic) * (u + shift));
 }
 }  // namespace
 
@@ -488,15 +488,15 @@ extern "C" int rlis_moe_combine(const float* y, const int* pair_slot, const floa
 // out[t, i] = glu(gate column i, linear column i of gu[t, :]); limit +inf: no clipping.
 // bias float32 [2 inter] in the order of gu's columns, or null.
 extern "C" int rlis_glu_act(const void* gu, void* out, int n_tokens, int inter, float slope, float limit, float shift,
-                            int interleave, const float* bias, int dtype, cudaStream_t stream) {
+                            float cubic, int interleave, const float* bias, int dtype, cudaStream_t stream) {
     const size_t total = (size_t)n_tokens * inter;
     if (total == 0) return 0;
     if (interleave < 0 || (interleave > 0 && inter % interleave != 0)) return RLIS_ERR_UNSUPPORTED;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == RLIS_F32)
-        rlis_launch(glu_act_kernel<float>, blocks, 256, 0, stream, (const float*)gu, (float*)out, inter, total, slope, limit, shift, interleave, bias);
+        rlis_launch(glu_act_kernel<float>, blocks, 256, 0, stream, (const float*)gu, (float*)out, inter, total, slope, limit, shift, cubic, interleave, bias);
     else if (dtype == RLIS_BF16)
-        rlis_launch(glu_act_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)gu, (bf16*)out, inter, total, slope, limit, shift, interleave, bias);
+        rlis_launch(glu_act_kernel<bf16>, blocks, 256, 0, stream, (const bf16*)gu, (bf16*)out, inter, total, slope, limit, shift, cubic, interleave, bias);
     else
         return RLIS_ERR_UNSUPPORTED;
     return RLIS_LAUNCH_CHECK();

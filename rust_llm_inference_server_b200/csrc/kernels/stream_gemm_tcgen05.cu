@@ -70,6 +70,17 @@
 //     streams in place, x_t <- sum_s mix[s, t] x_s + out[t] y, weighs them, u = sum_t in[t] x_t, and writes h = bf16(tanh(
 //     alpha u) w + b), the rows of the product that follows: no partial sums, no scale left to apply, no norm kernel.
 //
+// A layer norm is taken apart in the same way: the sink leaves the sums of resid beside those of resid^2, and the product
+// after it, whose rows are bf16(resid * norm weight) with the mean still in them, takes the mean's share off: with u[f] =
+// sum_k W[f, k] norm_weight[k], known once the weights are, its result is (sum - mean u[f]) / sqrt(variance + eps).
+//
+// Sublayers that stand side by side on one normed input need two more things, so that a block of theirs is two products
+// around its mixer and no norm:
+//   * "mixed" (the first product): the first n_plain features of a stacked matrix are stored as they are, the rest is a
+//     gate|up matrix and is gated; the two results go to two places;
+//   * a second source: y = x W^T + x2 W2^T.  The blocks of k of the second pair follow those of the first, so the split of k,
+//     the ring and the sums are those of one product over K + K2.
+//
 // Every mbarrier wait is bounded (a fifth of a second); a wait that runs out sets an error word
 // (rlis_stream_gemm_error), every role runs to its end without further waits, and the CTA frees
 // its tensor memory before it returns.
@@ -94,7 +105,7 @@ constexpr int MAX_SPLITS = 16;          // the largest cluster (above 8 is opt-i
 constexpr int MAX_STREAMS = 8;          // streams epilogue
 
 template <int NT> constexpr size_t stream_smem_bytes(int n_stages = stages_of<NT>()) {
-    return (size_t)n_stages * (W_STAGE_BYTES + NT * SK * 2) + 1024 /* alignment */ + 1152 /* SCtrl */;
+    return (size_t)n_stages * (W_STAGE_BYTES + NT * SK * 2) + 1024 /* alignment */ + 1664 /* SCtrl */;
 }
 
 // A timeline for measurements, compiled in only with -DRLIS_TIMELINE (the build adds it when the
@@ -124,9 +135,10 @@ struct SCtrl {
     uint64_t red_full;      // the partial sums of the tokens this CTA finishes have arrived from the cluster
     uint32_t tmem_base;
     int abort;
-    float red[4];           // sink epilogue: the warps' sums of squares
+    float red[8];           // sink epilogue: the warps' sums of squares, and their sums
     float coef[MAX_STREAMS * MAX_STREAMS + 2 * MAX_STREAMS];   // streams epilogue: mix, out, in
     float rstd[128];        // scaled rows: the norm's scale of every token
+    float mean[128];        // ... and its mean, for a layer norm (else 0)
 };
 
 // What the two norm epilogues need (all null / 0 when unused).
@@ -135,11 +147,19 @@ struct NormFuse {
     int n_partials;
     int dim;                    // the norm's width
     float eps;
-    float* resid;               // sink: [M, N] float32, updated in place
+    const float* in_sums;       // [n_partials, M]: the rows' sums, for a layer norm (null: an RMS norm)
+    const float* colsum;        // [N]: sum_k W[f, k] norm weight[k], with in_sums
+    float* resid;               // sink: [M, N] float32, written
+    const float* resid_in;      // sink: what the result is added to (resid itself: in place; null: nothing)
+    float* out_sums;            // sink: [tiles, M] sums of the new rows, or null
+    int exact;                  // sink: the result joins unrounded
     const float* norm_w;        // sink: [N] weight of the norm that follows
     bf16* xn;                   // sink: [M, N] = bf16(resid * norm_w)
     float* out_partials;        // sink: [tiles, M]
-    float gate_slope;           // gated epilogue: g sigmoid(slope g) * u (1: silu; +inf: max(g, 0))
+    float gate_slope;           // gated epilogue: g sigmoid(slope (g + cubic g^3)) * u (1, 0: silu; +inf: max(g, 0))
+    float gate_cubic;
+    int n_plain;                // mixed epilogue: features below it are stored in y [M, n_plain], the others gated into y2
+    bf16* y2;
     const float* bias;          // [N] added to the sums, or null
     // streams (epilogue 3): what x_s are read from (row stride, stream stride; 0: one row is every stream) and written to
     // ([M, S, N]), their coefficients, and the dynamic tanh that follows (norm_w its weight, xn its result)
@@ -176,12 +196,22 @@ constexpr int CHUNK_F = 8;                   // features of a chunk
 constexpr int N_CHUNKS = SF / CHUNK_F;       // 16 chunks a tile
 
 template <int EPI, typename OutT>
-__device__ __forceinline__ void store_token(OutT* __restrict__ y, float v, int t, int f, int lane, int N, float slope) {
+__device__ __forceinline__ void store_token(OutT* __restrict__ y, float v, int t, int f, int lane, int N, const NormFuse& nf) {
     if (EPI == 1) {
         // lanes 8i..8i+3 hold gate, 8i+4..8i+7 the matching up values
         const float other = __shfl_xor_sync(0xffffffffu, v, 4);
         if ((lane & 4) == 0 && f + 4 < N)
-            y[(size_t)t * (N >> 1) + ((f >> 3) << 2) + (f & 3)] = from_f<OutT>(glu_gate(v, slope) * other);
+            y[(size_t)t * (N >> 1) + ((f >> 3) << 2) + (f & 3)] = from_f<OutT>(glu_gate(v, nf.gate_slope, nf.gate_cubic) * other);
+    } else if (EPI == 4) {
+        // (n_plain is a multiple of 8: a group of eight lanes is on one side of it)
+        const float other = __shfl_xor_sync(0xffffffffu, v, 4);
+        if (f < nf.n_plain) {
+            y[(size_t)t * nf.n_plain + f] = from_f<OutT>(v);
+        } else if ((lane & 4) == 0 && f + 4 < N) {
+            const int i = f - nf.n_plain;
+            nf.y2[(size_t)t * ((N - nf.n_plain) >> 1) + ((i >> 3) << 2) + (i & 3)] =
+                __float2bfloat16_rn(glu_gate(v, nf.gate_slope, nf.gate_cubic) * other);
+        }
     } else if (f < N) {
         y[(size_t)t * N + f] = from_f<OutT>(v);
     }
@@ -194,14 +224,21 @@ __device__ __forceinline__ void sink_token(const NormFuse& nf, float* red, float
                                            int N, bool live, float r_old, float w, float bias) {
     float r = 0.f;
     if (live && f < N) {
-        r = r_old + (__bfloat162float(__float2bfloat16_rn(v)) + bias);
+        r = r_old + ((nf.exact ? v : __bfloat162float(__float2bfloat16_rn(v))) + bias);
         nf.resid[(size_t)t * N + f] = r;
         nf.xn[(size_t)t * N + f] = __float2bfloat16_rn(r * w);
     }
     const float s = warp_sum(r * r);
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = s;
+    if (nf.out_sums != nullptr) {
+        const float s1 = warp_sum(r);
+        if ((threadIdx.x & 31) == 0) red[4 + (threadIdx.x >> 5)] = s1;
+    }
     __syncthreads();
-    if (threadIdx.x == 0 && live) nf.out_partials[(size_t)tile * M + t] = (red[0] + red[1]) + (red[2] + red[3]);
+    if (threadIdx.x == 0 && live) {
+        nf.out_partials[(size_t)tile * M + t] = (red[0] + red[1]) + (red[2] + red[3]);
+        if (nf.out_sums != nullptr) nf.out_sums[(size_t)tile * M + t] = (red[4] + red[5]) + (red[6] + red[7]);
+    }
     __syncthreads();
 }
 
@@ -232,7 +269,9 @@ __device__ __forceinline__ void streams_token(const NormFuse& nf, const float* c
 template <int NT, int EPI, typename OutT>
 __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_constant__ CUtensorMap map_w,
                                                                 const __grid_constant__ CUtensorMap map_x,
-                                                                OutT* __restrict__ y, int M, int N, int K,
+                                                                const __grid_constant__ CUtensorMap map_w2,
+                                                                const __grid_constant__ CUtensorMap map_x2,
+                                                                OutT* __restrict__ y, int M, int N, int K, int K2,
                                                                 int kb_per_split, int n_stages, const NormFuse nf) {
     extern __shared__ unsigned char sg_smem_raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(sg_smem_raw) + 1023) & ~(uintptr_t)1023);
@@ -265,7 +304,8 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int tile = blockIdx.x, split = blockIdx.y, splits = gridDim.y;
     const int n0 = tile * SF;
-    const int k_blocks = (K + SK - 1) / SK;
+    const int kb_first = (K + SK - 1) / SK;                 // blocks of k of the first pair; the second pair's follow
+    const int k_blocks = kb_first + (K2 + SK - 1) / SK;
     const int kb0 = split * kb_per_split;
     const int kb1 = min(kb0 + kb_per_split, k_blocks);
     const bool has_work = kb0 < kb1;                        // a split past the end of k adds zeros
@@ -301,19 +341,26 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
         // stream is resolved (programmatic dependent launch); x and y wait for it.
         const int n_kb = kb1 - kb0;
         const int early = n_kb < STG ? n_kb : STG;
+        auto load_w = [&](int s, int kb) {
+            tma_load_2d(w_tiles + (size_t)s * W_STAGE_BYTES, kb < kb_first ? &map_w : &map_w2, (kb < kb_first ? kb : kb - kb_first) * SK,
+                        n0, &ctrl->full[s]);
+        };
+        auto load_x = [&](int s, int kb) {
+            tma_load_2d(x_tiles + (size_t)s * X_STAGE_BYTES, kb < kb_first ? &map_x : &map_x2, (kb < kb_first ? kb : kb - kb_first) * SK,
+                        0, &ctrl->full[s]);
+        };
         for (int it = 0; it < early; ++it) {
             bar_expect_tx(&ctrl->full[it], W_STAGE_BYTES + X_STAGE_BYTES);
-            tma_load_2d(w_tiles + (size_t)it * W_STAGE_BYTES, &map_w, (kb0 + it) * SK, n0, &ctrl->full[it]);
+            load_w(it, kb0 + it);
         }
         pdl_wait();
-        for (int it = 0; it < early; ++it)
-            tma_load_2d(x_tiles + (size_t)it * X_STAGE_BYTES, &map_x, (kb0 + it) * SK, 0, &ctrl->full[it]);
+        for (int it = 0; it < early; ++it) load_x(it, kb0 + it);
         for (int it = early; it < n_kb; ++it) {
             const int s = it % STG, kb = kb0 + it;
             if (!bar_wait(&ctrl->empty[s], ((it / STG) - 1) & 1, &ctrl->abort)) break;
             bar_expect_tx(&ctrl->full[s], W_STAGE_BYTES + X_STAGE_BYTES);
-            tma_load_2d(w_tiles + (size_t)s * W_STAGE_BYTES, &map_w, kb * SK, n0, &ctrl->full[s]);
-            tma_load_2d(x_tiles + (size_t)s * X_STAGE_BYTES, &map_x, kb * SK, 0, &ctrl->full[s]);
+            load_w(s, kb);
+            load_x(s, kb);
         }
         pdl_trigger();     // everything this CTA reads is requested: the next kernel may start its own requests
     } else if (warp == 1 && lane == 0) {
@@ -337,18 +384,29 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
 #ifdef RLIS_TIMELINE
     if (tl_on) g_timeline[tl_slot][8] = *reinterpret_cast<volatile unsigned long long*>(&g_timeline_last_end);
 #endif
-    const bool scaled = EPI < 2 && nf.in_partials != nullptr;
+    const bool scaled = (EPI < 2 || EPI == 4) && nf.in_partials != nullptr;
     if (scaled && (int)threadIdx.x < M) {
         // this token's scale: the partial sums in the order of the tiles (RMSNorm: 1 / sqrt(mean + eps))
         float ss = 0.f;
         for (int p = 0; p < nf.n_partials; ++p) ss += nf.in_partials[(size_t)p * M + threadIdx.x];
-        ctrl->rstd[threadIdx.x] = 1.0f / sqrtf(ss / (float)nf.dim + nf.eps);
+        float mean = 0.f, var = ss / (float)nf.dim;
+        if (nf.in_sums != nullptr) {
+            float s1 = 0.f;
+            for (int p = 0; p < nf.n_partials; ++p) s1 += nf.in_sums[(size_t)p * M + threadIdx.x];
+            mean = s1 / (float)nf.dim;
+            var = fmaxf(fmaf(-mean, mean, var), 0.f);
+        }
+        ctrl->mean[threadIdx.x] = mean;
+        ctrl->rstd[threadIdx.x] = 1.0f / sqrtf(var + nf.eps);
     }
     // sink: what the first token this thread finishes needs from memory, requested before the sums arrive
     const int f = n0 + warp * 32 + lane;
     float sink_w = 0.f, sink_r0 = 0.f, st_b = 0.f;
     float st_x[EPI == 3 ? MAX_STREAMS : 1];
     const float bias = nf.bias != nullptr && f < N ? nf.bias[f] : 0.f;
+    const float colsum = scaled && nf.in_sums != nullptr && f < N ? nf.colsum[f] : 0.f;
+    // the norm's scale (and mean) of token t applied to a sum of feature f, whose column sum is cs
+    auto normed = [&](float v, int t, float cs) { return scaled ? fmaf(-ctrl->mean[t], cs, v) * ctrl->rstd[t] : v; };
     if constexpr (EPI == 3) {
         if (threadIdx.x < MAX_STREAMS * MAX_STREAMS) {
             const int s = threadIdx.x / MAX_STREAMS, to = threadIdx.x % MAX_STREAMS, S = nf.n_streams;
@@ -368,7 +426,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
     if (EPI == 2 && f < N) {
         sink_w = nf.norm_w[f];
         const int t0 = splits == 1 ? 0 : split;
-        if (t0 < M) sink_r0 = nf.resid[(size_t)t0 * N + f];
+        if (t0 < M && nf.resid_in != nullptr) sink_r0 = nf.resid_in[(size_t)t0 * N + f];
     }
     const bool waited = has_work ? bar_wait(&ctrl->acc_full, 0, &ctrl->abort) : true;
     const bool ok = __syncthreads_and(waited ? 1 : 0) != 0;       // the same for all threads
@@ -388,7 +446,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                 for (int j = 0; j < 16; ++j) {
                     const int t = c * 16 + j;
                     if (t >= M) continue;           // the same for all threads
-                    const float r_old = t == 0 ? sink_r0 : (ok && f < N ? nf.resid[(size_t)t * N + f] : 0.f);
+                    const float r_old = t == 0 ? sink_r0 : (ok && f < N && nf.resid_in != nullptr ? nf.resid_in[(size_t)t * N + f] : 0.f);
                     sink_token(nf, ctrl->red, __uint_as_float(r[j]), t, f, tile, M, N, ok, r_old, sink_w, bias);
                 }
                 continue;
@@ -406,8 +464,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
 #pragma unroll
                 for (int j = 0; j < 16; ++j)
                     if (c * 16 + j < M)
-                        store_token<EPI, OutT>(y, __uint_as_float(r[j]) * (scaled ? ctrl->rstd[c * 16 + j] : 1.0f) + bias,
-                                               c * 16 + j, f, lane, N, nf.gate_slope);
+                        store_token<EPI, OutT>(y, normed(__uint_as_float(r[j]), c * 16 + j, colsum) + bias, c * 16 + j, f, lane, N, nf);
             }
         }
     } else {
@@ -449,20 +506,21 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
             for (int c2 = split, slot = 0; c2 < N_CHUNKS; c2 += splits, ++slot) {
                 const int fo = n0 + c2 * CHUNK_F + fi;
                 const float fbias = nf.bias != nullptr && fo < N ? nf.bias[fo] : 0.f;
+                const float fsum = scaled && nf.in_sums != nullptr && fo < N ? nf.colsum[fo] : 0.f;
 #pragma unroll 1
                 for (int t = tg; t < ((M + 15) & ~15); t += S_THREADS / CHUNK_F) {
                     const float* src = part + (slot * splits) * (CHUNK_F * NT) + (t / 4) * (CHUNK_F * 4) + fi * 4 + (t & 3);
                     float v = 0.f;
                     for (int sdr = 0; sdr < splits; ++sdr) v += src[sdr * (CHUNK_F * NT)];
-                    const float sc = scaled && t < M ? ctrl->rstd[t] : 1.0f;
+                    if (t < M) v = normed(v, t, fsum);
                     if (EPI == 1) {
                         // (every lane takes part in the exchange of the gated epilogue; rows past M are not stored)
-                        const float g = v * sc + fbias;
+                        const float g = v + fbias;
                         const float other = __shfl_xor_sync(0xffffffffu, g, 4);
                         if (ok && t < M && (fi & 4) == 0 && fo + 4 < N)
-                            y[(size_t)t * (N >> 1) + ((fo >> 3) << 2) + (fo & 3)] = from_f<OutT>(glu_gate(g, nf.gate_slope) * other);
+                            y[(size_t)t * (N >> 1) + ((fo >> 3) << 2) + (fo & 3)] = from_f<OutT>(glu_gate(g, nf.gate_slope, nf.gate_cubic) * other);
                     } else if (ok && t < M && fo < N) {
-                        y[(size_t)t * N + fo] = from_f<OutT>(v * sc + fbias);
+                        y[(size_t)t * N + fo] = from_f<OutT>(v + fbias);
                     }
                 }
             }
@@ -495,7 +553,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                 float v = 0.f;
                 for (int s = 0; s < splits; ++s) v += part[(slot * splits + s) * SF + (int)threadIdx.x];
                 if (EPI == 2) {
-                    const float r_old = slot == 0 ? sink_r0 : (good && f < N ? nf.resid[(size_t)t * N + f] : 0.f);
+                    const float r_old = slot == 0 ? sink_r0 : (good && f < N && nf.resid_in != nullptr ? nf.resid_in[(size_t)t * N + f] : 0.f);
                     sink_token(nf, ctrl->red, v, t, f, tile, M, N, good, r_old, sink_w, bias);
                 } else if constexpr (EPI == 3) {
                     if (good && f < N) {
@@ -503,7 +561,7 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
                         streams_token(nf, ctrl->coef, st_x, v, bias, sink_w, st_b, t, f, N);
                     }
                 } else if (good) {
-                    store_token<EPI, OutT>(y, v * (scaled ? ctrl->rstd[t] : 1.0f) + bias, t, f, lane, N, nf.gate_slope);
+                    store_token<EPI, OutT>(y, normed(v, t, colsum) + bias, t, f, lane, N, nf);
                 }
             }
         }
@@ -524,11 +582,23 @@ __global__ __launch_bounds__(S_THREADS) void stream_gemm_kernel(const __grid_con
 int g_target_ctas = 0;      // 0: twice the number of SMs
 int g_min_stages = -1;      // stages a CTA is given at least (measurements; -1: by the rows, see launch_stream)
 
+// The second pair of operands of a product (K 0: there is none).
+struct SecondSource {
+    const void* x = nullptr;
+    long long ldx = 0;
+    const void* W = nullptr;
+    int K = 0;
+};
+
 template <int NT, int EPI, typename OutT>
 int launch_stream(const void* x, long long ldx, const void* W, void* y, int M, int N, int K, const NormFuse& nf,
-                  cudaStream_t stream) {
-    CUtensorMap map_w, map_x;
+                  cudaStream_t stream, const SecondSource& two = SecondSource()) {
+    CUtensorMap map_w, map_x, map_w2, map_x2;
     if (!make_map(&map_w, W, N, K, SF) || !make_map(&map_x, x, M, K, NT, ldx)) return RLIS_ERR_UNSUPPORTED;
+    map_w2 = map_w;
+    map_x2 = map_x;
+    if (two.K > 0 && (!make_map(&map_w2, two.W, N, two.K, SF) || !make_map(&map_x2, two.x, M, two.K, NT, two.ldx)))
+        return RLIS_ERR_UNSUPPORTED;
     static bool attr_done = false;
     if (!attr_done) {
         cudaFuncSetAttribute(stream_gemm_kernel<NT, EPI, OutT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -536,7 +606,7 @@ int launch_stream(const void* x, long long ldx, const void* W, void* y, int M, i
         cudaFuncSetAttribute(stream_gemm_kernel<NT, EPI, OutT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         attr_done = true;
     }
-    const int tiles = (N + SF - 1) / SF, k_blocks = (K + SK - 1) / SK;
+    const int tiles = (N + SF - 1) / SF, k_blocks = (K + SK - 1) / SK + (two.K + SK - 1) / SK;
     int target = g_target_ctas;
     if (target <= 0) {
         int dev = 0, sms = 148;
@@ -570,8 +640,8 @@ int launch_stream(const void* x, long long ldx, const void* W, void* y, int M, i
     if (n_stages < min_stages) n_stages = min_stages < STG ? min_stages : STG;
     while (n_stages < STG && (size_t)n_stages * stage_bytes < exchange) ++n_stages;
     rlis_launch_cluster(stream_gemm_kernel<NT, EPI, OutT>, dim3((unsigned)tiles, (unsigned)splits), S_THREADS,
-                        stream_smem_bytes<NT>(n_stages), stream, dim3(1, (unsigned)splits, 1), map_w, map_x, (OutT*)y, M, N, K,
-                        per, n_stages, nf);
+                        stream_smem_bytes<NT>(n_stages), stream, dim3(1, (unsigned)splits, 1), map_w, map_x, map_w2, map_x2,
+                        (OutT*)y, M, N, K, two.K, per, n_stages, nf);
     return RLIS_LAUNCH_CHECK();
 }
 
@@ -631,15 +701,49 @@ static bool stream_takes(const void* x, long long ldx, const void* W, int M, int
     return M <= 128 && K > 0 && (K & 7) == 0 && ldx >= K && (ldx & 7) == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 &&
            (reinterpret_cast<uintptr_t>(x) & 15) == 0;
 }
+// Layer norm (scaled rows and sink): in_sums / out_sums beside the sums of squares, and colsum [N] with in_sums.  Sink:
+// resid_in what the result is added to (resid: in place; null: nothing), exact 1: unrounded.  Mixed (epilogue 4, M up to 16):
+// y [M, n_plain] and y2 [M, (N - n_plain) / 2], n_plain a multiple of 8.  x2 not null (M up to 16): a second pair, K2 wide.
+struct RlisStreamExtra {
+    const float *in_sums, *colsum;
+    const float* resid_in;
+    float* out_sums;
+    int exact, n_plain;
+    void* y2;
+    float gate_cubic;
+    const void* x2;
+    long long ldx2;
+    const void* W2;
+    int K2;
+};
 extern "C" int rlis_stream_gemm_fused(const void* x, long long ldx, const void* W, void* y, int M, int N, int K, int out_dtype,
                                       int epilogue, const float* bias, const float* in_partials, int n_partials, int norm_dim,
                                       float eps, float* resid, const float* norm_w, void* xn, float* out_partials,
-                                      float gate_slope, cudaStream_t stream) {
+                                      float gate_slope, const RlisStreamExtra* extra, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     if (!stream_takes(x, ldx, W, M, K) || (epilogue == 1 && (N & 7) != 0)) return RLIS_ERR_UNSUPPORTED;
     NormFuse nf{};
     nf.gate_slope = gate_slope;
     nf.bias = bias;
+    nf.resid_in = resid;
+    SecondSource two;
+    if (extra != nullptr) {
+        nf.resid_in = extra->resid_in;
+        nf.out_sums = extra->out_sums;
+        nf.exact = extra->exact;
+        nf.gate_cubic = extra->gate_cubic;
+        if (extra->in_sums != nullptr && (in_partials == nullptr || extra->colsum == nullptr)) return RLIS_ERR_UNSUPPORTED;
+        nf.in_sums = extra->in_sums;
+        nf.colsum = extra->colsum;
+        if (extra->x2 != nullptr) {
+            if (M > 16 || in_partials != nullptr || !stream_takes(extra->x2, extra->ldx2, extra->W2, M, extra->K2))
+                return RLIS_ERR_UNSUPPORTED;
+            two.x = extra->x2;
+            two.ldx = extra->ldx2;
+            two.W = extra->W2;
+            two.K = extra->K2;
+        }
+    }
     if (in_partials != nullptr) {
         if (epilogue == 2 || n_partials <= 0 || norm_dim <= 0) return RLIS_ERR_UNSUPPORTED;
         nf.in_partials = in_partials;
@@ -654,7 +758,19 @@ extern "C" int rlis_stream_gemm_fused(const void* x, long long ldx, const void* 
         nf.norm_w = norm_w;
         nf.xn = reinterpret_cast<bf16*>(xn);
         nf.out_partials = out_partials;
-        return launch_stream<16, 2, bf16>(x, ldx, W, nullptr, M, N, K, nf, stream);
+        return launch_stream<16, 2, bf16>(x, ldx, W, nullptr, M, N, K, nf, stream, two);
+    }
+    if (epilogue == 4) {
+        if (M > 16 || extra == nullptr || extra->y2 == nullptr || extra->n_plain < 0 || extra->n_plain > N || (extra->n_plain & 7) != 0 ||
+            (N & 7) != 0)
+            return RLIS_ERR_UNSUPPORTED;
+        nf.n_plain = extra->n_plain;
+        nf.y2 = reinterpret_cast<bf16*>(extra->y2);
+        return launch_stream<16, 4, bf16>(x, ldx, W, y, M, N, K, nf, stream, two);
+    }
+    if (two.K > 0) {
+        if (epilogue != 0 || out_dtype != RLIS_BF16) return RLIS_ERR_UNSUPPORTED;
+        return launch_stream<16, 0, bf16>(x, ldx, W, y, M, N, K, nf, stream, two);
     }
     if (M <= 16) return dispatch_stream<16>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
     if (M <= 32) return dispatch_stream<32>(x, ldx, W, y, M, N, K, out_dtype, epilogue, nf, stream);
