@@ -16,6 +16,8 @@
 // b cos + a sin) either way).  `proj_bias` (float32, one entry a column of the projection's row): added to queries,
 // keys and values as they are read.  `gate_cols` > 1: the gate has one logit a channel of every head (gate[t, h *
 // dv + c]) instead of one a head.
+// `maps` > 1 (norm_store): a query or key head holds `maps` vectors of d entries side by side, each rotated and normed on its
+// own, over one value; the cache keeps a key head's vectors as one row of maps * d entries.
 //
 // row_norm_store: queries and keys RMS-normed over their whole projections (all heads together, one weight an entry), before
 // they are split into heads.
@@ -44,12 +46,12 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_kernel(
     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slots,
     int n_units, int nh, int nkv, int d, int dv, int page_size,
     const float* __restrict__ inv_freq, int rot_dims, float rot_mag, const int* __restrict__ positions,
-    float q_temp_coef, int q_temp_every, int rot_half, const float* __restrict__ proj_bias) {
+    float q_temp_coef, int q_temp_every, int rot_half, const float* __restrict__ proj_bias, int maps) {
     pdl_wait_and_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int unit = blockIdx.x * WARPS + warp;
     if (unit >= n_units) return;
-    const int per = nh + nkv;
+    const int per = nh + nkv * maps;           // (nh counts the query vectors)
     const int t = unit / per, u = unit - t * per;
     const T* row = proj + (size_t)t * stride;
     const bool is_q = u < nh;
@@ -110,10 +112,10 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_kernel(
         const int slot = slots != nullptr ? slots[t] : -1;
         if (slot >= 0) {
             const long long page = slot / page_size;
-            const int off = slot % page_size;
-            const long long r0 = (page * nkv + (u - nh)) * page_size + off;
-            dst = k_cache + r0 * d;
-            vrow = r0 * dv;
+            const int off = slot % page_size, g = (u - nh) / maps, j = (u - nh) - g * maps;
+            const long long r0 = (page * nkv + g) * page_size + off;
+            dst = k_cache + (r0 * maps + j) * d;
+            if (j == 0) vrow = r0 * dv;
         }
     }
     if (dst != nullptr) {
@@ -124,7 +126,7 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_kernel(
         }
     }
     if (vrow >= 0) {
-        const int g = u - nh;
+        const int g = (u - nh) / maps;
         const T* vs = row + v_off + g * dv;
         const float* vb = proj_bias != nullptr ? proj_bias + v_off + g * dv : nullptr;
         const T* vo = v_other != nullptr ? v_other + (size_t)t * v_other_stride + g * dv : nullptr;
@@ -147,7 +149,7 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_vec_kernel(
     T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ slots,
     int n_units, int nh, int nkv, int d, int dv, int page_size, int lanes,
     const float* __restrict__ inv_freq, int rot_dims, float rot_mag, const int* __restrict__ positions,
-    float q_temp_coef, int q_temp_every, int rot_half, const float* __restrict__ proj_bias) {
+    float q_temp_coef, int q_temp_every, int rot_half, const float* __restrict__ proj_bias, int maps) {
     pdl_wait_and_trigger();
     constexpr int VN = Vec16<T>::N;
     const int lane = threadIdx.x & 31;
@@ -155,7 +157,7 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_vec_kernel(
     const int per_warp = 32 / lanes;
     const int unit = (blockIdx.x * WARPS + (threadIdx.x >> 5)) * per_warp + sub;
     const bool live = unit < n_units;
-    const int per = nh + nkv;
+    const int per = nh + nkv * maps;
     const int t = live ? unit / per : 0, u = live ? unit - t * per : 0;
     const T* row = proj + (size_t)t * stride;
     const bool is_q = u < nh;
@@ -219,9 +221,10 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_vec_kernel(
     } else {
         const int slot = slots != nullptr ? slots[t] : -1;
         if (slot >= 0) {
-            const long long r0 = ((long long)(slot / page_size) * nkv + (u - nh)) * page_size + slot % page_size;
-            dst = k_cache + r0 * d;
-            vrow = r0 * dv;
+            const int g = (u - nh) / maps, j = (u - nh) - g * maps;
+            const long long r0 = ((long long)(slot / page_size) * nkv + g) * page_size + slot % page_size;
+            dst = k_cache + (r0 * maps + j) * d;
+            if (j == 0) vrow = r0 * dv;
         }
     }
     if (dst != nullptr) {
@@ -231,7 +234,7 @@ __global__ __launch_bounds__(WARPS * 32) void qk_norm_store_vec_kernel(
         *reinterpret_cast<uint4*>(dst + li * VN) = *reinterpret_cast<const uint4*>(o);
     }
     if (vrow >= 0) {
-        const int g = u - nh;
+        const int g = (u - nh) / maps;
         const T* vs = row + v_off + g * dv;
         const T* vo = v_other != nullptr ? v_other + (size_t)t * v_other_stride + g * dv : nullptr;
         for (int c = li * VN; c < dv; c += lanes * VN) {
@@ -425,20 +428,22 @@ __global__ __launch_bounds__(WARPS * 32) void attn_bias_kernel(
 // proj [T, stride]: the stacked projection's rows; queries at column q_off (nh heads of d), keys at
 // k_off (nkv of d), values at v_off (nkv of dv).  q_w, k_w float32 [d] (null: no norm).  v_other (null:
 // no mixing): rows of another layer's values [T, v_other_stride], mixed in with weight lambda.
-// slots null: nothing is stored (the call reads another call's cache) and only q_out is made.
+// maps: vectors a query or key head holds (1: ordinary heads; then q_out has nh * maps of them and the keys' cache rows maps * d
+// entries).  slots null: nothing is stored (the call reads another call's cache) and only q_out is made.
 extern "C" int rlis_qk_norm_store(const void* proj, long long stride, int q_off, int k_off, int v_off,
                                   const float* q_w, const float* k_w, float eps, const void* v_other,
                                   long long v_other_stride, float lambda, void* q_out, void* k_cache, void* v_cache,
                                   const int* slots, int n_tokens, int nh, int nkv, int d, int dv, int page_size,
                                   const float* inv_freq, int rot_dims, float rot_mag, const int* positions,
-                                  float q_temp_coef, int q_temp_every, int rot_half, const float* proj_bias, int dtype,
+                                  float q_temp_coef, int q_temp_every, int rot_half, const float* proj_bias, int maps, int dtype,
                                   cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
-    if (d <= 0 || d > MAX_D || dv <= 0 || nh <= 0 || nkv <= 0) return RLIS_ERR_UNSUPPORTED;
+    if (d <= 0 || d > MAX_D || dv <= 0 || nh <= 0 || nkv <= 0 || maps < 1) return RLIS_ERR_UNSUPPORTED;
+    nh *= maps;                                // from here on the query vectors
     if (rot_dims < 0 || rot_dims > d || (rot_dims & 1) || (rot_dims > 0 && (inv_freq == nullptr || positions == nullptr)) ||
         (q_temp_every > 0 && positions == nullptr))
         return RLIS_ERR_UNSUPPORTED;
-    const long long units = (long long)n_tokens * (nh + nkv);
+    const long long units = (long long)n_tokens * (nh + (long long)nkv * maps);
     if (units > 0x7fffffffLL) return RLIS_ERR_UNSUPPORTED;
     {
         // the vector form where everything lies on 16-byte boundaries and a head is VN * 2^k elements
@@ -458,12 +463,12 @@ extern "C" int rlis_qk_norm_store(const void* proj, long long stride, int q_off,
                 rlis_launch(qk_norm_store_vec_kernel<float>, vblocks, WARPS * 32, 0, stream, (const float*)proj, stride, q_off,
                             k_off, v_off, q_w, k_w, eps, (const float*)v_other, v_other_stride, lambda, (float*)q_out,
                             (float*)k_cache, (float*)v_cache, slots, (int)units, nh, nkv, d, dv, page_size, lanes, inv_freq, rot_dims,
-                            rot_mag, positions, q_temp_coef, q_temp_every, rot_half, proj_bias);
+                            rot_mag, positions, q_temp_coef, q_temp_every, rot_half, proj_bias, maps);
             else
                 rlis_launch(qk_norm_store_vec_kernel<bf16>, vblocks, WARPS * 32, 0, stream, (const bf16*)proj, stride, q_off,
                             k_off, v_off, q_w, k_w, eps, (const bf16*)v_other, v_other_stride, lambda, (bf16*)q_out,
                             (bf16*)k_cache, (bf16*)v_cache, slots, (int)units, nh, nkv, d, dv, page_size, lanes, inv_freq, rot_dims,
-                            rot_mag, positions, q_temp_coef, q_temp_every, rot_half, proj_bias);
+                            rot_mag, positions, q_temp_coef, q_temp_every, rot_half, proj_bias, maps);
             return RLIS_LAUNCH_CHECK();
         }
     }
@@ -472,12 +477,12 @@ extern "C" int rlis_qk_norm_store(const void* proj, long long stride, int q_off,
         rlis_launch(qk_norm_store_kernel<float>, blocks, WARPS * 32, 0, stream, (const float*)proj, stride, q_off, k_off,
                     v_off, q_w, k_w, eps, (const float*)v_other, v_other_stride, lambda, (float*)q_out, (float*)k_cache,
                     (float*)v_cache, slots, (int)units, nh, nkv, d, dv, page_size, inv_freq, rot_dims, rot_mag, positions,
-                    q_temp_coef, q_temp_every, rot_half, proj_bias);
+                    q_temp_coef, q_temp_every, rot_half, proj_bias, maps);
     else if (dtype == RLIS_BF16)
         rlis_launch(qk_norm_store_kernel<bf16>, blocks, WARPS * 32, 0, stream, (const bf16*)proj, stride, q_off, k_off,
                     v_off, q_w, k_w, eps, (const bf16*)v_other, v_other_stride, lambda, (bf16*)q_out, (bf16*)k_cache,
                     (bf16*)v_cache, slots, (int)units, nh, nkv, d, dv, page_size, inv_freq, rot_dims, rot_mag, positions,
-                    q_temp_coef, q_temp_every, rot_half, proj_bias);
+                    q_temp_coef, q_temp_every, rot_half, proj_bias, maps);
     else
         return RLIS_ERR_UNSUPPORTED;
     return RLIS_LAUNCH_CHECK();

@@ -7,7 +7,9 @@
 //                     (and, for the layer that projects both latents at once, the query latent's norm)
 //   latent_q_rope   : qa[t, h, r:] = rotate(q[t, h, d:]), float32 (or bfloat16 for the tensor-core kernels)
 //   attention_latent: softmax over keys 0..pos (or the last `window`), optionally with one more
-//                     term exp(sink_h) in the denominator that has no value
+//                     term exp(sink_h) in the denominator that has no value; a head's result is
+//                     multiplied by sigmoid(gate_h) where a gate is given (the value map is linear,
+//                     so gating the sum over latents gates the head)
 //
 // Rotation: rotate-half over the first `rot_dims` entries of the rotated part, angle = position *
 // inv_freq[i] in float32, cos and sin multiplied by `mag`; the remaining entries pass unchanged.
@@ -72,7 +74,7 @@ __global__ __launch_bounds__(128) void latent_kv_store_kernel(
 }
 
 template <typename T, typename TO>
-__global__ void latent_q_rope_kernel(const T* __restrict__ q, TO* __restrict__ qa,
+__global__ void latent_q_rope_kernel(const T* __restrict__ q, long long q_stride, TO* __restrict__ qa,
                                      const float* __restrict__ inv_freq, const int* __restrict__ positions,
                                      int n_heads, int d_plain, int rot_width, int rot_dims, int rank, float mag,
                                      long long total) {
@@ -82,7 +84,7 @@ __global__ void latent_q_rope_kernel(const T* __restrict__ q, TO* __restrict__ q
     const int i = (int)(idx % rot_width);
     const long long th = idx / rot_width;                      // token * heads + head
     const int t = (int)(th / n_heads);
-    const T* src = q + th * (d_plain + rot_width) + d_plain;
+    const T* src = q + (size_t)t * q_stride + (size_t)(th - (long long)t * n_heads) * (d_plain + rot_width) + d_plain;
     float v = to_f<T>(src[i]);
     if (i < rot_dims) {
         const int half = rot_dims / 2;
@@ -103,7 +105,7 @@ __global__ __launch_bounds__(WARPS * 32) void attention_latent_kernel(
     const float* __restrict__ qa, const T* __restrict__ cache, T* __restrict__ out,
     const float* __restrict__ sinks, const int* __restrict__ seq_of_token, const int* __restrict__ positions,
     const int* __restrict__ block_tables, const int* __restrict__ token_rows, int max_blocks, int n_rows,
-    int nh, int dk, int dv, int page_size, float scale, int window) {
+    int nh, int dk, int dv, int page_size, float scale, int window, const T* __restrict__ gate, long long gate_stride) {
     pdl_wait();
     extern __shared__ float qs_all[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -178,7 +180,8 @@ __global__ __launch_bounds__(WARPS * 32) void attention_latent_kernel(
         m = m_new;
     }
     T* orow = out + ((size_t)t * nh + h) * dv;
-    const float inv_l = 1.0f / l;
+    float inv_l = 1.0f / l;
+    if (gate != nullptr) inv_l *= 1.0f / (1.0f + expf(-to_f<T>(gate[(size_t)t * gate_stride + h])));
 #pragma unroll
     for (int i = 0; i < MAX_DV_REGS; ++i) {
         const int dim = lane + 32 * i;
@@ -209,7 +212,7 @@ extern "C" int rlis_latent_kv_store(const void* z, long long z_stride, const flo
 }
 
 // out_bf16 != 0: qa is bfloat16 (for the tensor-core attention kernels), else float32.
-extern "C" int rlis_latent_q_rope(const void* q, void* qa, const float* inv_freq, const int* positions,
+extern "C" int rlis_latent_q_rope(const void* q, long long q_stride, void* qa, const float* inv_freq, const int* positions,
                                   int n_tokens, int n_heads, int d_plain, int rot_width, int rot_dims, int rank,
                                   float mag, int dtype, int out_bf16, cudaStream_t stream) {
     const long long total = (long long)n_tokens * n_heads * rot_width;
@@ -217,23 +220,25 @@ extern "C" int rlis_latent_q_rope(const void* q, void* qa, const float* inv_freq
     if (rot_dims < 0 || rot_dims > rot_width || rot_dims % 2) return RLIS_ERR_UNSUPPORTED;
     const unsigned blocks = (unsigned)((total + 255) / 256);
     if (dtype == RLIS_F32 && !out_bf16)
-        rlis_launch(latent_q_rope_kernel<float, float>, blocks, 256, 0, stream, (const float*)q, (float*)qa, inv_freq,
+        rlis_launch(latent_q_rope_kernel<float, float>, blocks, 256, 0, stream, (const float*)q, q_stride, (float*)qa, inv_freq,
                     positions, n_heads, d_plain, rot_width, rot_dims, rank, mag, total);
     else if (dtype == RLIS_BF16 && !out_bf16)
-        rlis_launch(latent_q_rope_kernel<bf16, float>, blocks, 256, 0, stream, (const bf16*)q, (float*)qa, inv_freq,
+        rlis_launch(latent_q_rope_kernel<bf16, float>, blocks, 256, 0, stream, (const bf16*)q, q_stride, (float*)qa, inv_freq,
                     positions, n_heads, d_plain, rot_width, rot_dims, rank, mag, total);
     else if (dtype == RLIS_BF16)
-        rlis_launch(latent_q_rope_kernel<bf16, bf16>, blocks, 256, 0, stream, (const bf16*)q, (bf16*)qa, inv_freq,
+        rlis_launch(latent_q_rope_kernel<bf16, bf16>, blocks, 256, 0, stream, (const bf16*)q, q_stride, (bf16*)qa, inv_freq,
                     positions, n_heads, d_plain, rot_width, rot_dims, rank, mag, total);
     else
         return RLIS_ERR_UNSUPPORTED;
     return RLIS_LAUNCH_CHECK();
 }
 
+// gate (null: none): logits in the element type, head h of token t at gate[t * gate_stride + h].
 extern "C" int rlis_attention_latent(const float* qa, const void* cache, void* out, const float* sinks,
                                      const int* seq_of_token, const int* positions, const int* block_tables,
                                      const int* token_rows, int max_blocks, int n_tokens, int nh, int dk, int dv,
-                                     int page_size, float scale, int window, int dtype, cudaStream_t stream) {
+                                     int page_size, float scale, int window, const void* gate, long long gate_stride,
+                                     int dtype, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (dk <= 0 || dv <= 0 || dv > dk || dv > 32 * MAX_DV_REGS || dk > 2048 || nh <= 0) return RLIS_ERR_UNSUPPORTED;
     const long long n_rows = (long long)n_tokens * nh;
@@ -243,11 +248,11 @@ extern "C" int rlis_attention_latent(const float* qa, const void* cache, void* o
     if (dtype == RLIS_F32)
         rlis_launch(attention_latent_kernel<float>, blocks, WARPS * 32, smem, stream, qa, (const float*)cache,
                     (float*)out, sinks, seq_of_token, positions, block_tables, token_rows, max_blocks, (int)n_rows,
-                    nh, dk, dv, page_size, scale, window);
+                    nh, dk, dv, page_size, scale, window, (const float*)gate, gate_stride);
     else if (dtype == RLIS_BF16)
         rlis_launch(attention_latent_kernel<bf16>, blocks, WARPS * 32, smem, stream, qa, (const bf16*)cache,
                     (bf16*)out, sinks, seq_of_token, positions, block_tables, token_rows, max_blocks, (int)n_rows,
-                    nh, dk, dv, page_size, scale, window);
+                    nh, dk, dv, page_size, scale, window, (const bf16*)gate, gate_stride);
     else
         return RLIS_ERR_UNSUPPORTED;
     return RLIS_LAUNCH_CHECK();

@@ -41,7 +41,13 @@ struct LatentArgs {
     int max_blocks, nh, dk, page_size, window, pieces, piece_keys;
     float scale;
     int q_bf16;
+    const bf16* gate;         // logits, one a head: head h of token t at gate[t * gate_stride + h]; null: none
+    long long gate_stride;
 };
+
+__device__ __forceinline__ float latent_gate(const bf16* gate, long long stride, int t, int h) {
+    return gate != nullptr ? 1.0f / (1.0f + expf(-__bfloat162float(gate[(size_t)t * stride + h]))) : 1.0f;
+}
 
 // Prompts: 64 query rows (tokens of one head) a CTA, four warp pairs, stages of 64 keys.
 template <int DV>
@@ -279,15 +285,17 @@ __global__ __launch_bounds__(256) void latent_flash_kernel(const LatentArgs a) {
         stage ^= 1;
     }
 
-    const float inv0 = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f;
-    const float inv1 = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
+    float inv0 = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f;
+    float inv1 = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
     if (rv0) {
+        inv0 *= latent_gate(a.gate, a.gate_stride, q_row0 + row_base + g, head0);
         bf16* o = a.out + ((size_t)(q_row0 + row_base + g) * nh + head0) * DV + col0;
 #pragma unroll
         for (int n = 0; n < NO; ++n)
             *reinterpret_cast<uint32_t*>(o + n * 8 + 2 * c) = pack_bf16(oacc[n][0] * inv0, oacc[n][1] * inv0);
     }
     if (rv1) {
+        inv1 *= latent_gate(a.gate, a.gate_stride, q_row0 + row_base + g + 8, head0);
         bf16* o = a.out + ((size_t)(q_row0 + row_base + g + 8) * nh + head0) * DV + col0;
 #pragma unroll
         for (int n = 0; n < NO; ++n)
@@ -325,8 +333,9 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
     const int head0 = blockIdx.x * 16;
     const int pos = a.ctx_lens[b] - 1;
     const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-    const int k_lo = max(lo, (int)blockIdx.z * a.piece_keys);
-    const int k_hi = min(pos + 1, (int)(blockIdx.z + 1) * a.piece_keys);
+    // the pieces cut what the token sees: they start at the window's first key
+    const int k_lo = lo + (int)blockIdx.z * a.piece_keys;
+    const int k_hi = min(pos + 1, k_lo + a.piece_keys);
     const int* table = a.block_tables + (size_t)b * a.max_blocks;
     const int page_size = a.page_size;
 
@@ -488,14 +497,16 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
     cp_async_wait<0>();
 
     if (a.pieces == 1) {
-        const float inv0 = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f, inv1 = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
+        float inv0 = l_run[0] > 0.f ? 1.0f / l_run[0] : 0.f, inv1 = l_run[1] > 0.f ? 1.0f / l_run[1] : 0.f;
         if (rv0) {
+            inv0 *= latent_gate(a.gate, a.gate_stride, q_row0, h0);
             bf16* o = a.out + ((size_t)q_row0 * nh + h0) * DV + col0;
 #pragma unroll
             for (int n = 0; n < NO; ++n)
                 *reinterpret_cast<uint32_t*>(o + n * 8 + 2 * c) = pack_bf16(oacc[n][0] * inv0, oacc[n][1] * inv0);
         }
         if (rv1) {
+            inv1 *= latent_gate(a.gate, a.gate_stride, q_row0, h1);
             bf16* o = a.out + ((size_t)q_row0 * nh + h1) * DV + col0;
 #pragma unroll
             for (int n = 0; n < NO; ++n)
@@ -540,7 +551,8 @@ int launch_latent_decode(const LatentArgs& a, dim3 grid, cudaStream_t stream) {
 // pieces' weights exp2(max_p - max) are worked out once, by one thread a piece.
 template <int DV>
 __global__ void latent_merge_kernel(const float* __restrict__ scratch, bf16* __restrict__ out,
-                                    const int* __restrict__ dec_rows, int nh, int head_tiles, int pieces) {
+                                    const int* __restrict__ dec_rows, int nh, int head_tiles, int pieces,
+                                    const bf16* __restrict__ gate, long long gate_stride) {
     pdl_wait_and_trigger();
     extern __shared__ float wts[];                 // [pieces] weights, then [pieces] scratch
     __shared__ float red[33];
@@ -565,7 +577,7 @@ __global__ void latent_merge_kernel(const float* __restrict__ scratch, bf16* __r
         l += part[p * piece_stride + DV + 1] * w;
     }
     l = block_sum(l, red);                         // (its barriers also publish the weights)
-    const float inv = l > 0.f ? 1.0f / l : 0.f;
+    const float inv = (l > 0.f ? 1.0f / l : 0.f) * latent_gate(gate, gate_stride, dec_rows[di], h);
     bf16* o = out + ((size_t)dec_rows[di] * nh + h) * DV;
     // two columns a thread at a time (rows of DV + 2 floats are 8-byte aligned), eight pieces' loads in flight
     for (int col = threadIdx.x * 2; col < DV; col += blockDim.x * 2) {
@@ -609,11 +621,11 @@ extern "C" int rlis_attention_latent_prefill(const void* qa, int q_bf16, const v
                                              const int* tiles, int n_tiles, const int* cu_seqlens,
                                              const int* ctx_lens, const int* block_tables, int max_blocks, int nh,
                                              int dk, int dv, int page_size, float scale, int window,
-                                             cudaStream_t stream) {
+                                             const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (!rlis_attention_latent_mma_takes(dk, dv) || n_tiles > 65535 || nh <= 0) return RLIS_ERR_UNSUPPORTED;
     LatentArgs a = {qa, (const bf16*)cache, (bf16*)out, sinks, tiles, cu_seqlens, ctx_lens, block_tables, nullptr,
-                    nullptr, nullptr, max_blocks, nh, dk, page_size, window, 1, 0, scale, q_bf16};
+                    nullptr, nullptr, max_blocks, nh, dk, page_size, window, 1, 0, scale, q_bf16, (const bf16*)gate, gate_stride};
     dim3 grid(nh, n_tiles);
     switch (dv) {
         case 64: return launch_latent<64>(a, grid, stream);
@@ -629,14 +641,16 @@ extern "C" int rlis_attention_latent_decode(const void* qa, int q_bf16, const vo
                                             float* scratch, const int* dec_rows, const int* dec_seqs,
                                             const int* ctx_lens, const int* block_tables, int max_blocks, int n_dec,
                                             int nh, int dk, int dv, int page_size, float scale, int window,
-                                            int pieces, int piece_keys, cudaStream_t stream) {
+                                            int pieces, int piece_keys, const void* gate, long long gate_stride,
+                                            cudaStream_t stream) {
     if (n_dec <= 0) return 0;
     if (!rlis_attention_latent_mma_takes(dk, dv) || n_dec > 65535 || nh <= 0 || pieces < 1 || pieces > 4096 ||
         (pieces > 1 && (scratch == nullptr || piece_keys <= 0 || piece_keys % LF_BN_MAX)))
         return RLIS_ERR_UNSUPPORTED;
     if (pieces == 1) piece_keys = 0x40000000;
     LatentArgs a = {qa, (const bf16*)cache, (bf16*)out, sinks, nullptr, nullptr, ctx_lens, block_tables, dec_rows,
-                    dec_seqs, scratch, max_blocks, nh, dk, page_size, window, pieces, piece_keys, scale, q_bf16};
+                    dec_seqs, scratch, max_blocks, nh, dk, page_size, window, pieces, piece_keys, scale, q_bf16,
+                    (const bf16*)gate, gate_stride};
     const int head_tiles = (nh + 15) / 16;
     dim3 grid(head_tiles, n_dec, pieces);
     int rc;
@@ -649,10 +663,10 @@ extern "C" int rlis_attention_latent_decode(const void* qa, int q_bf16, const vo
     if (rc != 0 || pieces == 1) return rc;
     dim3 mgrid(nh, n_dec);
     switch (dv) {
-        case 64: rlis_launch(latent_merge_kernel<64>, mgrid, 32, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces); break;
-        case 128: rlis_launch(latent_merge_kernel<128>, mgrid, 64, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces); break;
-        case 256: rlis_launch(latent_merge_kernel<256>, mgrid, 128, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces); break;
-        default: rlis_launch(latent_merge_kernel<512>, mgrid, 256, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces); break;
+        case 64: rlis_launch(latent_merge_kernel<64>, mgrid, 32, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces, (const bf16*)gate, gate_stride); break;
+        case 128: rlis_launch(latent_merge_kernel<128>, mgrid, 64, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces, (const bf16*)gate, gate_stride); break;
+        case 256: rlis_launch(latent_merge_kernel<256>, mgrid, 128, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces, (const bf16*)gate, gate_stride); break;
+        default: rlis_launch(latent_merge_kernel<512>, mgrid, 256, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces, (const bf16*)gate, gate_stride); break;
     }
     return RLIS_LAUNCH_CHECK();
 }

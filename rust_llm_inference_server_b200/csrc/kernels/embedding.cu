@@ -26,7 +26,7 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
 // multiple of 4.
 __global__ void embedding_sink_kernel(const int* __restrict__ ids, const bf16* __restrict__ table,
                                       float* __restrict__ out, const float* __restrict__ norm_weight,
-                                      bf16* __restrict__ xn, float* __restrict__ partials, int n_tokens,
+                                      bf16* __restrict__ xn, float* __restrict__ partials, float* __restrict__ sums, int n_tokens,
                                       int hidden, int vocab, float scale) {
     pdl_wait_and_trigger();
     const int t = blockIdx.x;
@@ -37,7 +37,7 @@ __global__ void embedding_sink_kernel(const int* __restrict__ ids, const bf16* _
     const int tiles = (hidden + 127) / 128;
     for (int tile = warp; tile < tiles; tile += warps) {
         const int f = tile * 128 + lane * 4;
-        float ss = 0.f;
+        float ss = 0.f, s1 = 0.f;
         if (f < hidden) {
             float v[4] = {0.f, 0.f, 0.f, 0.f};
             if (known) {
@@ -53,21 +53,27 @@ __global__ void embedding_sink_kernel(const int* __restrict__ ids, const bf16* _
             pk.y = pack_bf16(v[2] * w.z, v[3] * w.w);
             *reinterpret_cast<uint2*>(xn + (size_t)t * hidden + f) = pk;
             ss = (v[0] * v[0] + v[1] * v[1]) + (v[2] * v[2] + v[3] * v[3]);
+            s1 = (v[0] + v[1]) + (v[2] + v[3]);
         }
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
         if (lane == 0) partials[(size_t)tile * n_tokens + t] = ss;
+        if (sums != nullptr) {
+            s1 = warp_sum(s1);
+            if (lane == 0) sums[(size_t)tile * n_tokens + t] = s1;
+        }
     }
 }
 
-// out [n_tokens, hidden] float32, xn [n_tokens, hidden] bf16, partials [ceil(hidden / 128), n_tokens].
+// out [n_tokens, hidden] float32, xn [n_tokens, hidden] bf16, partials [ceil(hidden / 128), n_tokens]; sums (null: not
+// wanted) like partials: the sums of the rows, for a layer norm.
 extern "C" int rlis_embedding_sink(const int* ids, const void* table, float* out, const float* norm_weight,
-                                   void* xn, float* partials, int n_tokens, int hidden, int vocab, float scale,
+                                   void* xn, float* partials, float* sums, int n_tokens, int hidden, int vocab, float scale,
                                    cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if ((hidden & 3) != 0) return RLIS_ERR_UNSUPPORTED;
     rlis_launch(embedding_sink_kernel, n_tokens, 128, 0, stream, ids, (const bf16*)table, out, norm_weight,
-                (bf16*)xn, partials, n_tokens, hidden, vocab, scale);
+                (bf16*)xn, partials, sums, n_tokens, hidden, vocab, scale);
     return RLIS_LAUNCH_CHECK();
 }
 

@@ -10,6 +10,7 @@ no reduced-precision matrix mode can enter.
 
 from __future__ import annotations
 
+import ctypes
 import functools
 
 import torch
@@ -97,7 +98,7 @@ def embedding(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: 
 def embedding_sink(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, scale: float | None, sink):
     """`embedding` for a step whose first norm is left to the product after it (`sink`, a
     ResidualSink over `out`): also returns that norm's ScaledRows, bf16(row * weight) and the sums of
-    squares of every 128 features.  bfloat16 tables whose width is a multiple of 8."""
+    squares (of a layer norm also the sums) of every 128 features.  bfloat16 tables whose width is a multiple of 8."""
     V, H = table.shape
     T = ids.shape[0]
     _req(ids, "ids", torch.int32, (T,))
@@ -107,12 +108,14 @@ def embedding_sink(ids: torch.Tensor, table: torch.Tensor, out: torch.Tensor, sc
     if sink.resid.data_ptr() != out.data_ptr() or H % 8:
         raise KernelError("embedding_sink: the sink is over another residual stream, or the width is no multiple of 8")
     xn = torch.empty((T, H), dtype=torch.bfloat16, device=out.device)
-    partials = torch.empty(((H + 127) // 128, T), dtype=torch.float32, device=out.device)
+    partials = torch.empty((2 if sink.centred else 1, (H + 127) // 128, T), dtype=torch.float32, device=out.device)
     check(lib().rlis_embedding_sink(ids.data_ptr(), table.data_ptr(), out.data_ptr(), sink.weight.data_ptr(),
-                                    xn.data_ptr(), partials.data_ptr(), T, H, V,
+                                    xn.data_ptr(), partials.data_ptr(), partials[1].data_ptr() if sink.centred else None, T, H, V,
                                     1.0 if scale is None else float(scale), _stream()), "embedding_sink")
     _count("embedding.sink")
-    return ScaledRows(xn, partials, H, sink.eps)
+    if sink.centred:
+        return ScaledRows(xn, partials[0], H, sink.eps, sums=partials[1], weight=sink.weight)
+    return ScaledRows(xn, partials[0], H, sink.eps)
 
 
 def logit_transform(logits: torch.Tensor, scale: float | None, soft_cap: float | None) -> torch.Tensor:
@@ -129,13 +132,7 @@ def logit_transform(logits: torch.Tensor, scale: float | None, soft_cap: float |
     return logits
 
 
-def rmsnorm(resid: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
-            delta: torch.Tensor | None = None, rows: torch.Tensor | None = None) -> torch.Tensor:
-    """If `delta` is given: resid += delta (float32).  out = rmsnorm(resid) * weight, rounded once.
-
-    resid float32 [T, H] (updated in place), weight float32 [H], out and delta in the activation
-    type.  With `rows` (int32 [R]): out [R, H] is computed from rows resid[rows] (+ delta[rows])
-    and resid is left unchanged."""
+def _norm_rows(name: str, resid, weight, eps: float, out, delta, rows) -> torch.Tensor:
     T, H = resid.shape
     _req(resid, "resid", torch.float32)
     _req(weight, "weight", torch.float32, (H,))
@@ -144,14 +141,34 @@ def rmsnorm(resid: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Te
         _req(rows, "rows", torch.int32, (None,))
         n_out = rows.shape[0]
     _req(out, "out", None, (n_out, H))
-    if delta is not None:
-        _req(delta, "delta", out.dtype, (T, H))
-    check(lib().rlis_rmsnorm(resid.data_ptr(), delta.data_ptr() if delta is not None else None,
-                             weight.data_ptr(), out.data_ptr(),
-                             rows.data_ptr() if rows is not None else None, n_out, H, float(eps),
-                             _code(out.dtype), _stream()), "rmsnorm")
-    _count("rmsnorm" if rows is None else "rmsnorm.rows")
+    deltas = tuple(delta) if isinstance(delta, (tuple, list)) else (delta,) if delta is not None else ()
+    if len(deltas) > 2:
+        raise KernelError(f"{name}: up to two additions, got {len(deltas)}")
+    for d in deltas:
+        _req(d, "delta", out.dtype, (T, H))
+    ptrs = [d.data_ptr() for d in deltas] + [None] * (2 - len(deltas))
+    check(getattr(lib(), "rlis_" + name)(resid.data_ptr(), *ptrs, weight.data_ptr(), out.data_ptr(),
+                                         rows.data_ptr() if rows is not None else None, n_out, H, float(eps),
+                                         _code(out.dtype), _stream()), name)
+    _count(name if rows is None else name + ".rows")
     return out
+
+
+def rmsnorm(resid: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+            delta=None, rows: torch.Tensor | None = None) -> torch.Tensor:
+    """If `delta` is given (a tensor, or a pair of them): resid += delta (float32).  out = rmsnorm(resid) * weight, rounded
+    once.
+
+    resid float32 [T, H] (updated in place), weight float32 [H], out and delta in the activation
+    type.  With `rows` (int32 [R]): out [R, H] is computed from rows resid[rows] (+ delta[rows])
+    and resid is left unchanged."""
+    return _norm_rows("rmsnorm", resid, weight, eps, out, delta, rows)
+
+
+def layer_norm(resid: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, delta=None,
+               rows: torch.Tensor | None = None) -> torch.Tensor:
+    """The same with the row's mean taken off first: out = (resid - mean) / sqrt(variance + eps) * weight."""
+    return _norm_rows("layer_norm", resid, weight, eps, out, delta, rows)
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, interleave: int = 0) -> torch.Tensor:
@@ -607,16 +624,17 @@ def latent_kv_store(z: torch.Tensor, weight: torch.Tensor, eps: float, inv_freq:
 def latent_q_rope(q: torch.Tensor, qa: torch.Tensor, inv_freq: torch.Tensor, rot_dims: int, magnitude: float,
                   positions: torch.Tensor, n_heads: int, d_plain: int, rot: int, rank: int) -> torch.Tensor:
     """qa[t, h, rank:] = the rotated part q[t, h, d_plain:] after rotation, in float32.  q [T, nh (d_plain
-    + rot)] in the activation type; qa [T, nh (rank + rot)] float32, or bfloat16 for the tensor-core
+    + rot)] in the activation type (may be a column slice of wider rows); qa [T, nh (rank + rot)] float32, or bfloat16 for the tensor-core
     attention kernels."""
     T = q.shape[0]
-    _req(q, "q", None, (T, n_heads * (d_plain + rot)))
+    if not q.is_cuda or tuple(q.shape) != (T, n_heads * (d_plain + rot)) or q.stride(1) != 1:
+        raise KernelError("latent_q_rope: q must be [T, nh (d_plain + rot)] rows on the device with unit stride")
     _req(qa, "qa", None, (T, n_heads * (rank + rot)))
     if qa.dtype not in (torch.float32, torch.bfloat16) or (qa.dtype == torch.bfloat16 and q.dtype != torch.bfloat16):
         raise KernelError(f"latent_q_rope: qa of {qa.dtype} for q of {q.dtype} is not taken")
     _req(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,))
     _req(positions, "positions", torch.int32, (T,))
-    check(lib().rlis_latent_q_rope(q.data_ptr(), qa.data_ptr(), inv_freq.data_ptr(), positions.data_ptr(), T,
+    check(lib().rlis_latent_q_rope(q.data_ptr(), q.stride(0), qa.data_ptr(), inv_freq.data_ptr(), positions.data_ptr(), T,
                                    n_heads, d_plain, rot, int(rot_dims), rank, float(magnitude), _code(q.dtype),
                                    1 if qa.dtype == torch.bfloat16 else 0, _stream()), "latent_q_rope")
     _count("latent_q_rope")
@@ -649,8 +667,9 @@ def _latent_decode_pieces(n_decode: int, head_tiles: int, max_ctx: int, sms: int
     return max(1, -(-max_ctx // keys)), keys
 
 
-def latent_decode_pieces(n_decode: int, n_heads: int, max_ctx: int) -> tuple:
-    return _latent_decode_pieces(int(n_decode), (int(n_heads) + 15) // 16, max(1, int(max_ctx)), num_sms())
+def latent_decode_pieces(n_decode: int, n_heads: int, max_ctx: int, window: int = 0) -> tuple:
+    seen = min(int(max_ctx), int(window)) if window else int(max_ctx)
+    return _latent_decode_pieces(int(n_decode), (int(n_heads) + 15) // 16, max(1, seen), num_sms())
 
 
 def _latent_step_takes_mma(step, dtype, dk: int, rank: int) -> bool:
@@ -670,9 +689,10 @@ def latent_attention_queries_dtype(step, dtype, dk: int, rank: int):
 
 def attention_latent(qa: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, step, group: int, n_heads: int,
                      rank: int, page_size: int, scale: float, sinks: torch.Tensor | None = None,
-                     window: int = 0) -> torch.Tensor:
+                     window: int = 0, gate: torch.Tensor | None = None) -> torch.Tensor:
     """Causal attention of every token of the step over its request's cached latent rows, which all
-    heads share: score = scale * qa[t, h] . row, out[t, h] = sum of softmax weights times row[:rank].
+    heads share: score = scale * qa[t, h] . row, out[t, h] = sum of softmax weights times row[:rank], multiplied by
+    sigmoid(gate[t, h]) where a `gate` is given ([T, nh], a column slice of wider rows in the cache's type).
     `sinks` float32 [nh]: exp(sink_h) joins the denominator of head h and nothing else.  qa float32
     [T, nh dk] (bfloat16 is taken too when the whole step goes to the tensor-core kernels, see
     `latent_attention_queries_dtype`); cache [pages, 1, page_size, dk]; out [T, nh rank] in the cache's type.
@@ -690,13 +710,18 @@ def attention_latent(qa: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, s
     if qa.dtype != latent_attention_queries_dtype(step, cache.dtype, dk, rank) and qa.dtype != torch.float32:
         raise KernelError(f"attention_latent: queries of {qa.dtype} where this step takes float32")
     q16 = 1 if qa.dtype == torch.bfloat16 else 0
+    gp, gs = None, 0
+    if gate is not None:
+        if gate.dtype != cache.dtype or tuple(gate.shape) != (T, n_heads) or gate.stride(1) != 1 or not gate.is_cuda:
+            raise KernelError("attention_latent: the gate must be [T, nh] rows with unit stride in the cache's type")
+        gp, gs = gate.data_ptr(), gate.stride(0)
     tables = step.block_tables[group]
     sink_ptr = sinks.data_ptr() if sinks is not None else None
     n_dec = getattr(step, "n_decode", 0)
     n_tiles = getattr(step, "n_prefill_tiles", 0)
     if _latent_step_takes_mma(step, cache.dtype, dk, rank):
         if n_dec:
-            pieces, keys = latent_decode_pieces(n_dec, n_heads, step.max_decode_ctx)
+            pieces, keys = latent_decode_pieces(n_dec, n_heads, step.max_decode_ctx, window)
             scratch = None
             if pieces > 1:
                 scratch = step.buffer("latent_partial", (n_dec * ((n_heads + 15) // 16) * pieces * 16 * (rank + 2),),
@@ -705,20 +730,20 @@ def attention_latent(qa: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, s
                 qa.data_ptr(), q16, cache.data_ptr(), out.data_ptr(), sink_ptr,
                 scratch.data_ptr() if scratch is not None else None, step.dec_rows.data_ptr(),
                 step.dec_seqs.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1], n_dec,
-                n_heads, dk, rank, page_size, float(scale), int(window), pieces, keys, _stream()),
+                n_heads, dk, rank, page_size, float(scale), int(window), pieces, keys, gp, gs, _stream()),
                 "attention_latent_decode")
             _count("attention_latent.decode.mma" + (".split" if pieces > 1 else ""))
         if n_tiles:
             check(lib().rlis_attention_latent_prefill(
                 qa.data_ptr(), q16, cache.data_ptr(), out.data_ptr(), sink_ptr, step.prefill_tiles.data_ptr(), n_tiles,
                 step.cu_seqlens.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1], n_heads,
-                dk, rank, page_size, float(scale), int(window), _stream()), "attention_latent_prefill")
+                dk, rank, page_size, float(scale), int(window), gp, gs, _stream()), "attention_latent_prefill")
             _count("attention_latent.prefill.mma")
         return out
     check(lib().rlis_attention_latent(qa.data_ptr(), cache.data_ptr(), out.data_ptr(), sink_ptr,
                                       step.seq_of_token.data_ptr(), step.positions.data_ptr(), tables.data_ptr(),
                                       None, tables.shape[1], T, n_heads, dk, rank, page_size, float(scale),
-                                      int(window), _code(cache.dtype), _stream()), "attention_latent")
+                                      int(window), gp, gs, _code(cache.dtype), _stream()), "attention_latent")
     _count("attention_latent")
     return out
 
@@ -863,10 +888,12 @@ class ScaledRows:
     """Rows of a norm's output whose scale is still to be applied: `x` = bf16(resid * weight) [T, dim]
     and `partials` float32 [P, T], the sums of resid^2 over P slices of the width.  The product that
     takes them multiplies its result by 1 / sqrt(sum of a row's partials / dim + eps): the norm
-    between two decode products without a kernel of its own.  Made by `stream_gemm(..., sink=)`."""
+    between two decode products without a kernel of its own.  Made by `stream_gemm(..., sink=)`.
+    Of a layer norm (`weight` given): `sums` [P, T], the sums of resid over the same slices; the product also takes the
+    mean's share off (see `column_sums`)."""
 
-    def __init__(self, x, partials, dim, eps):
-        self.x, self.partials, self.dim, self.eps = x, partials, int(dim), float(eps)
+    def __init__(self, x, partials, dim, eps, sums=None, weight=None):
+        self.x, self.partials, self.dim, self.eps, self.sums, self.weight = x, partials, int(dim), float(eps), sums, weight
 
     shape = property(lambda self: self.x.shape)
     dtype = property(lambda self: self.x.dtype)
@@ -875,11 +902,26 @@ class ScaledRows:
 
 class ResidualSink:
     """Where the last product of a part may put its result itself: added to the float32 residual
-    stream `resid` [T, dim] in place, and handed on as the ScaledRows of the RMSNorm that follows
-    (`weight` float32 [dim], `eps`)."""
+    stream `resid` [T, dim] in place, and handed on as the ScaledRows of the norm that follows
+    (`weight` float32 [dim], `eps`; `centred`: a layer norm, else an RMS norm).  `base`: what the result is added to instead of
+    the stream itself (float32 [T, dim]).  `exact`: the result joins in float32 instead of rounded to bfloat16 first."""
 
-    def __init__(self, resid, weight, eps):
+    def __init__(self, resid, weight, eps, centred: bool = False, base=None, exact: bool = False):
         self.resid, self.weight, self.eps = resid, weight, float(eps)
+        self.centred, self.base, self.exact = bool(centred), base, bool(exact)
+
+
+def column_sums(w: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """float32 [N]: sum_k w[n, k] weight[k], what a row's mean adds to the result of a product with `w` over the rows of a
+    layer norm with `weight`.  Worked out once and kept with the matrix."""
+    kept = w.__dict__.setdefault("_column_sums", {})
+    entry = kept.get(id(weight))
+    if entry is None or entry[0] is not weight:
+        out = torch.empty((w.shape[0],), dtype=torch.float32, device=w.device)
+        for n in range(0, w.shape[0], 8192):
+            out[n:n + 8192] = (w[n:n + 8192].double() @ weight.double()).float()
+        entry = kept[id(weight)] = (weight, out)
+    return entry[1]
 
 
 class StreamsSink:
@@ -901,15 +943,25 @@ def _stream_rows(x: torch.Tensor, name: str) -> int:
     return x.stride(0)
 
 
+class _StreamExtra(ctypes.Structure):
+    """What the streaming product takes beyond its plain arguments (csrc/kernels/stream_gemm_tcgen05.cu: RlisStreamExtra)."""
+    _fields_ = [("in_sums", ctypes.c_void_p), ("colsum", ctypes.c_void_p), ("resid_in", ctypes.c_void_p),
+                ("out_sums", ctypes.c_void_p), ("exact", ctypes.c_int), ("n_plain", ctypes.c_int), ("y2", ctypes.c_void_p),
+                ("gate_cubic", ctypes.c_float), ("x2", ctypes.c_void_p), ("ldx2", ctypes.c_longlong), ("W2", ctypes.c_void_p),
+                ("K2", ctypes.c_int)]
+
+
 def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = False, sink=None, slope: float = 1.0,
-                bias: torch.Tensor | None = None):
+                bias: torch.Tensor | None = None, cubic: float = 0.0, n_plain: int | None = None, second: tuple | None = None):
     """y = x @ w^T (+ bias, float32 [N]) for at most 128 rows of bfloat16 x: the decode step's weight-streaming product on
     the tcgen05 tensor cores (TMA-fed, weights as the M side, k split over CTAs).  x may be a column slice of wider rows.
     `swiglu4`: w is a gate|up matrix interleaved in blocks of 4 rows (bias in the same order) and the result is silu(gate)
-    * up, [M, N / 2]; with a `slope`, gate sigmoid(slope gate) * up (+inf: max(gate, 0) * up).  `x` may be ScaledRows: the
-    rows' scale is applied to the result.  `sink` (up to 16 rows), a ResidualSink: the
-    result, rounded to bfloat16 (+ bias), is added to sink.resid in place and the ScaledRows of the norm that
-    follows are returned instead of y; a StreamsSink: the streams are updated and the normed rows are returned."""
+    * up, [M, N / 2]; with a `slope` (and `cubic`), gate sigmoid(slope (gate + cubic gate^3)) * up (+inf: max(gate, 0) * up).
+    `n_plain` (up to 16 rows): the first n_plain rows of w are an ordinary matrix and the rest such a gate|up matrix; the
+    result is the pair ([M, n_plain], [M, (N - n_plain) / 2]).  `x` may be ScaledRows: the rows' scale (and, of a layer norm,
+    the mean's share) is applied to the result.  `second` = (x2, w2) (up to 16 rows): x2 @ w2^T is added.  `sink` (up to 16
+    rows), a ResidualSink: the result, rounded to bfloat16 (+ bias), is added to sink.resid in place and the ScaledRows of the
+    norm that follows are returned instead of y; a StreamsSink: the streams are updated and the normed rows are returned."""
     scaled = x if isinstance(x, ScaledRows) else None
     if scaled is not None:
         x = scaled.x
@@ -922,8 +974,17 @@ def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = Fa
     if bias is not None:
         _req(bias, "bias", torch.float32, (N,))
     bp = bias.data_ptr() if bias is not None else None
-    if sink is not None and (scaled is not None or swiglu4 or M > DECODE_GEMM_ROWS):
+    if sink is not None and (scaled is not None or swiglu4 or n_plain is not None or M > DECODE_GEMM_ROWS):
         raise KernelError(f"stream_gemm: a sink takes a plain product of up to {DECODE_GEMM_ROWS} unscaled rows")
+    extra = _StreamExtra(gate_cubic=float(cubic))
+    if second is not None:
+        x2, w2 = second
+        if scaled is not None or swiglu4 or n_plain is not None or M > DECODE_GEMM_ROWS or isinstance(sink, StreamsSink):
+            raise KernelError(f"stream_gemm: a second source takes a plain product of up to {DECODE_GEMM_ROWS} unscaled rows")
+        if x2.shape[0] != M or x2.shape[1] % 8:
+            raise KernelError(f"stream_gemm: the second source's rows {tuple(x2.shape)} do not fit {M} rows in vectors of 8")
+        _req(w2, "w2", torch.bfloat16, (N, x2.shape[1]))
+        extra.x2, extra.ldx2, extra.W2, extra.K2 = x2.data_ptr(), _stream_rows(x2, "stream_gemm"), w2.data_ptr(), x2.shape[1]
     if sink is None:
         in_p, n_p, dim, eps = None, 0, 0, 0.0
         if scaled is not None:
@@ -932,12 +993,22 @@ def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = Fa
             if scaled.dim != K:
                 raise KernelError(f"stream_gemm: scaled rows of width {scaled.dim} for a product over {K}")
             in_p, dim, eps = scaled.partials.data_ptr(), scaled.dim, scaled.eps
-        out = torch.empty((M, N // 2 if swiglu4 else N), dtype=out_dtype, device=x.device)
+            if scaled.sums is not None:
+                _req(scaled.sums, "sums", torch.float32, (n_p, M))
+                extra.in_sums, extra.colsum = scaled.sums.data_ptr(), column_sums(w, scaled.weight).data_ptr()
+        epilogue, y2 = 1 if swiglu4 else 0, None
+        out = torch.empty((M, N // 2 if swiglu4 else N if n_plain is None else n_plain), dtype=out_dtype, device=x.device)
+        if n_plain is not None:
+            if n_plain % 8 or N % 8 or not 0 <= n_plain <= N or M > DECODE_GEMM_ROWS or out_dtype != torch.bfloat16 or swiglu4:
+                raise KernelError(f"stream_gemm: {n_plain} plain rows of {N} with {M} rows of x are not taken")
+            epilogue, y2 = 4, torch.empty((M, (N - n_plain) // 2), dtype=torch.bfloat16, device=x.device)
+            extra.n_plain, extra.y2 = int(n_plain), y2.data_ptr()
         check(lib().rlis_stream_gemm_fused(x.data_ptr(), ldx, w.data_ptr(), out.data_ptr(), M, N, K, _code(out_dtype),
-                                           1 if swiglu4 else 0, bp, in_p, n_p, dim, eps, None, None, None, None, float(slope),
-                                           _stream()), "stream_gemm")
-        _count("stream_gemm" + (".scaled" if scaled is not None else "") + (".swiglu" if swiglu4 else ""))
-        return out
+                                           epilogue, bp, in_p, n_p, dim, eps, None, None, None, None, float(slope),
+                                           ctypes.addressof(extra), _stream()), "stream_gemm")
+        _count("stream_gemm" + (".scaled" if scaled is not None else "") + (".centred" if extra.in_sums else "")
+               + (".swiglu" if swiglu4 else ".mixed" if n_plain is not None else "") + (".two" if second is not None else ""))
+        return out if n_plain is None else (out, y2)
     if isinstance(sink, StreamsSink):
         S, nm = sink.n_streams, sink.norm
         _req(sink.x, "sink.x", torch.float32, (M, N) if sink.x.dim() == 2 else (M, S, N))
@@ -957,13 +1028,21 @@ def stream_gemm(x, w: torch.Tensor, out_dtype=torch.bfloat16, swiglu4: bool = Fa
         return h
     _req(sink.resid, "sink.resid", torch.float32, (M, N))
     _req(sink.weight, "sink.weight", torch.float32, (N,))
+    if sink.base is not None:
+        _req(sink.base, "sink.base", torch.float32, (M, N))
     xn = torch.empty((M, N), dtype=torch.bfloat16, device=x.device)
-    partials = torch.empty(((N + 127) // 128, M), dtype=torch.float32, device=x.device)
+    tiles = (N + 127) // 128
+    partials = torch.empty((2 if sink.centred else 1, tiles, M), dtype=torch.float32, device=x.device)
+    extra.resid_in = (sink.base if sink.base is not None else sink.resid).data_ptr()
+    extra.out_sums = partials[1].data_ptr() if sink.centred else None
+    extra.exact = 1 if sink.exact else 0
     check(lib().rlis_stream_gemm_fused(x.data_ptr(), ldx, w.data_ptr(), None, M, N, K, _code(torch.bfloat16), 2, bp, None, 0, 0,
                                        0.0, sink.resid.data_ptr(), sink.weight.data_ptr(), xn.data_ptr(),
-                                       partials.data_ptr(), 1.0, _stream()), "stream_gemm")
-    _count("stream_gemm.sink")
-    return ScaledRows(xn, partials, N, sink.eps)
+                                       partials.data_ptr(), 1.0, ctypes.addressof(extra), _stream()), "stream_gemm")
+    _count("stream_gemm.sink" + (".centred" if sink.centred else "") + (".two" if second is not None else ""))
+    if sink.centred:
+        return ScaledRows(xn, partials[0], N, sink.eps, sums=partials[1], weight=sink.weight)
+    return ScaledRows(xn, partials[0], N, sink.eps)
 
 
 def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu: tuple | None = None,
@@ -971,7 +1050,7 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu:
     """y = x @ w^T on the tcgen05 tensor cores (TMA-fed, accumulator in tensor memory), bfloat16
     operands.  epilogue "plain": bf16 [M, N]; "float32": float32 [M, N]; "swiglu4": w is a gate|up
     matrix interleaved in blocks of 4 rows and the result is silu(gate) * up, bf16 [M, N / 2]; "glu4":
-    the same layout with the gating of `glu` = (slope, limit or None, up_shift), see `glu_act`, after `bias` (float32 [N]
+    the same layout with the gating of `glu` = (slope, limit or None, up_shift[, cubic]), see `glu_act`, after `bias` (float32 [N]
     in the order of w's rows; this epilogue only) is added."""
     M, K = x.shape
     N = w.shape[0]
@@ -989,9 +1068,10 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, epilogue: str = "plain", glu:
     out = torch.empty((M, N // 2 if gated else N), dtype=torch.float32 if code == 2 else torch.bfloat16,
                       device=x.device)
     if code == 3:
-        slope, limit, shift = glu
+        slope, limit, shift, *cubic = glu
         check(lib().rlis_gemm_tcgen05_glu(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, float(slope),
                                           float("inf") if limit is None else float(limit), float(shift),
+                                          float(cubic[0]) if cubic else 0.0,
                                           bias.data_ptr() if bias is not None else None, _stream()), "gemm_tcgen05")
     else:
         check(lib().rlis_gemm_tcgen05(x.data_ptr(), w.data_ptr(), out.data_ptr(), M, N, K, code, _stream()),
@@ -1058,16 +1138,16 @@ def fuses_norms(n_rows: int, dtype, *widths: int) -> bool:
             and all(w % 8 == 0 for w in widths))
 
 
-def linear(x, w: torch.Tensor, out_dtype=None, sink=None, bias: torch.Tensor | None = None):
+def linear(x, w: torch.Tensor, out_dtype=None, sink=None, bias: torch.Tensor | None = None, second: tuple | None = None):
     """y = x @ w^T for w stored (out, in); x may be a column slice of wider rows.  float32: this package's FFMA kernel.
     bfloat16: up to 16 rows go to this package's weight-streaming tcgen05 kernel, more to the library GEMM; both
     accumulate in float32, and `out_dtype=torch.float32` keeps that precision (used for logits).
-    ScaledRows as x and a `sink` (with an optional `bias` of the product) are for the streaming kernel only (see
-    `fuses_norms`)."""
-    if isinstance(x, ScaledRows) or sink is not None:
+    ScaledRows as x, a `sink` (with an optional `bias` of the product) and a `second` source = (x2, w2), whose product is
+    added, are for the streaming kernel only (see `fuses_norms`)."""
+    if isinstance(x, ScaledRows) or sink is not None or second is not None:
         if not fuses_norms(x.shape[0], x.dtype, x.shape[1]):
             raise KernelError("linear: scaled rows or a sink with a product that does not take them")
-        return stream_gemm(x, w, out_dtype or torch.bfloat16, sink=sink, bias=bias)
+        return stream_gemm(x, w, out_dtype or torch.bfloat16, sink=sink, bias=bias, second=second)
     if bias is not None:
         raise KernelError("linear: a bias is taken with a sink")
     if x.dtype == torch.float32:
@@ -1090,6 +1170,18 @@ def linear(x, w: torch.Tensor, out_dtype=None, sink=None, bias: torch.Tensor | N
     if out_dtype is None or out_dtype == torch.bfloat16:
         return torch.mm(x, w.t())
     return torch.mm(x, w.t(), out_dtype=out_dtype)
+
+
+def linear_add(x: torch.Tensor, w: torch.Tensor, base: torch.Tensor) -> torch.Tensor:
+    """base + x @ w^T in float32 (base float32 [T, N]; x and w float32, or bfloat16 with float32 sums): this package's FFMA
+    product and an addition, or the library's product that adds."""
+    T, N = x.shape[0], w.shape[0]
+    _req(base, "base", torch.float32, (T, N))
+    if x.dtype == torch.float32:
+        return sum_norm(gemm_f32(x, w), 1.0, [(base, None, 1.0)], None, 0.0)
+    if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not x.is_cuda:
+        raise KernelError(f"linear_add: expected matching float32 or bfloat16 operands on the device, got {x.dtype}, {w.dtype}")
+    return torch.addmm(base, x, w.t(), out_dtype=torch.float32)
 
 
 def rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Tensor | None,
@@ -1379,8 +1471,8 @@ def attention(q, k_cache, v_cache, out, step, group: int, n_heads: int, n_kv_hea
 
 
 def glu_act(gate_up: torch.Tensor, out: torch.Tensor, slope: float = 1.0, limit: float | None = None,
-            up_shift: float = 0.0, interleave: int = 0, bias: torch.Tensor | None = None) -> torch.Tensor:
-    """out[t, i] = g sigmoid(slope g) (u + up_shift) with g = gate_up[t, i] and u = gate_up[t, I + i], both in
+            up_shift: float = 0.0, interleave: int = 0, bias: torch.Tensor | None = None, cubic: float = 0.0) -> torch.Tensor:
+    """out[t, i] = g sigmoid(slope (g + cubic g^3)) (u + up_shift) with g = gate_up[t, i] and u = gate_up[t, I + i], both in
     float32 (slope +inf: max(g, 0) (u + up_shift)); with a `limit`, g is cut at limit from above and u clipped to [-limit, limit] first.
     interleave B > 0: blocks of B gate columns each followed by their B columns of u.  `bias` (float32 [2 I] in the order
     of gate_up's columns) is added to g and u before anything else."""
@@ -1392,7 +1484,7 @@ def glu_act(gate_up: torch.Tensor, out: torch.Tensor, slope: float = 1.0, limit:
     if bias is not None:
         _req(bias, "bias", torch.float32, (I2,))
     check(lib().rlis_glu_act(gate_up.data_ptr(), out.data_ptr(), T, I2 // 2, float(slope),
-                             float("inf") if limit is None else float(limit), float(up_shift), int(interleave),
+                             float("inf") if limit is None else float(limit), float(up_shift), float(cubic), int(interleave),
                              bias.data_ptr() if bias is not None else None, _code(out.dtype), _stream()), "glu_act")
     _count("glu_act")
     return out
@@ -1402,7 +1494,7 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w, k
                   q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, slots, n_heads: int,
                   n_kv_heads: int, dim: int, v_dim: int, page_size: int, rotation: tuple | None = None,
                   positions: torch.Tensor | None = None, q_temp: tuple | None = None, rot_half: bool = False,
-                  proj_bias: torch.Tensor | None = None) -> torch.Tensor:
+                  proj_bias: torch.Tensor | None = None, maps: int = 1) -> torch.Tensor:
     """From the rows of a stacked projection `proj` [T, N] (queries at column q_off, keys at k_off, values
     at v_off): q_out [T, nh dim] = per-head rmsnorm(q) * q_w, and at `slots` of the paged caches the keys
     rmsnorm(k) * k_w and the values, mixed as (1 - lam) v + lam v_other where `v_other` (a [T, nkv v_dim]
@@ -1414,18 +1506,20 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w, k
     (values are taken as projected, so v_off = k_off caches the unrotated keys as values).  `q_temp` = (coef,
     every): queries are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1) at position p.  Both take
     `positions` (int32 [T]).  `rot_half`: entry i turns with entry i + r / 2 instead of its neighbour.  `proj_bias`
-    (float32 [N]): added to the queries, keys and values as they are read from `proj`."""
+    (float32 [N]): added to the queries, keys and values as they are read from `proj`.  `maps`: every query and key head
+    holds that many vectors of `dim` entries side by side (rotated and normed one by one) over one value; q_out is then
+    [T, nh maps dim] and a cached key row maps dim wide."""
     T, N = proj.shape
     _req(proj, "proj")
-    _req(q_out, "q_out", proj.dtype, (T, n_heads * dim))
+    _req(q_out, "q_out", proj.dtype, (T, n_heads * maps * dim))
     for w, nm in ((q_w, "q_w"), (k_w, "k_w")):
         if w is not None:
             _req(w, nm, torch.float32, (dim,))
-    if v_off + n_kv_heads * v_dim > N or k_off + n_kv_heads * dim > N or q_off + n_heads * dim > N:
+    if v_off + n_kv_heads * v_dim > N or k_off + n_kv_heads * maps * dim > N or q_off + n_heads * maps * dim > N:
         raise KernelError("qk_norm_store: the column offsets reach beyond the projection's rows")
     if slots is not None:
         _req(slots, "slots", torch.int32, (T,))
-        _req(k_cache, "k_cache", proj.dtype, (None, n_kv_heads, page_size, dim))
+        _req(k_cache, "k_cache", proj.dtype, (None, n_kv_heads, page_size, maps * dim))
         _req(v_cache, "v_cache", proj.dtype, (None, n_kv_heads, page_size, v_dim))
     vo, vo_stride = None, 0
     if v_other is not None:
@@ -1451,7 +1545,7 @@ def qk_norm_store(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, q_w, k
                                    slots.data_ptr() if slots is not None else None, T, n_heads, n_kv_heads, dim, v_dim,
                                    page_size, inv_freq.data_ptr() if rot_dims else None, int(rot_dims), float(rot_mag),
                                    positions.data_ptr() if (rot_dims or every) else None, float(coef), int(every),
-                                   1 if rot_half else 0, proj_bias.data_ptr() if proj_bias is not None else None,
+                                   1 if rot_half else 0, proj_bias.data_ptr() if proj_bias is not None else None, int(maps),
                                    _code(proj.dtype), _stream()), "qk_norm_store")
     _count("qk_norm_store" + (".mix" if v_other is not None else "") + (".rot" if rot_dims else ""))
     return q_out
@@ -1582,6 +1676,35 @@ def attention_biased(q, k_cache, v_cache, out, bias, gate, step, group: int, n_h
                                     n_kv_heads, dim, v_dim, page_size, float(scale), int(window), sp, lp, gc,
                                     _code(q.dtype), _stream()), "attention_bias")
     _count("attention_bias")
+    return out
+
+
+def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_heads: int, n_kv_heads: int, dim: int,
+                         v_dim: int, page_size: int, scale: float, cap: float, lam: float, out_scale: float, eps: float,
+                         window: int = 0) -> torch.Tensor:
+    """Causal grouped-query attention of every token of the step with two maps a head: query and key heads hold two vectors
+    of `dim` entries, score = scale * q_m . k_m, then cap * tanh(score / cap) with a `cap` > 0; both maps weigh the same
+    values; o = a_1 - lam a_2 is divided by its root mean square over the v_dim entries (eps under the root), times out_scale
+    and sigmoid(gate[t, head]).  q [T, nh 2 dim]; k_cache [pages, nkv, page_size, 2 dim]; v_cache [pages, nkv, page_size, v_dim];
+    out [T, nh v_dim]; gate [T, nh] (a column slice of wider rows) or None."""
+    T = q.shape[0]
+    _req(q, "q", None, (T, n_heads * 2 * dim))
+    _req(out, "out", q.dtype, (T, n_heads * v_dim))
+    _req(k_cache, "k_cache", q.dtype, (None, n_kv_heads, page_size, 2 * dim))
+    _req(v_cache, "v_cache", q.dtype, (None, n_kv_heads, page_size, v_dim))
+    gp, gs = None, 0
+    if gate is not None:
+        if gate.dtype != q.dtype or tuple(gate.shape) != (T, n_heads) or gate.stride(1) != 1 or not gate.is_cuda:
+            raise KernelError("attention_difference: the gate must be [T, nh] rows with unit stride in q's type")
+        gp, gs = gate.data_ptr(), gate.stride(0)
+    tables = step.block_tables[group]
+    rows, n_rows = None, T
+    check(lib().rlis_attention_difference(
+        q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), gp, gs, step.seq_of_token.data_ptr(),
+        step.positions.data_ptr(), tables.data_ptr(), rows.data_ptr() if rows is not None else None, tables.shape[1], n_rows,
+        n_heads, n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), float(lam), float(out_scale),
+        float(eps), _code(q.dtype), _stream()), "attention_difference")
+    _count("attention_difference")
     return out
 
 

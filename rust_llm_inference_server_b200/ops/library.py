@@ -22,10 +22,11 @@ LL = c_longlong
 # name -> argument types (the stream is always last)
 SIGNATURES = {
     "rlis_embedding": [P, P, P, I, I, I, F, I, P],
-    "rlis_embedding_sink": [P, P, P, P, P, P, I, I, I, F, P],
+    "rlis_embedding_sink": [P, P, P, P, P, P, P, I, I, I, F, P],
     "rlis_logit_transform": [P, I, I, LL, F, F, P],
     "rlis_attention_prefill_tile": [],
-    "rlis_rmsnorm": [P, P, P, P, P, I, I, F, I, P],
+    "rlis_rmsnorm": [P, P, P, P, P, P, I, I, F, I, P],
+    "rlis_layer_norm": [P, P, P, P, P, P, I, I, F, I, P],
     "rlis_swiglu": [P, P, I, I, I, I, P],
     "rlis_gemm_f32_nt": [P, P, P, I, I, I, P],
     "rlis_gemm_f32_nt_batched": [P, P, P, I, I, I, LL, LL, LL, I, LL, LL, LL, P],
@@ -41,21 +42,22 @@ SIGNATURES = {
     "rlis_act_norm": [P, LL, I, P, P, LL, P, LL, I, I, F, I, P],
     "rlis_bias_act": [P, P, P, LL, I, I, I, P],
     "rlis_latent_kv_store": [P, LL, P, P, P, P, P, I, I, I, I, F, F, I, P, P, P, I, P],
-    "rlis_latent_q_rope": [P, P, P, P, I, I, I, I, I, I, F, I, I, P],
-    "rlis_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P],
+    "rlis_latent_q_rope": [P, LL, P, P, P, I, I, I, I, I, I, F, I, I, P],
+    "rlis_attention_latent": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, P, LL, I, P],
     "rlis_attention_latent_mma_takes": [I, I],
-    "rlis_attention_latent_prefill": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, P],
-    "rlis_attention_latent_decode": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
+    "rlis_attention_latent_prefill": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, P, LL, P],
+    "rlis_attention_latent_decode": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P, LL, P],
     "rlis_lightning_scan": [P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, I, P, I, P],
     "rlis_recurrence_inputs": [P, LL, I, I, I, P, I, I, I, I, P, I, P, F, I, P, P, I, P],
     "rlis_recurrence_scan_rows": [P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, P, I, F, P, P, I, P],
     "rlis_recurrence_scan": [P, LL, I, I, I, I, P, P, P, P, P, P, I, I, I, I, I, P],
-    "rlis_qk_norm_store": [P, LL, I, I, I, P, P, F, P, LL, F, P, P, P, P, I, I, I, I, I, I, P, I, F, P, F, I, I, P, I, P],
+    "rlis_qk_norm_store": [P, LL, I, I, I, P, P, F, P, LL, F, P, P, P, P, I, I, I, I, I, I, P, I, F, P, F, I, I, P, I, I, P],
     "rlis_qk_row_norm_store": [P, LL, I, I, I, P, P, F, P, P, P, P, I, I, I, I, I, I, I, P],
     "rlis_attention_bias": [P, P, P, P, P, I, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, I, P, P, I, I, P],
     "rlis_attention_bias_mma_takes": [I, I],
     "rlis_attention_bias_prefill": [P, P, P, P, P, I, P, LL, P, I, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P],
     "rlis_attention_bias_decode": [P, P, P, P, P, P, I, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, I, P],
+    "rlis_attention_difference": [P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, F, F, F, I, P],
     "rlis_moe_route": [P, P, P, P, P, P, I, I, I, I, F, P, I, I, I, I, I, P],
     "rlis_moe_align": [P, P, P, P, I, I, I, I, P],
     "rlis_moe_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, I, P],
@@ -64,7 +66,7 @@ SIGNATURES = {
     "rlis_moe_gemm_mma": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, P],
     "rlis_moe_mma_takes_tile": [I],
     "rlis_moe_combine": [P, P, P, P, P, P, I, I, I, P, P, I, I, P],
-    "rlis_glu_act": [P, P, I, I, F, F, F, I, P, I, P],
+    "rlis_glu_act": [P, P, I, I, F, F, F, F, I, P, I, P],
     "rlis_rope_cache": [P, P, P, P, P, P, P, I, I, I, I, I, I, P],
     "rlis_attention_generic": [P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, P],
     "rlis_attention_decode": [P, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P],
@@ -78,8 +80,8 @@ SIGNATURES = {
     "rlis_sample_filtered": [P, P, P, I, I, LL, P],
     "rlis_nll_rows": [P, P, P, I, I, LL, P],
     "rlis_gemm_tcgen05": [P, P, P, I, I, I, I, P],
-    "rlis_gemm_tcgen05_glu": [P, P, P, I, I, I, F, F, F, P, P],
-    "rlis_stream_gemm_fused": [P, LL, P, P, I, I, I, I, I, P, P, I, I, F, P, P, P, P, F, P],
+    "rlis_gemm_tcgen05_glu": [P, P, P, I, I, I, F, F, F, F, P, P],
+    "rlis_stream_gemm_fused": [P, LL, P, P, I, I, I, I, I, P, P, I, I, F, P, P, P, P, F, P, P],
     "rlis_stream_gemm_streams": [P, LL, P, I, I, I, P, P, LL, LL, I, P, P, P, P, F, P, P, P, P],
     "rlis_take_errors": [P, P],
     "rlis_stream_gemm_timeline": [I],
