@@ -9,8 +9,10 @@ from __future__ import annotations
 import torch
 
 from ..config.model_config import read_config_json
+from .. import ops
 from ..ops import ScaledRows
 from ..config.registry import lookup_architecture
+from ..parts.block import StreamJoin
 from ..parts.base import Part, build_block, build_embedding, build_lm_head, build_norm
 from ..parts.spec import EmbeddingSpec, LMHeadSpec, ModelSpec
 from ..weights.loader import PlacedSource, check_checkpoint
@@ -47,6 +49,17 @@ class Model:
         self.lm_head = build_lm_head(head, dtype, self.device)
         self._tail = _Tail(self.final_norm, self.lm_head)
         self.calls = tuple(spec.order)
+        # what is done to the stream before some calls (equal specs are one part), and everything in the order it runs:
+        # (block, call or None)
+        self.entries = {}
+        self._stations = []
+        for ci, call in enumerate(self.calls):
+            if call.entry is not None:
+                if call.entry not in self.entries:
+                    self.entries[call.entry] = build_block(call.entry, dtype, self.device)
+                self._stations.append((self.entries[call.entry], None))
+            if 0 <= call.layer < len(self.blocks):
+                self._stations.append((self.blocks[call.layer], ci))
         self._plan_caches()
         # parts whose launch configuration depends on more than the step's shape
         self._variant_parts = [p for p in self.parts()
@@ -68,6 +81,8 @@ class Model:
         yield self.embedding
         for blk in self.blocks:
             yield from blk.parts()
+        for entry in self.entries.values():
+            yield from entry.parts()
         yield self.final_norm
         yield self.lm_head
 
@@ -128,7 +143,8 @@ class Model:
         T = step.n_tokens
         resid = step.buffer("resid", (T, self.spec.hidden), torch.float32)
         delta = None
-        first = self.blocks[self.calls[0].layer] if self.calls else None
+        step.carry.clear()
+        first = self._stations[0][0] if self._stations else None
         emb_fuses = getattr(self.embedding, "fuses_norms", None)
         sink = first.entry_sink(resid, step) if (emb_fuses is not None and emb_fuses(step) and
                                                  getattr(first, "chains_norms", False)) else None
@@ -136,15 +152,20 @@ class Model:
             delta = self.embedding.forward(step.token_ids, resid, step, sink=sink)
         else:
             self.embedding.forward(step.token_ids, resid, step)
-        for ci, call in enumerate(self.calls):
-            blk = self.blocks[call.layer]
-            nxt = self.blocks[self.calls[ci + 1].layer] if ci + 1 < len(self.calls) else self._tail
+        if self.entries:
+            if delta is not None and isinstance(first, StreamJoin):
+                step.carry[StreamJoin.EMBEDDED] = delta.x       # the embedding's row, rounded and otherwise as it is
+            else:
+                x0 = step.buffer("embedded", (T, self.spec.hidden), self.dtype)
+                step.carry[StreamJoin.EMBEDDED] = ops.post_norm_residual(None, resid, None, 0.0, out=x0)
+        for si, (blk, ci) in enumerate(self._stations):
+            nxt = self._stations[si + 1][0] if si + 1 < len(self._stations) else self._tail
+            args = (caches[self.calls[ci].cache], states[ci], self.calls[ci].writes_cache) if ci is not None else (None, None, True)
             if getattr(blk, "chains_norms", False) and hasattr(nxt, "entry_sink"):
                 # the block may leave its last addition and the next block's first norm to the products around them
-                resid, delta = blk.forward(resid, delta, step, caches[call.cache], states[ci], call.writes_cache,
-                                           next_block=nxt)
+                resid, delta = blk.forward(resid, delta, step, *args, next_block=nxt)
             else:
-                resid, delta = blk.forward(resid, delta, step, caches[call.cache], states[ci], call.writes_cache)
+                resid, delta = blk.forward(resid, delta, step, *args)
         return resid, delta
 
     def logits(self, resid, delta, step, rows: torch.Tensor):

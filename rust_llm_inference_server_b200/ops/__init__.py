@@ -1708,6 +1708,15 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
     return out
 
 
+def difference_attention_sizes(dtype, dim: int, v_dim: int) -> bool:
+    """Whether the tensor-core kernels for attention of two maps a head exist for these sizes."""
+    return False
+
+
+def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    return False
+
+
 class MoePlan:
     """Where a step's (token, choice) pairs go: the chosen experts and weights, the pairs sorted by expert
     into slots in tiles of `tile` rows, and the shared expert's gate; all on the device."""

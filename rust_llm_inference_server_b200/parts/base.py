@@ -11,6 +11,9 @@ from typing import Callable, Optional
 
 import torch
 
+from .. import ops
+from ..ops.profile import span
+
 
 class TensorSource:
     """What a part loads from: `get(name, role)` returns the tensor on the device.
@@ -119,6 +122,41 @@ class Mixer(Part):
     def forward(self, x: torch.Tensor, step, cache: Optional[LayerCache],
                 state: Optional[torch.Tensor], writes_cache: bool = True) -> torch.Tensor:
         raise NotImplementedError
+
+
+class ProjectedMixer(Mixer):
+    """A mixer that is one product, something over the rows of its result, and one more product: `w_in` [rows, hidden] (rows a
+    multiple of 8), `mix(proj, ...)` -> [T, inner], `w_o` [hidden, inner].  An arrangement whose sublayers stand side by side
+    joins `w_in` and `w_o` with the feed-forward's products and calls `mix` alone (`parts/block.py: ParallelBlock`)."""
+
+    w_in: torch.Tensor
+    w_o: torch.Tensor
+
+    @property
+    def inner(self) -> int:
+        raise NotImplementedError
+
+    def mix(self, proj: torch.Tensor, step, cache, state, writes_cache: bool = True) -> torch.Tensor:
+        raise NotImplementedError
+
+    def fuses_norms(self, step) -> bool:
+        return ops.fuses_norms(step.n_tokens, self.dtype, self.spec.hidden, self.inner)
+
+    def forward(self, x, step, cache, state, writes_cache=True, sink=None):
+        with span("mixer in proj"):
+            proj = ops.linear(x, self.w_in)
+        heads = self.mix(proj, step, cache, state, writes_cache)
+        with span("o proj"):
+            return ops.linear(heads, self.w_o, sink=sink)
+
+
+def stack_rows(parts: list) -> torch.Tensor:
+    """Matrices of equal width one below the other, with zero rows up to a multiple of 8 (16-byte rows of the result)."""
+    w = torch.cat(parts, dim=0)
+    pad = -w.shape[0] % 8
+    if pad:
+        w = torch.cat([w, w.new_zeros((pad, w.shape[1]))], dim=0)
+    return w.contiguous()
 
 
 class FeedForward(Part):

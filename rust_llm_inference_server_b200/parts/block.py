@@ -17,7 +17,7 @@ import torch
 
 from .. import ops
 from ..ops.profile import span
-from .base import (Part, build_feed_forward, build_mixer, build_norm, register_arrangement)
+from .base import (Part, ProjectedMixer, build_feed_forward, build_mixer, build_norm, register_arrangement)
 
 
 class PreNormBlock:
@@ -227,6 +227,133 @@ class PostNormBlock:
         return resid, (StreamRows(h) if chained else None)
 
 
+class ParallelBlock:
+    """h = norm1(x); x += mixer(h) + feed_forward(h), the second term only when the layer has a feed-forward.  The residual
+    stream and the sums are float32: the two results are the block's pending additions (a pair), which the next norm joins.
+
+    In steps of a few rows a block with a `ProjectedMixer` and a gated unit is two products around the mixer and no norm: the
+    mixer's first matrix and gate|up lie in one stacked matrix, whose product applies the norm and gates its second part; the
+    mixer's and the unit's last products are one product with two sources, which adds to the stream and feeds the next norm."""
+
+    chains_norms = True      # `forward` takes `next_block`
+
+    def __init__(self, spec, dtype, device):
+        self.norm1 = build_norm(spec.norm1, dtype, device)
+        self.mixer = build_mixer(spec.mixer, dtype, device)
+        self.feed_forward = build_feed_forward(spec.feed_forward, dtype, device) if spec.feed_forward is not None else None
+        if spec.norm2 is not None:
+            raise ValueError("sublayers side by side have one norm")
+        self.joint = _JointInput(self) if isinstance(self.mixer, ProjectedMixer) and hasattr(self.feed_forward, "w_gate_up") else None
+
+    def parts(self):
+        return tuple(p for p in (self.norm1, self.mixer, self.feed_forward, self.joint) if p is not None)
+
+    def _fuses(self, step) -> bool:
+        if self.feed_forward is None:
+            return self.mixer.fuses_norms(step)
+        return self.joint is not None and self.joint.w is not None and self.mixer.fuses_norms(step) \
+            and self.feed_forward.fuses_norms(step)
+
+    def entry_sink(self, resid, step):
+        return self.norm1.sink(resid, step) if self._fuses(step) else None
+
+    def forward(self, resid, pending, step, cache, state, writes_cache=True, next_block=None):
+        h = pending if isinstance(pending, ops.ScaledRows) else self.norm1.forward(resid, pending, step)
+        fuses = self._fuses(step)
+        sink = next_block.entry_sink(resid, step) if fuses and next_block is not None else None
+        if self.feed_forward is None:
+            if sink is not None:
+                return resid, self.mixer.forward(h, step, cache, state, writes_cache, sink=sink)
+            return resid, self.mixer.forward(h, step, cache, state, writes_cache)
+        if not fuses:
+            return resid, (self.mixer.forward(h, step, cache, state, writes_cache), self.feed_forward.forward(h, step))
+        ff = self.feed_forward
+        with span("mixer in proj, mlp gate+up"):
+            proj, act = ops.stream_gemm(h, self.joint.w, n_plain=self.joint.n_plain, slope=ff.slope, cubic=ff.cubic)
+        heads = self.mixer.mix(proj, step, cache, state, writes_cache)
+        with span("o proj + mlp down proj"):
+            if sink is not None:
+                sink.exact = True            # the two results were never rounded apart
+                return resid, ops.linear(heads, self.mixer.w_o, sink=sink, second=(act, ff.w_down))
+            return resid, (ops.linear(heads, self.mixer.w_o), ops.linear(act, ff.w_down))
+
+
+class _JointInput(Part):
+    """The matrices that read a parallel block's normed input, one below the other: the mixer's, then gate|up.  The two
+    parts keep views of it."""
+
+    graph_safe = True
+
+    def __init__(self, block):
+        self.block = block
+        self.w = None
+
+    def load(self, src) -> None:
+        mixer, ff = self.block.mixer, self.block.feed_forward
+        if mixer.w_in.dtype != torch.bfloat16 or getattr(ff, "interleave", 0) != 4 or ff.b_gate_up is not None or ff.b_down is not None:
+            return
+        self.n_plain = mixer.w_in.shape[0]
+        self.w = torch.cat([mixer.w_in, ff.w_gate_up], dim=0).contiguous()
+        mixer.w_in, ff.w_gate_up = self.w[:self.n_plain], self.w[self.n_plain:]
+
+
+class StreamJoin(Part):
+    """x <- W [x | x0], x0 being the stream as the embedding left it (`step.carry`): what a pass over looped layers starts with.
+    Run between two blocks like a block without a cache.  With W = [W_x | W_0], W_0 x0 is the same on every pass of a step and
+    worked out once; a pass then costs W_x x.  The stream goes into the product rounded to the compute type, its new value is
+    float32.  In steps of a few rows the block before leaves the rounded stream (a sink with a weight of ones), and the product
+    adds W_0 x0 and feeds the first norm of the block after."""
+
+    graph_safe = True
+    chains_norms = True
+
+    EMBEDDED = "stream.embedded"
+
+    def __init__(self, spec, dtype, device):
+        self.spec = spec
+        self.dtype = dtype
+        self.ones = torch.ones((spec.hidden,), dtype=torch.float32, device=device)
+        self.base_key = "stream_join." + spec.weight
+
+    def tensors(self) -> dict:
+        return {self.spec.weight: (self.spec.hidden, 2 * self.spec.hidden)}
+
+    def load(self, src) -> None:
+        w, n = src.get(self.spec.weight), self.spec.hidden
+        self.w_x, self.w_0 = w[:, :n].contiguous(), w[:, n:].contiguous()
+
+    def parts(self):
+        return (self,)
+
+    def fuses_norms(self, step) -> bool:
+        return ops.fuses_norms(step.n_tokens, self.dtype, self.spec.hidden)
+
+    def entry_sink(self, resid, step):
+        return ops.ResidualSink(resid, self.ones, 0.0) if self.fuses_norms(step) else None
+
+    def _stream(self, resid, pending, step):
+        """The complete stream in the compute type."""
+        if isinstance(pending, ops.ScaledRows):
+            return pending.x
+        deltas = pending if isinstance(pending, tuple) else (pending,) if pending is not None else ()
+        h = step.buffer("stream_copy", (resid.shape[0], self.spec.hidden), self.dtype) if self.dtype != torch.float32 else None
+        if deltas or h is not None:
+            ops.sum_norm(resid, 1.0, [(d, None, 1.0) for d in deltas], None, 0.0, out=h)
+        return h if h is not None else resid
+
+    def forward(self, resid, pending, step, cache=None, state=None, writes_cache=True, next_block=None):
+        with span("stream + embedding"):
+            x = self._stream(resid, pending, step)
+            base = step.carry.get(self.base_key)
+            if base is None:
+                base = step.carry[self.base_key] = ops.linear(step.carry[self.EMBEDDED], self.w_0, out_dtype=torch.float32)
+            sink = next_block.entry_sink(resid, step) if self.fuses_norms(step) and next_block is not None else None
+            if isinstance(sink, ops.ResidualSink):
+                sink.base, sink.exact = base, True
+                return resid, ops.linear(x, self.w_x, sink=sink)
+            return ops.linear_add(x, self.w_x, base), None
+
+
 class HyperBlock:
     """Pre-norm sublayers over S residual streams (hyper-connections).  A sublayer reads norm(sum_s read[s] x_s); its
     result y goes back by x_t <- sum_s mix[s, t] x_s + write[t] y, old streams on the right.  The streams are float32: one
@@ -283,7 +410,8 @@ class HyperBlock:
             streams = pending
         else:
             if pending is not None:      # a block of another arrangement has left its last addition
-                ops.stream_mix(resid, 1, y=pending, x_out=resid.unsqueeze(1))
+                for delta in pending if isinstance(pending, tuple) else (pending,):
+                    ops.stream_mix(resid, 1, y=delta, x_out=resid.unsqueeze(1))
             streams = Streams(resid, self.streams)
         ask = getattr(next_block, "entry_streams", None)
         after = ask(step, self.streams) if ask is not None else None
@@ -413,3 +541,5 @@ register_arrangement("sandwich", SandwichBlock)
 register_arrangement("outnorm", OutNormBlock)
 register_arrangement("postnorm", PostNormBlock)
 register_arrangement("hyper", HyperBlock)
+register_arrangement("parallel", ParallelBlock)
+register_arrangement("stream_join", StreamJoin)

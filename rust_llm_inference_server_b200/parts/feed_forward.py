@@ -21,9 +21,10 @@ class SwiGLU(FeedForward):
         self.dtype = dtype
         self.w_gate_up = None
         self.w_down = None
-        # the form g sigmoid(slope g) * u has kernels that gate inside a product (silu at slope 1, relu at an infinite
-        # one); a clipping limit or a shifted linear branch go through the gating kernel that takes them as parameters
+        # the form g sigmoid(slope (g + cubic g^3)) * u has kernels that gate inside a product (silu at slope 1, relu at an
+        # infinite one, gelu in its tanh form); a clipping limit or a shifted linear branch go through the gating kernel that takes them as parameters
         self.slope = float(getattr(spec, "slope", 1.0))
+        self.cubic = float(getattr(spec, "cubic", 0.0))
         self.plain = getattr(spec, "limit", None) is None and float(getattr(spec, "up_shift", 0.0)) == 0.0
         self.b_gate_up = self.b_down = None
         if (getattr(spec, "gate_bias", None) is None) != (getattr(spec, "up_bias", None) is None):
@@ -63,19 +64,19 @@ class SwiGLU(FeedForward):
         T = x.shape[0]
         limit, shift = getattr(s, "limit", None), float(getattr(s, "up_shift", 0.0))
         fusable = self.dtype == torch.bfloat16 and self.interleave == 4 and s.hidden % 8 == 0
-        silu = self.plain and self.slope == 1.0 and self.b_gate_up is None
+        silu = self.plain and self.slope == 1.0 and self.cubic == 0.0 and self.b_gate_up is None
         if fusable and self.plain and T <= ops.STREAM_GEMM_ROWS:
             # product and gating in one kernel
-            return ops.stream_gemm(x, self.w_gate_up, swiglu4=True, slope=self.slope, bias=self.b_gate_up)
+            return ops.stream_gemm(x, self.w_gate_up, swiglu4=True, slope=self.slope, cubic=self.cubic, bias=self.b_gate_up)
         if fusable and T >= 128 and s.intermediate % 128 == 0:
             # prefill: the tcgen05 product with the gating in its epilogue (the gate|up activations never reach HBM)
             return ops.gemm_tcgen05(x, self.w_gate_up, "swiglu4") if silu \
-                else ops.gemm_tcgen05(x, self.w_gate_up, "glu4", glu=(self.slope, limit, shift), bias=self.b_gate_up)
+                else ops.gemm_tcgen05(x, self.w_gate_up, "glu4", glu=(self.slope, limit, shift, self.cubic), bias=self.b_gate_up)
         gu = ops.linear(x, self.w_gate_up)
         act = step.buffer("ffn_act", (T, s.intermediate), self.dtype)
         if silu:
             return ops.swiglu(gu, act, self.interleave)
-        return ops.glu_act(gu, act, self.slope, limit, shift, self.interleave, bias=self.b_gate_up)
+        return ops.glu_act(gu, act, self.slope, limit, shift, self.interleave, bias=self.b_gate_up, cubic=self.cubic)
 
     def forward(self, x, step, sink=None, defer_bias: bool = False):
         """With `defer_bias` the caller adds `self.b_down` itself (in float32, while it joins the result)."""

@@ -8,10 +8,10 @@ import torch
 
 from .. import ops
 from ..ops.profile import span
-from .base import KVCacheSpec, Mixer, build_position, register_mixer
+from .base import KVCacheSpec, ProjectedMixer, build_position, register_mixer, stack_rows
 
 
-class LatentAttention(Mixer):
+class LatentAttention(ProjectedMixer):
     """The key map is folded into the query, so attention runs on the cached rows themselves:
 
         qa[t, h] = [W_uk_h^T q_plain[t, h] | rotate(q_rot[t, h])]        float32
@@ -20,7 +20,9 @@ class LatentAttention(Mixer):
 
     which equals scoring against [W_uk_h c_j | k_rot_j] and summing W_uv_h c_j.  Norms of the two
     latents, the rotation, scores, softmax (with the optional sink term) and value sums are float32.
-    A spec without `kv_down` stores nothing: its call reads the slot another call has filled."""
+    A spec without `kv_down` stores nothing: its call reads the slot another call has filled.  One stacked product makes
+    what reads the mixer's input: the query latent (or, without one, the queries), the key/value latent, the shared key
+    part and the gate logits; a gate is applied to the sum over latents, where that is normalised."""
 
     graph_safe = True
 
@@ -40,13 +42,23 @@ class LatentAttention(Mixer):
         self.scale = float(spec.scale)
         self.window = int(spec.window) if spec.window else 0
         self.own_kv = spec.kv_down is not None
+        if (spec.q_down is None) != (spec.q_norm is None) or (spec.q_down is None) != (spec.q_rank is None):
+            raise ValueError("queries have a latent (its map, norm and rank) or none")
+        self.q_latent = spec.q_down is not None
+        # columns of the stacked product: query latent or queries | kv latent | shared key part | gate logits
+        self.kv_off = spec.q_rank if self.q_latent else spec.n_heads * (spec.dim + spec.rot_dim)
+        self.g_off = self.kv_off + (spec.kv_rank + spec.rot_dim if self.own_kv else 0)
 
     def tensors(self) -> dict:
         s = self.spec
-        out = {s.q_down: (s.q_rank, s.hidden), s.q_norm: (s.q_rank,),
-               s.q_up: (s.n_heads * (s.dim + s.rot_dim), s.q_rank),
+        out = {s.q_up: (s.n_heads * (s.dim + s.rot_dim), s.q_rank if self.q_latent else s.hidden),
                s.k_up: (s.n_heads * s.dim, s.kv_rank), s.v_up: (s.n_heads * s.v_dim, s.kv_rank),
                s.o_proj: (s.hidden, s.n_heads * s.v_dim)}
+        if self.q_latent:
+            out[s.q_down] = (s.q_rank, s.hidden)
+            out[s.q_norm] = (s.q_rank,)
+        if s.head_gate is not None:
+            out[s.head_gate] = (s.n_heads, s.hidden)
         if self.own_kv:
             out[s.kv_down] = (s.kv_rank + s.rot_dim, s.hidden)
             out[s.kv_norm] = (s.kv_rank,)
@@ -56,11 +68,12 @@ class LatentAttention(Mixer):
 
     def load(self, src) -> None:
         s = self.spec
-        down = [src.get(s.q_down)] + ([src.get(s.kv_down)] if self.own_kv else [])
-        self.w_down = torch.cat(down, dim=0).contiguous()          # q latent | kv latent | shared key part
-        self.q_norm = src.get(s.q_norm, "vector")
+        names = [s.q_down if self.q_latent else s.q_up] + ([s.kv_down] if self.own_kv else []) \
+            + ([s.head_gate] if s.head_gate is not None else [])
+        self.w_in = stack_rows([src.get(n) for n in names])
+        self.q_norm = src.get(s.q_norm, "vector") if self.q_latent else None
         self.kv_norm = src.get(s.kv_norm, "vector") if self.own_kv else None
-        self.w_q_up = src.get(s.q_up).contiguous()
+        self.w_q_up = src.get(s.q_up).contiguous() if self.q_latent else None
         # [head, kv_rank, dim]: the key map transposed, so that it applies to queries
         self.w_k_fold = src.get(s.k_up).view(s.n_heads, s.dim, s.kv_rank).transpose(1, 2).contiguous()
         self.w_v_up = src.get(s.v_up).view(s.n_heads, s.v_dim, s.kv_rank).contiguous()
@@ -84,44 +97,50 @@ class LatentAttention(Mixer):
         # decode attention cuts the context into pieces by the longest context of the step
         if not step.n_decode or not self._mma():
             return None
-        return ops.latent_decode_pieces(step.n_decode, self.spec.n_heads, step.max_decode_ctx)
+        return ops.latent_decode_pieces(step.n_decode, self.spec.n_heads, step.max_decode_ctx, self.window)
 
-    def forward(self, x, step, cache, state, writes_cache=True):
+    @property
+    def inner(self) -> int:
+        return self.spec.n_heads * self.spec.v_dim
+
+    def mix(self, proj, step, cache, state, writes_cache=True):
         s = self.spec
-        T, H = x.shape[0], s.n_heads
+        T, H = proj.shape[0], s.n_heads
         dk = s.kv_rank + s.rot_dim
-        with span("latent down proj"):
-            down = ops.linear(x, self.w_down)
-        cq = step.buffer("latent_cq", (T, s.q_rank), self.dtype)
-        if self.own_kv and writes_cache:
+        stores = self.own_kv and writes_cache
+        cq = step.buffer("latent_cq", (T, s.q_rank), self.dtype) if self.q_latent else None
+        if stores:
             # one launch: the kv latent's norm, the shared key part's rotation, the paged write, and the
             # query latent's norm
+            q_args = dict(q_latent=proj[:, :s.q_rank], q_weight=self.q_norm, q_out=cq) if self.q_latent else {}
             with span("latent norms + rope + cache write"):
-                ops.latent_kv_store(down[:, s.q_rank:], self.kv_norm, self.eps, self.inv_freq, self.rot_dims,
+                ops.latent_kv_store(proj[:, self.kv_off:self.kv_off + dk], self.kv_norm, self.eps, self.inv_freq, self.rot_dims,
                                     self.magnitude, step.positions, step.slots[cache.group], cache.k, s.kv_rank,
-                                    cache.page_size, q_latent=down[:, :s.q_rank], q_weight=self.q_norm, q_out=cq)
-        else:
+                                    cache.page_size, **q_args)
+        elif self.q_latent:
             with span("q latent norm"):
-                ops.act_norm(down[:, :s.q_rank], self.q_norm, self.eps, cq)
-        with span("q up proj"):
-            q = ops.linear(cq, self.w_q_up)
+                ops.act_norm(proj[:, :s.q_rank], self.q_norm, self.eps, cq)
+        q = proj[:, :self.kv_off]
+        if self.q_latent:
+            with span("q up proj"):
+                q = ops.linear(cq, self.w_q_up)
         # float32, or bfloat16 when the whole step goes to the tensor-core attention kernels
         qa_dtype = ops.latent_attention_queries_dtype(step, self.dtype, dk, s.kv_rank)
         qa = step.buffer("latent_qa" if qa_dtype == torch.float32 else "latent_qa16", (T, H * dk), qa_dtype)
         with span("q fold + rope"):
-            ops.per_head_linear(q.view(T, H, s.dim + s.rot_dim)[:, :, :s.dim], self.w_k_fold,
+            ops.per_head_linear(q.unflatten(1, (H, s.dim + s.rot_dim))[:, :, :s.dim], self.w_k_fold,
                                 qa.view(T, H, dk)[:, :, :s.kv_rank])
             ops.latent_q_rope(q, qa, self.inv_freq, self.rot_dims, self.magnitude, step.positions, H, s.dim,
                               s.rot_dim, s.kv_rank)
         lat = step.buffer("latent_o", (T, H * s.kv_rank), self.dtype)
+        gate = proj[:, self.g_off:self.g_off + H] if s.head_gate is not None else None
         with span("attention"):
             ops.attention_latent(qa, cache.k, lat, step, cache.group, H, s.kv_rank, cache.page_size, self.scale,
-                                 self.sinks, self.window)
+                                 self.sinks, self.window, gate=gate)
         o = step.buffer("attn_o", (T, H * s.v_dim), self.dtype)
         with span("v up proj"):
             ops.per_head_linear(lat.view(T, H, s.kv_rank), self.w_v_up, o.view(T, H, s.v_dim))
-        with span("o proj"):
-            return ops.linear(o, self.w_o)
+        return o
 
 
 register_mixer("latent_attention", LatentAttention)

@@ -54,6 +54,41 @@ class RMSNorm(Norm):
         return ops.StreamNorm("rmsnorm", self.weight, eps=self.eps)
 
 
+class LayerNorm(Norm):
+    """y = (x - mean) / sqrt(variance + eps) * w, mean and variance of the row in float32, no bias.  (Its weight is `gain`:
+    the arrangements that take an RMS norm apart themselves ask for a `weight`.)"""
+
+    graph_safe = True
+
+    def __init__(self, spec, dtype, device):
+        self.dim = spec.dim
+        self.eps = float(np.float32(spec.eps))
+        self.weight_name = spec.weight
+        self.dtype = dtype
+        self.gain = None
+
+    def tensors(self) -> dict:
+        return {self.weight_name: (self.dim,)}
+
+    def load(self, src) -> None:
+        self.gain = src.get(self.weight_name, "vector").contiguous()
+
+    def forward(self, resid, delta, step):
+        out = step.buffer("norm_out", (resid.shape[0], self.dim), self.dtype)
+        with span("residual add + layer norm"):
+            return ops.layer_norm(resid, self.gain, self.eps, out, delta)
+
+    def forward_rows(self, resid, delta, step, rows):
+        out = step.buffer("norm_rows_out", (rows.shape[0], self.dim), self.dtype)
+        with span("residual add + layer norm"):
+            return ops.layer_norm(resid, self.gain, self.eps, out, delta, rows)
+
+    def sink(self, resid, step):
+        if not ops.fuses_norms(resid.shape[0], self.dtype, self.dim):
+            return None
+        return ops.ResidualSink(resid, self.gain, self.eps, centred=True)
+
+
 class DynamicTanh(Norm):
     """y = tanh(alpha x) * w + b, in float32: no mean and no variance, so nothing of a row has to be known before its
     entries can be written (and a product's epilogue can apply it, see `ops.StreamsSink`)."""
@@ -78,17 +113,28 @@ class DynamicTanh(Norm):
     def stream_norm(self):
         return ops.StreamNorm("dynamic_tanh", self.weight, self.bias, self.alpha)
 
+    @staticmethod
+    def _one(delta, step):
+        """Two additions of a block whose sublayers stand side by side as one."""
+        if not isinstance(delta, tuple):
+            return delta
+        out = step.buffer("delta_sum", tuple(delta[0].shape), delta[0].dtype)
+        return ops.sum_norm(None, 0.0, [(d, None, 1.0) for d in delta], None, 0.0, out=out)
+
     def forward(self, resid, delta, step):
+        delta = self._one(delta, step)
         out = step.buffer("norm_out", (resid.shape[0], self.dim), self.dtype)
         with span("residual add + dynamic tanh"):
             return ops.stream_mix(resid, 1, y=delta, x_out=resid.unsqueeze(1) if delta is not None else None,
                                   norm=self.stream_norm(), h=out)
 
     def forward_rows(self, resid, delta, step, rows):
+        delta = self._one(delta, step)
         out = step.buffer("norm_rows_out", (rows.shape[0], self.dim), self.dtype)
         with span("residual add + dynamic tanh"):
             return ops.stream_mix(resid, 1, y=delta, norm=self.stream_norm(), h=out, rows=rows)
 
 
 register_norm("rmsnorm", RMSNorm)
+register_norm("layer_norm", LayerNorm)
 register_norm("dynamic_tanh", DynamicTanh)

@@ -10,6 +10,7 @@ layers.rs:171-173) and constants (config.rs:5-26).
 
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 from typing import Any, Optional
 
@@ -22,6 +23,15 @@ class RMSNormSpec:
     weight: str                      # tensor name, shape (dim,)
     offset: float = 0.0
     kind: str = "rmsnorm"
+
+
+@dataclass(frozen=True)
+class LayerNormSpec:
+    """y = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w."""
+    dim: int
+    eps: float
+    weight: str                      # tensor name, shape (dim,)
+    kind: str = "layer_norm"
 
 
 @dataclass(frozen=True)
@@ -159,24 +169,55 @@ class BiasedAttentionSpec:
 
 
 @dataclass(frozen=True)
+class DifferenceAttentionSpec:
+    """Causal grouped-query attention with two maps a head over the same values: query head i holds [q_1 | q_2] and key head g
+    [k_1 | k_2], `dim` entries each, all turned by `rotation` (any pairing); score_m = scale * q_m . k_m, then soft_cap *
+    tanh(score / soft_cap) where one is given; a_m = softmax(score_m) V.  With lambda = exp(sum lq1 lk1) - exp(sum lq2 lk2) +
+    offset (`lambdas` names the four vectors of size dim), o = a_1 - lambda a_2 is divided by its root mean square over the
+    head's v_dim entries (eps under the root), times out_scale, times sigmoid of the head's row of `head_gate` applied to the
+    mixer's input (None: no gate); out = W_o o."""
+    hidden: int
+    n_heads: int
+    n_kv_heads: int
+    dim: int
+    v_dim: int
+    scale: float
+    eps: float
+    q_proj: str                      # (n_heads * 2 * dim, hidden), head by head [map 1, map 2]
+    k_proj: str                      # (n_kv_heads * 2 * dim, hidden)
+    v_proj: str                      # (n_kv_heads * v_dim, hidden)
+    o_proj: str                      # (hidden, n_heads * v_dim)
+    lambdas: tuple                   # (lq1, lk1, lq2, lk2)
+    offset: float
+    out_scale: float
+    soft_cap: Optional[float] = None
+    rotation: Any = None
+    window: Optional[int] = None
+    head_gate: Optional[str] = None  # (n_heads, hidden)
+    kind: str = "difference_attention"
+
+
+@dataclass(frozen=True)
 class LatentAttentionSpec:
     """Causal attention whose keys and values are linear maps of a cached latent.  Per token the
     cache holds [c | k_rot]: c = rmsnorm(W_dkv h)[:kv_rank] * kv_norm and the rotated key part
     (`rot_dim` wide, shared by all heads).  Queries: q = W_uq (rmsnorm(W_dq h) * q_norm), per head
     [dim unrotated | rot_dim rotated].  Head h: key = [W_uk_h c | k_rot], value = W_uv_h c, score =
     scale * q . key.  `sink`: a tensor (n_heads,) whose exp joins each head's softmax denominator.
-    `kv_down` None: the layer has no W_dkv and reads the cache slot of another call."""
+    `kv_down` None: the layer has no W_dkv and reads the cache slot of another call.  `q_down` None: queries have no latent,
+    q = W_uq h (q_up is then (n_heads * (dim + rot_dim), hidden); q_rank and q_norm are None).  `head_gate`: head h's output is
+    multiplied by sigmoid of row h applied to the mixer's input."""
     hidden: int
     n_heads: int
     dim: int                         # unrotated query/key entries per head
     rot_dim: int                     # rotated entries per head
     v_dim: int
-    q_rank: int
+    q_rank: Optional[int]
     kv_rank: int
     scale: float
     eps: float
-    q_down: str                      # (q_rank, hidden)
-    q_norm: str                      # (q_rank,)
+    q_down: Optional[str]            # (q_rank, hidden)
+    q_norm: Optional[str]            # (q_rank,)
     q_up: str                        # (n_heads * (dim + rot_dim), q_rank)
     kv_down: Optional[str]           # (kv_rank + rot_dim, hidden)
     kv_norm: Optional[str]           # (kv_rank,)
@@ -186,6 +227,7 @@ class LatentAttentionSpec:
     sink: Optional[str] = None       # (n_heads,)
     position: Any = field(default_factory=NoPositionSpec)
     window: Optional[int] = None
+    head_gate: Optional[str] = None  # (n_heads, hidden)
     kind: str = "latent_attention"
 
 
@@ -354,7 +396,8 @@ class SwiGLUSpec:
     """W_down (g sigmoid(slope g) (u + up_shift)) with g = W_gate h and u = W_up h; with a `limit`, g is
     cut at limit from above and u clipped to [-limit, limit] first.  The defaults are SwiGLU.  A `slope` of
     +infinity is the limit max(g, 0) (u + up_shift): a unit gated by relu.  `gate_bias`, `up_bias` (both or neither) are
-    added to g and u before anything else, `down_bias` to the result."""
+    added to g and u before anything else, `down_bias` to the result.  `cubic`: the gate is g sigmoid(slope (g + cubic g^3));
+    slope 2 sqrt(2 / pi) and cubic 0.044715 are the tanh form of gelu (`GELU_TANH`)."""
     hidden: int
     intermediate: int
     gate_proj: str                   # (intermediate, hidden)
@@ -366,7 +409,12 @@ class SwiGLUSpec:
     gate_bias: Optional[str] = None  # (intermediate,)
     up_bias: Optional[str] = None    # (intermediate,)
     down_bias: Optional[str] = None  # (hidden,)
+    cubic: float = 0.0
     kind: str = "swiglu"
+
+
+# 0.5 z (1 + tanh(u)) is z sigmoid(2 u), so gelu in its tanh form is one of SwiGLUSpec's gates
+GELU_TANH = {"slope": 2.0 * math.sqrt(2.0 / math.pi), "cubic": 0.044715}
 
 
 @dataclass(frozen=True)
@@ -457,7 +505,8 @@ class LayerSpec:
     sum is normed, x = norm1(stream_mult * x + mixer(x)), then x = norm2(stream_mult * x + feed_forward(x)), the
     sublayers reading x itself and the second line only with a feed-forward.  arrangement "hyper": pre-norm sublayers over
     several residual streams, joined as `hyper1` and `hyper2` (HyperSpec) say; the streams start equal, and the layers that
-    follow (or the final norm) read their sum."""
+    follow (or the final norm) read their sum.  arrangement "parallel": one norm, and both sublayers read its output, h =
+    norm1(x), x += mixer(h) + feed_forward(h) (norm2 is None; a layer may have no feed-forward)."""
     norm1: Any
     mixer: Any
     norm2: Any
@@ -474,14 +523,25 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
+class StreamJoinSpec:
+    """A linear map of the residual stream beside the stream as the embedding left it, x <- W [x | x0]: what a pass over a
+    looped stretch of layers may start with (`LayerCall.entry`)."""
+    hidden: int
+    weight: str                      # (hidden, 2 * hidden), x first
+    arrangement: str = "stream_join"
+
+
+@dataclass(frozen=True)
 class LayerCall:
     """One entry of the run order: run `layer` with cache slot `cache`.  A layer may be named by
     several calls (its weights are shared, each call has a cache slot and state of its own unless
     it names another call's slot).  `writes_cache=False`: the call stores nothing and reads the
-    slot that an earlier call of the same step has filled."""
+    slot that an earlier call of the same step has filled.  `entry` (a StreamJoinSpec): what is done to the
+    residual stream right before the layer runs; calls with equal specs share the tensors."""
     layer: int
     cache: int
     writes_cache: bool = True
+    entry: Any = None
 
 
 @dataclass(frozen=True)
