@@ -87,6 +87,18 @@
 // badly), and as two ordinary CTAs that leave their rows in a scratch buffer for the one that takes
 // the tile's last ticket, 57 -> 78 us; at 4096 tokens and more nothing is shared and nothing changes.)
 //
+// Two maps a head (DIFF; the contract of attention_difference.cu): the same kernel at its head size of 128, with one query
+// head a CTA.  A cached key row is [map 1 | map 2], up to 64 entries each, in the two sub-tiles of a row of K; the 128 rows of
+// the instruction are (map 1, tokens 0..63) and (map 2, tokens 0..63), and a row of Q is its map's vector in that map's
+// sub-tile and zeros in the other, so one product over both sub-tiles gives both maps' scores (the zeros double the score
+// product, 8 of a block's 12 k-steps; values, rounds of softmax and the value product are shared, and both maps' outputs end
+// up in one CTA).  Heads narrower than 64 and values narrower than 128 arrive padded with zeros (three-dimensional tensor
+// maps whose innermost extent is the head's).  Scores are capped in registers: cap tanh(s / cap) by an odd polynomial where
+// every score of a warp's chunk is small against the cap (|s / cap| <= 1/4: the error is below 2^-28 of the cap), else by one
+// exponential and one reciprocal.  Capped scores need no running maximum: up to a cap of 64 the exponentials are taken as they
+// are (2^92 fits bfloat16 and the float32 sums with room for the keys), so O is never rescaled.  At the end the warps of map 2
+// leave their rows in shared memory and those of map 1 subtract, norm, gate and store.
+//
 // Every mbarrier wait is bounded (a fifth of a second); a wait that runs out sets the error word
 // (rlis_attention_prefill_tc_error), every role runs to its end without further waits, and the
 // CTA frees its tensor memory before it returns.
@@ -249,13 +261,60 @@ __device__ __forceinline__ void store_row(uint32_t tmem_row, float inv, bool pre
 // take, and the rescaling of O in tensor memory becomes rare after the first blocks.
 constexpr float RESCALE_AFTER = 8.0f;
 
-template <int HD, int TN>
+// What two maps a head need beyond the rest (see attention_difference.cu).
+struct DiffArgs {
+    const bf16* gate;
+    long long gate_stride;
+    float cap, lambda, out_scale, eps;
+    int dv;
+};
+constexpr float FIXED_REFERENCE_CAP = 64.0f;    // capped scores up to here are exponentiated as they are
+
+__device__ __forceinline__ void tma_load_3d(void* dst, const CUtensorMap* map, int x, int y, int z, uint64_t* bar) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+        ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z)
+        : "memory");
+}
+
+// s <- log2(e) cap tanh(s scale / cap) of 32 scores.
+__device__ __forceinline__ void cap_of_chunk(uint32_t (&v)[32], float scale, float cap) {
+    constexpr float LOG2E = 1.4426950408889634f;
+    const float k = scale / cap;
+    float most[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < 32; i += 8)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+            most[j] = max3(most[j], fabsf(__uint_as_float(v[i + 2 * j])), fabsf(__uint_as_float(v[i + 2 * j + 1])));
+    const bool small = max3(most[0], most[1], fmaxf(most[2], most[3])) * fabsf(k) <= 0.25f;
+    if (__all_sync(0xffffffffu, small)) {
+        // tanh(u) = u (1 - u^2/3 + 2 u^4/15 - 17 u^6/315 + 62 u^8/2835 - ...): the next term is below 2^-28 here
+        const float kk = k * k, top = scale * LOG2E;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+            const float s = __uint_as_float(v[i]), u2 = s * s * kk;
+            const float p = fmaf(u2, fmaf(u2, fmaf(u2, fmaf(u2, 62.f / 2835.f, -17.f / 315.f), 2.f / 15.f), -1.f / 3.f), 1.f);
+            v[i] = __float_as_uint(s * top * p);
+        }
+    } else {
+        const float e2 = 2.0f * LOG2E * k, top = cap * LOG2E;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+            const float e = ex2_approx(__uint_as_float(v[i]) * e2);            // e^{2u}: tanh(u) = 1 - 2 / (1 + e^{2u})
+            v[i] = __float_as_uint(fmaf(-2.0f * top, __fdividef(1.0f, 1.0f + fminf(e, 1e30f)), top));
+        }
+    }
+}
+
+template <int HD, int TN, bool DIFF = false>
 __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
     const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
     const __grid_constant__ CUtensorMap map_v, bf16* __restrict__ out, const int* __restrict__ tiles,
     const int* __restrict__ cu_seqlens, const int* __restrict__ ctx_lens,
     const int* __restrict__ block_tables, int max_blocks, int nh, int nkv, int page_size,
-    int cache_rows, float scale, int window, int splits) {
+    int cache_rows, float scale, int window, int splits, const DiffArgs diff) {
+    static_assert(!DIFF || (HD == 128 && TN == 64), "two maps of 64 are a row of 128");
     extern __shared__ __align__(1024) unsigned char pt_smem_raw[];
     if ((smem_u32(pt_smem_raw) & 1023u) != 0u) {       // the swizzled tiles need it; never seen, but checked
         if (threadIdx.x == 0) atomicExch(&g_tc_error, 2);
@@ -275,11 +334,11 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
     // The query heads of a kv head go in pairs; with an odd number the last pair holds its one head
     // twice, and the copy's rows are not stored.
     const int b = tiles[2 * blockIdx.y], t0 = tiles[2 * blockIdx.y + 1];
-    const int pairs = (nrep + 1) / 2;
+    const int pairs = DIFF ? nrep : (nrep + 1) / 2;
     const int pidx = blockIdx.x / splits;
     const int kvh = pidx / pairs;
-    const int head0 = kvh * nrep + (pidx % pairs) * 2;
-    const bool two = (pidx % pairs) * 2 + 1 < nrep;
+    const int head0 = DIFF ? pidx : kvh * nrep + (pidx % pairs) * 2;
+    const bool two = !DIFF && (pidx % pairs) * 2 + 1 < nrep;
     const int head1 = two ? head0 + 1 : head0;
     const int rank = blockIdx.x % splits;                    // of this CTA in its cluster: it takes blocks rank, rank + splits, ...
     const int q_start = cu_seqlens[b];
@@ -341,6 +400,12 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
             bar_expect_tx(&ctrl->q_full, Q_BYTES);
 #pragma unroll
             for (int hf = 0; hf < HALVES; ++hf) {        // sub-tile hf: rows 0..63 head 0, rows 64..127 head 1
+                if constexpr (DIFF) {                    // ... map 1 and map 2; a map's rows are zeros in the other's sub-tile
+                    tma_load_3d(q_tile + hf * LINE_TILE, &map_q, 0, hf == 0 ? 2 * head0 : 2 * nh, q_start + t0, &ctrl->q_full);
+                    tma_load_3d(q_tile + hf * LINE_TILE + LINE_TILE / 2, &map_q, 0, hf == 1 ? 2 * head0 + 1 : 2 * nh, q_start + t0,
+                                &ctrl->q_full);
+                    continue;
+                }
                 tma_load_2d(q_tile + hf * LINE_TILE, &map_q, head0 * HD + hf * 64, q_start + t0, &ctrl->q_full);
                 tma_load_2d(q_tile + hf * LINE_TILE + LINE_TILE / 2, &map_q, head1 * HD + hf * 64, q_start + t0,
                             &ctrl->q_full);
@@ -365,7 +430,9 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
                 // (it may have been given back): a coordinate past the end of the tensor, zeros arrive
                 const bool wanted = key < ctx && (window <= 0 || key + page_size > pos0 - window + 1);
                 const int row = wanted ? (table[key / page_size] * nkv + kvh) * page_size : cache_rows;
-                tma_load_2d(tile + (size_t)hf * KV_LINE_TILE + (size_t)pg * page_bytes, is_v ? &map_v : &map_k, hf * 64, row, full);
+                unsigned char* dst = tile + (size_t)hf * KV_LINE_TILE + (size_t)pg * page_bytes;
+                if (DIFF && !is_v) tma_load_3d(dst, &map_k, 0, hf, row, full);
+                else tma_load_2d(dst, is_v ? &map_v : &map_k, hf * 64, row, full);
             }
             __syncwarp();
             return true;
@@ -456,7 +523,8 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
         const int pos = pos0 + (srow & 63);
         const int lo = window > 0 ? max(0, pos - window + 1) : 0;
         const uint32_t lane_addr = slane_addr;
-        const float scale_log2 = scale * 1.4426950408889634f;
+        const bool capped = DIFF && diff.cap > 0.f, fixed_ref = capped && diff.cap <= FIXED_REFERENCE_CAP;
+        const float scale_log2 = capped ? 1.0f : scale * 1.4426950408889634f;      // (capping leaves scores in units of log2(e))
         const uint32_t tmem_p_row = tmem_p + lane_addr;
         bool ok = true;
         for (int it = 0; it < n_blk; ++it) {
@@ -479,7 +547,15 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
             const bool need_mask = key0 + TN - 1 > pos0 || window > 0;
             const int kmax = pos - key0, kmin = lo - key0;           // visible: kmin <= index <= kmax
             float mx = -INFINITY;
-            if (need_mask) {
+            if constexpr (DIFF) {
+                if (capped) {
+                    cap_of_chunk(s0, scale, diff.cap);
+                    cap_of_chunk(s1, scale, diff.cap);
+                }
+            }
+            if (DIFF && fixed_ref) {
+                mx = 0.f;
+            } else if (need_mask) {
                 max_of_chunk<true>(s0, 0, kmin, kmax, mx);
                 max_of_chunk<true>(s1, 1, kmin, kmax, mx);
                 if constexpr (TN > 64) {
@@ -578,7 +654,58 @@ __global__ __launch_bounds__(PT_THREADS, 2) void attn_prefill_tc_kernel(
         // the row's place in the output: head (srow / 64) of the pair, token (srow % 64) of the tile
         const bool srow_valid = (srow & 63) < n_valid && (srow < 64 || two);
         bf16* sorow = out + ((size_t)(q_start + t0 + (srow & 63)) * nh + (srow < 64 ? head0 : head1)) * HD;
-        if (splits == 1) {
+        if constexpr (DIFF) {
+            // map 2's rows meet map 1's in shared memory (every product and copy is done: the tiles are free)
+            constexpr int RF = HD + 4;
+            float* xrow = reinterpret_cast<float*>(pt_smem_raw) + (size_t)(srow & 63) * RF;
+            const float inv = row_ok ? (srow < 64 ? 1.0f : diff.lambda) / l_run : __int_as_float(0x7fc00000);
+            if (srow >= 64) {
+#pragma unroll 1
+                for (int c = 0; c < HD / 32; ++c) {
+                    uint32_t v[32];
+                    tmem_ld32(tmem_o + slane_addr + (uint32_t)(c * 32), v);
+#pragma unroll
+                    for (int i = 0; i < 32; i += 4)
+                        *reinterpret_cast<float4*>(xrow + c * 32 + i) =
+                            make_float4(__uint_as_float(v[i]) * inv, __uint_as_float(v[i + 1]) * inv, __uint_as_float(v[i + 2]) * inv,
+                                        __uint_as_float(v[i + 3]) * inv);
+                }
+            }
+            asm volatile("bar.sync 1, 128;" ::: "memory");
+            if (srow < 64) {
+                float ss = 0.f;
+#pragma unroll 1
+                for (int c = 0; c < HD / 32; ++c) {
+                    uint32_t v[32];
+                    tmem_ld32(tmem_o + slane_addr + (uint32_t)(c * 32), v);
+#pragma unroll
+                    for (int i = 0; i < 32; i += 4) {
+                        float4 b = *reinterpret_cast<const float4*>(xrow + c * 32 + i);
+                        b.x = fmaf(__uint_as_float(v[i]), inv, -b.x);
+                        b.y = fmaf(__uint_as_float(v[i + 1]), inv, -b.y);
+                        b.z = fmaf(__uint_as_float(v[i + 2]), inv, -b.z);
+                        b.w = fmaf(__uint_as_float(v[i + 3]), inv, -b.w);
+                        ss += (b.x * b.x + b.y * b.y) + (b.z * b.z + b.w * b.w);     // (columns past dv are zeros)
+                        *reinterpret_cast<float4*>(xrow + c * 32 + i) = b;
+                    }
+                }
+                if (srow < n_valid && n_blk > 0) {
+                    const size_t tok = (size_t)(q_start + t0 + srow);
+                    float f = diff.out_scale / sqrtf(ss / (float)diff.dv + diff.eps);
+                    if (diff.gate != nullptr) f /= 1.0f + expf(-__bfloat162float(diff.gate[tok * diff.gate_stride + head0]));
+                    bf16* orow = out + (tok * nh + head0) * diff.dv;
+                    for (int c = 0; c < diff.dv; c += 8) {
+                        const float4 a = *reinterpret_cast<const float4*>(xrow + c), b = *reinterpret_cast<const float4*>(xrow + c + 4);
+                        uint4 pk;
+                        pk.x = pack_bf16(a.x * f, a.y * f);
+                        pk.y = pack_bf16(a.z * f, a.w * f);
+                        pk.z = pack_bf16(b.x * f, b.y * f);
+                        pk.w = pack_bf16(b.z * f, b.w * f);
+                        *reinterpret_cast<uint4*>(orow + c) = pk;
+                    }
+                }
+            }
+        } else if (splits == 1) {
             if (n_blk > 0) store_row<HD>(tmem_o + slane_addr, 1.0f / l_run, row_ok && srow_valid, sorow);
         } else {
             // The CTAs of the cluster took the blocks of keys in turn.  Once all their products are done
@@ -725,7 +852,7 @@ int launch_prefill_tc(const CUtensorMap& map_q, const CUtensorMap& map_k, const 
     if (splits != 1 && splits != 2 && splits != 4) return RLIS_ERR_UNSUPPORTED;
     rlis_launch_cluster(attn_prefill_tc_kernel<HD, TN>, dim3((unsigned)(pairs * splits), (unsigned)n_tiles), PT_THREADS,
                         SH::SMEM, stream, dim3((unsigned)splits, 1, 1), map_q, map_k, map_v, out, tiles, cu_seqlens,
-                        ctx_lens, block_tables, max_blocks, nh, nkv, page_size, cache_rows, scale, window, splits);
+                        ctx_lens, block_tables, max_blocks, nh, nkv, page_size, cache_rows, scale, window, splits, DiffArgs{});
     return RLIS_LAUNCH_CHECK();
 }
 }  // namespace
@@ -756,4 +883,55 @@ extern "C" int rlis_attention_prefill_tc(const void* q, const void* k_cache, con
                                           max_blocks, nh, nkv, page_size, (int)cache_rows, scale, window, max_ctx, stream);
     return launch_prefill_tc<128, 64>(map_q, map_k, map_v, (bf16*)out, tiles, n_tiles, cu_seqlens, ctx_lens, block_tables,
                                       max_blocks, nh, nkv, page_size, (int)cache_rows, scale, window, max_ctx, stream);
+}
+
+// Whether the tensor-core kernel takes two maps a head of these sizes (else the caller uses rlis_attention_difference).
+extern "C" int rlis_attention_difference_prefill_takes(int d, int dv, int page_size) {
+    return d > 0 && d <= 64 && d % 8 == 0 && dv > 0 && dv <= 128 && dv % 8 == 0 && page_size >= 8 && page_size <= 64 &&
+           64 % page_size == 0;
+}
+
+// A [rows, mid, cols] bf16 row-major tensor with boxes of 64 columns (zeros past `cols`) x 1 x box_rows.
+static bool make_map_3d(CUtensorMap* map, const void* ptr, long long rows, int mid, int cols, int box_rows) {
+    EncodeTiledFn fn = encode_fn();
+    if (fn == nullptr) return false;
+    const cuuint64_t dims[3] = {(cuuint64_t)cols, (cuuint64_t)mid, (cuuint64_t)rows};
+    const cuuint64_t strides[2] = {(cuuint64_t)cols * 2, (cuuint64_t)cols * mid * 2};
+    const cuuint32_t box[3] = {64u, 1u, (cuuint32_t)box_rows};
+    const cuuint32_t estr[3] = {1, 1, 1};
+    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+              CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+              CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
+// q [tokens, nh, 2 d]; k_cache [pages, nkv, page_size, 2 d]; v_cache [pages, nkv, page_size, dv]; out [tokens, nh dv];
+// gate (null: none): logits, head h of token t at gate[t * gate_stride + h]; tiles as for rlis_attention_prefill_tc.
+extern "C" int rlis_attention_difference_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const void* gate,
+                                                 long long gate_stride, const int* tiles, int n_tiles, const int* cu_seqlens,
+                                                 const int* ctx_lens, const int* block_tables, int max_blocks, int n_tokens,
+                                                 int n_pages, int nh, int nkv, int d, int dv, int page_size, float scale, float cap,
+                                                 int window, float lambda, float out_scale, float eps, cudaStream_t stream) {
+    if (n_tiles <= 0) return 0;
+    if (!rlis_attention_difference_prefill_takes(d, dv, page_size) || nkv <= 0 || nh % nkv != 0 || n_tiles > 65535 || cap < 0.f)
+        return RLIS_ERR_UNSUPPORTED;
+    if (((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache) |
+          reinterpret_cast<uintptr_t>(out)) & 15) != 0)
+        return RLIS_ERR_UNSUPPORTED;
+    const long long cache_rows = (long long)n_pages * nkv * page_size;
+    if (cache_rows >= (1ll << 31)) return RLIS_ERR_UNSUPPORTED;
+    CUtensorMap map_q, map_k, map_v;
+    if (!make_map_3d(&map_q, q, n_tokens, 2 * nh, d, TQ) || !make_map_3d(&map_k, k_cache, cache_rows, 2, d, page_size) ||
+        !make_map_2d(&map_v, v_cache, cache_rows, dv, page_size))
+        return RLIS_ERR_UNSUPPORTED;
+    using SH = PShape<128, 64>;
+    static bool attr_done = false;
+    if (!attr_done) {
+        cudaFuncSetAttribute(attn_prefill_tc_kernel<128, 64, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SH::SMEM);
+        attr_done = true;
+    }
+    const DiffArgs da{(const bf16*)gate, gate_stride, cap, lambda, out_scale, eps, dv};
+    rlis_launch_cluster(attn_prefill_tc_kernel<128, 64, true>, dim3((unsigned)nh, (unsigned)n_tiles), PT_THREADS, SH::SMEM, stream,
+                        dim3(1, 1, 1), map_q, map_k, map_v, (bf16*)out, tiles, cu_seqlens, ctx_lens, block_tables, max_blocks, nh, nkv,
+                        page_size, (int)cache_rows, scale, window, 1, da);
+    return RLIS_LAUNCH_CHECK();
 }
