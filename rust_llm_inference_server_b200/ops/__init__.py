@@ -1393,7 +1393,7 @@ def _set_stream_rows(value):
 
 library.PYTHON_SWITCHES.update(biased_mma=_set_flag("BIASED_MMA"), moe_mma=_set_flag("MOE_MMA"),
                                moe_grouped=_set_flag("MOE_GROUPED"), fuse_norms=_set_flag("FUSE_NORMS"), prefill_tcgen05=_set_flag("PREFILL_TCGEN05"),
-                               latent_mma=_set_flag("LATENT_MMA"), latent_ctas_per_sm=_set_latent_ctas,
+                               latent_mma=_set_flag("LATENT_MMA"), difference_mma=_set_flag("DIFFERENCE_MMA"), latent_ctas_per_sm=_set_latent_ctas,
                                stream_rows=_set_stream_rows)
 
 
@@ -1679,6 +1679,34 @@ def attention_biased(q, k_cache, v_cache, out, bias, gate, step, group: int, n_h
     return out
 
 
+DIFFERENCE_MMA = True      # debug switch "difference_mma": 0 takes the one-warp-a-row kernel for every size
+
+
+@functools.lru_cache(maxsize=None)
+def _difference_prefill_sizes(dim: int, v_dim: int, page_size: int) -> bool:
+    return bool(lib().rlis_attention_difference_prefill_takes(dim, v_dim, page_size))
+
+
+@functools.lru_cache(maxsize=None)
+def _difference_decode_sizes(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    return bool(lib().rlis_attention_difference_decode_takes(n_heads, n_kv_heads, dim, v_dim))
+
+
+def difference_prefill_takes_mma(dtype, dim: int, v_dim: int, page_size: int = 16) -> bool:
+    """Whether the tensor-core kernel for prompts with two maps a head exists for these sizes."""
+    return bool(DIFFERENCE_MMA and dtype == torch.bfloat16 and _difference_prefill_sizes(int(dim), int(v_dim), int(page_size)))
+
+
+def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+    """The same for single tokens."""
+    return bool(DIFFERENCE_MMA and dtype == torch.bfloat16
+                and _difference_decode_sizes(int(n_heads), int(n_kv_heads), int(dim), int(v_dim)))
+
+
+def difference_decode_pieces(n_decode: int, n_kv_heads: int, max_ctx: int, window: int = 0) -> int:
+    return biased_decode_pieces(n_decode, n_kv_heads, min(int(max_ctx), int(window)) if window else max_ctx)
+
+
 def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_heads: int, n_kv_heads: int, dim: int,
                          v_dim: int, page_size: int, scale: float, cap: float, lam: float, out_scale: float, eps: float,
                          window: int = 0) -> torch.Tensor:
@@ -1686,7 +1714,11 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
     of `dim` entries, score = scale * q_m . k_m, then cap * tanh(score / cap) with a `cap` > 0; both maps weigh the same
     values; o = a_1 - lam a_2 is divided by its root mean square over the v_dim entries (eps under the root), times out_scale
     and sigmoid(gate[t, head]).  q [T, nh 2 dim]; k_cache [pages, nkv, page_size, 2 dim]; v_cache [pages, nkv, page_size, v_dim];
-    out [T, nh v_dim]; gate [T, nh] (a column slice of wider rows) or None."""
+    out [T, nh v_dim]; gate [T, nh] (a column slice of wider rows) or None.
+
+    bfloat16 with sizes the tensor-core kernels take: single decoded tokens go to the split decode kernel (groups of up to 8
+    query heads), portions of prompts (the step's tile list) to the tcgen05 flash kernel.  Everything else, and all of float32,
+    to the kernel that takes one warp a (token, head)."""
     T = q.shape[0]
     _req(q, "q", None, (T, n_heads * 2 * dim))
     _req(out, "out", q.dtype, (T, n_heads * v_dim))
@@ -1698,7 +1730,33 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
             raise KernelError("attention_difference: the gate must be [T, nh] rows with unit stride in q's type")
         gp, gs = gate.data_ptr(), gate.stride(0)
     tables = step.block_tables[group]
+    n_dec = step.n_decode if difference_decode_takes_mma(q.dtype, n_heads, n_kv_heads, dim, v_dim) else 0
+    n_tiles = step.n_prefill_tiles if difference_prefill_takes_mma(q.dtype, dim, v_dim, page_size) else 0
+    if n_dec:
+        pieces = difference_decode_pieces(n_dec, n_kv_heads, step.max_decode_ctx, window)
+        scratch = step.buffer("attn_partial", (n_dec * n_heads * 2 * pieces * (lib().rlis_attention_difference_decode_width(v_dim) + 2),),
+                              torch.float32) if pieces > 1 else None
+        check(lib().rlis_attention_difference_decode(
+            q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), scratch.data_ptr() if scratch is not None else None,
+            gp, gs, step.dec_rows.data_ptr(), step.dec_seqs.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1],
+            n_dec, n_heads, n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), pieces, float(lam),
+            float(out_scale), float(eps), _stream()), "attention_difference_decode")
+        _count("attention_difference.decode.mma" + (".split" if pieces > 1 else ""))
+    if n_tiles:
+        check(lib().rlis_attention_difference_prefill(
+            q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), gp, gs, step.prefill_tiles.data_ptr(), n_tiles,
+            step.cu_seqlens.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1], T, k_cache.shape[0], n_heads,
+            n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), float(lam), float(out_scale), float(eps),
+            _stream()), "attention_difference_prefill")
+        _count("attention_difference.prefill.tcgen05")
+    # what the tensor-core kernels did not take: nothing, the portions only, the single tokens only, or everything
     rows, n_rows = None, T
+    if n_dec and (n_tiles or step.n_prefill_tokens == 0) or n_tiles and step.n_decode == 0:
+        return out
+    if n_dec:
+        rows, n_rows = step.prefill_rows, step.n_prefill_tokens
+    elif n_tiles:
+        rows, n_rows = step.dec_rows, step.n_decode
     check(lib().rlis_attention_difference(
         q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), gp, gs, step.seq_of_token.data_ptr(),
         step.positions.data_ptr(), tables.data_ptr(), rows.data_ptr() if rows is not None else None, tables.shape[1], n_rows,
@@ -1706,15 +1764,6 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
         float(eps), _code(q.dtype), _stream()), "attention_difference")
     _count("attention_difference")
     return out
-
-
-def difference_attention_sizes(dtype, dim: int, v_dim: int) -> bool:
-    """Whether the tensor-core kernels for attention of two maps a head exist for these sizes."""
-    return False
-
-
-def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
-    return False
 
 
 class MoePlan:

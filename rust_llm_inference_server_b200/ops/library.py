@@ -58,6 +58,11 @@ SIGNATURES = {
     "rlis_attention_bias_prefill": [P, P, P, P, P, I, P, LL, P, I, P, P, P, I, I, I, I, I, I, F, I, P, P, I, P],
     "rlis_attention_bias_decode": [P, P, P, P, P, P, I, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, I, I, P, P, I, P],
     "rlis_attention_difference": [P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, F, F, F, I, P],
+    "rlis_attention_difference_prefill": [P, P, P, P, P, LL, P, I, P, P, P, I, I, I, I, I, I, I, I, F, F, I, F, F, F, P],
+    "rlis_attention_difference_prefill_takes": [I, I, I],
+    "rlis_attention_difference_decode": [P, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, F, F, F, P],
+    "rlis_attention_difference_decode_takes": [I, I, I, I],
+    "rlis_attention_difference_decode_width": [I],
     "rlis_moe_route": [P, P, P, P, P, P, I, I, I, I, F, P, I, I, I, I, I, P],
     "rlis_moe_align": [P, P, P, P, I, I, I, I, P],
     "rlis_moe_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, I, P],

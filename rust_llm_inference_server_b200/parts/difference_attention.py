@@ -73,7 +73,7 @@ class DifferenceAttention(ProjectedMixer):
 
     @property
     def prefill_tile(self):
-        return ops.prefill_tile() if ops.difference_attention_sizes(self.dtype, self.spec.dim, self.spec.v_dim) else None
+        return ops.prefill_tile() if ops.difference_prefill_takes_mma(self.dtype, self.spec.dim, self.spec.v_dim) else None
 
     def launch_variant(self, step):
         s = self.spec
