@@ -199,3 +199,309 @@ def test_two_vectors_a_head_are_turned_and_stored_as_one_row(dtype, H, G, d, dv,
         np.testing.assert_allclose(host(vc[pg, :, at]), x[t, v_off:v_off + G * dv].reshape(G, dv), rtol=0, atol=0)
     for c in (kc, vc):
         assert float((c.float().permute(0, 2, 1, 3)[~torch.from_numpy(touched).cuda()] - 7.0).abs().max()) == 0.0
+
+
+DIFF_SHAPES = [(4, 2, 32, 16, 8), (3, 3, 24, 8, 16), (1, 1, 8, 24, 16), (6, 2, 64, 128, 16), (8, 1, 64, 64, 32), (16, 2, 48, 96, 64),
+               (10, 1, 40, 72, 16), (2, 1, 72, 136, 16), (5, 5, 20, 12, 16), (2, 2, 56, 120, 8)]
+
+
+def plain_difference_rows(q, keys, vals, scale, cap, window, lam, diff, eps, gate, st, H, G):
+    T = q.shape[0]
+    out = np.zeros((T, H, vals[0].shape[-1]))
+    for t in range(T):
+        b, pos = st.host_seq[t], st.host_pos[t]
+        lo = max(0, pos - window + 1) if window else 0
+        for h in range(H):
+            g = h // (H // G)
+            a = []
+            for m in (0, 1):
+                s = keys[b][lo:pos + 1, g, m] @ q[t, h, m] * scale
+                a.append(P.softmax(P.capped(s, cap) if cap else s) @ vals[b][lo:pos + 1, g])
+            out[t, h] = P.difference_of_maps(a[0], a[1], lam, diff, eps)
+    return out * P.sigmoid(gate)[:, :, None]
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, BF16])
+@pytest.mark.parametrize("cap,window", [(50.0, 0), (9.0, 0), (90.0, 0), (0.0, 0), (40.0, 70), (0.0, 33)])
+@pytest.mark.parametrize("H,G,d,dv,page", DIFF_SHAPES)
+def test_attention_of_two_maps_far_keys_page_borders_and_windows(dtype, H, G, d, dv, page, cap, window):
+    """Whole prompts, portions that start in the middle of a page, and single tokens in one launch.  Per head and map one key
+    is made to carry the weight (query and key scaled): the first token, a page's last and first slot, a key far back, the
+    token itself, and with a window the keys just inside and just outside its edge."""
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(H * 100 + d)
+    ctx, qn = [150, 70, 129, 1, 2, 900, 65, 420], [150, 1, 37, 1, 2, 1, 64, 1]
+    n_pages = sum(-(-c // page) for c in ctx) + 3
+    st = hand_step(ctx, qn, page, n_pages, rng)
+    T, scale, lam, diff, eps = st.n_tokens, 0.7 / np.sqrt(d), 0.62, 0.3, 1e-5
+    keys, vals = [rng.standard_normal((c, G, 2, d)) for c in ctx], [rng.standard_normal((c, G, dv)) for c in ctx]
+    q = rng.standard_normal((T, H, 2, d))
+    for t in range(T):
+        b, pos = st.host_seq[t], st.host_pos[t]
+        spots = [0, (pos // page) * page - 1, (pos // page) * page, pos // 2, pos, pos - window + 1, pos - window, pos - 1]
+        for h in range(H):
+            for m in (0, 1):
+                j = min(max(spots[(h + 3 * m + t) % len(spots)], 0), pos)
+                k = keys[b][j, h // (H // G), m]
+                q[t, h, m] = k * (11.0 / scale / float(k @ k)) if (t + h) % 3 else q[t, h, m]
+    gate = dev(rng.standard_normal((T, H + 11)) * 2, dtype)[:, 8:8 + H]
+    qd, out = dev(q.reshape(T, -1), dtype), torch.full((T, H * dv), float("nan"), dtype=dtype, device="cuda")
+    kr = [host(dev(k.reshape(k.shape[0], G, 2 * d), dtype)) for k in keys]
+    vr = [host(dev(v, dtype)) for v in vals]
+    kc, vc = fill_pools(st, kr, vr, page, n_pages, dtype)
+    ops.launches_by_kernel.clear()
+    ops.attention_difference(qd, kc, vc, out, gate, st, 0, H, G, d, dv, page, scale, cap, lam, 1.0 - diff, eps, window)
+    args = (host(qd).reshape(T, H, 2, d), [k.reshape(-1, G, 2, d) for k in kr], vr, scale)
+    want, got = plain_difference_rows(*args, cap, window, lam, diff, eps, host(gate), st, H, G), host(out).reshape(T, H, dv)
+    err = np.abs(got - want).max(axis=(1, 2))
+    assert np.isfinite(got).all() and err.max() <= (5e-5 if dtype == torch.float32 else 0.06), \
+        f"row {int(err.argmax())} (request {st.host_seq[int(err.argmax())]}, position {st.host_pos[int(err.argmax())]}): {err.max()}"
+    if cap == 9.0 or window:                                # the test bites
+        other = plain_difference_rows(*args, 0.0 if cap == 9.0 else cap, window + 1 if window else 0, lam, diff, eps, host(gate), st, H, G)
+        assert np.abs(other - want).max() > 0.15
+    ran = set(ops.launches_by_kernel)
+    if dtype == BF16 and ops.difference_prefill_takes_mma(dtype, d, dv, page):
+        assert "attention_difference.prefill.tcgen05" in ran
+    if dtype == BF16 and ops.difference_decode_takes_mma(dtype, H, G, d, dv):
+        assert ran & {"attention_difference.decode.mma", "attention_difference.decode.mma.split"}
+        if not window:
+            assert "attention_difference.decode.mma.split" in ran
+    ops.check_device_errors()
+
+
+def test_single_tokens_whose_contexts_are_not_cut():
+    """Contexts so short, and requests so many, that decode attention takes one piece each."""
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(4)
+    H, G, d, dv, page = 8, 2, 64, 128, 16
+    ctx = [1, 2, 15, 16, 17, 63, 64, 65, 127, 100]
+    st = hand_step(ctx, [1] * len(ctx), page, 60, rng)
+    T = st.n_tokens
+    keys, vals = [rng.standard_normal((c, G, 2 * d)) for c in ctx], [rng.standard_normal((c, G, dv)) for c in ctx]
+    q = dev(rng.standard_normal((T, H * 2 * d)) * 2, BF16)
+    kr, vr = [host(dev(k, BF16)) for k in keys], [host(dev(v, BF16)) for v in vals]
+    kc, vc = fill_pools(st, kr, vr, page, 60, BF16)
+    out = torch.full((T, H * dv), float("nan"), dtype=BF16, device="cuda")
+    ops.launches_by_kernel.clear()
+    ops.attention_difference(q, kc, vc, out, None, st, 0, H, G, d, dv, page, 0.2, 30.0, 0.5, 0.7, 1e-5)
+    want = plain_difference_rows(host(q).reshape(T, H, 2, d), [k.reshape(-1, G, 2, d) for k in kr], vr, 0.2, 30.0, 0, 0.5, 0.3, 1e-5,
+                                 np.full((T, H), 60.0), st, H, G)
+    np.testing.assert_allclose(host(out).reshape(T, H, dv), want, rtol=0, atol=0.05)
+    assert ops.launches_by_kernel == {"attention_difference.decode.mma": 1}
+
+
+@pytest.mark.parametrize("dtype", [torch.float32, BF16])
+@pytest.mark.parametrize("H,rank,rot,window,page", [(3, 40, 8, 7, 8), (6, 64, 32, 100, 16), (18, 128, 16, 600, 16), (2, 512, 64, 0, 32),
+                                                    (1, 16, 2, 1, 16), (5, 256, 32, 64, 64)])
+def test_latent_attention_with_a_gate_at_window_edges(dtype, H, rank, rot, window, page):
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(rank + window)
+    dk = rank + rot
+    ctx, qn = [150, 70, 129, 1, 2, 1500, 65, 720], [150, 1, 37, 1, 2, 1, 64, 1]
+    n_pages = sum(-(-c // page) for c in ctx) + 3
+    st = hand_step(ctx, qn, page, n_pages, rng)
+    T, scale = st.n_tokens, 0.5 / np.sqrt(dk)
+    rows = [host(dev(rng.standard_normal((c, dk)), dtype)) for c in ctx]
+    qa = rng.standard_normal((T, H, dk))
+    for t in range(T):
+        b, pos = st.host_seq[t], st.host_pos[t]
+        spots = [pos - window + 1, pos - window, 0, (pos // page) * page, (pos // page) * page - 1, pos]
+        for h in range(H):
+            j = min(max(spots[(h + t) % len(spots)], 0), pos)
+            if (t + h) % 3:
+                qa[t, h] = rows[b][j] * (7.0 / scale / float(rows[b][j] @ rows[b][j]))
+    cache, _ = fill_pools(st, [r[:, None] for r in rows], [r[:, None, :1] for r in rows], page, n_pages, dtype)
+    gate = dev(rng.standard_normal((T, H + 9)) * 2, dtype)[:, 9:]
+    out = torch.full((T, H * rank), float("nan"), dtype=dtype, device="cuda")
+    want = np.zeros((T, H, rank))
+    qd = dev(qa.reshape(T, -1))
+    qr = host(dev(qa, BF16)) if ops.latent_attention_queries_dtype(st, dtype, dk, rank) == BF16 else host(dev(qa))
+    ops.launches_by_kernel.clear()
+    ops.attention_latent(qd, cache, out, st, 0, H, rank, page, scale, None, window, gate=gate)
+    for t in range(T):
+        b, pos = st.host_seq[t], st.host_pos[t]
+        lo = max(0, pos - window + 1) if window else 0
+        for h in range(H):
+            want[t, h] = P.softmax(rows[b][lo:pos + 1] @ qr[t, h] * scale) @ rows[b][lo:pos + 1, :rank]
+    want *= P.sigmoid(host(gate))[:, :, None]
+    np.testing.assert_allclose(host(out).reshape(T, H, rank), want, rtol=0, atol=3e-5 if dtype == torch.float32 else 0.04)
+    if dtype == BF16 and ops.latent_attention_takes_mma(dtype, dk, rank):
+        split = window == 0 or window >= 256
+        assert ops.launches_by_kernel.get("attention_latent.decode.mma" + (".split" if split else ""))
+
+
+# ---- whole models ------------------------------------------------------------------------------
+
+ALONE = {
+    "attention_only": U.model(61, 48, 1e-5, [U.attention(4, 2, 16, 8, 0.5, 8.0, 0.3, (8, 100.0))]),
+    "latent_only": U.model(61, 48, 1e-5, [U.latent(3, 8, 8, 12, 16, 0.4, 11, 200.0)]),
+    "attention_with_unit": U.model(61, 48, 1e-5, [U.attention(2, 2, 24, 24, 0.3, 20.0, 0.7, (24, 1000.0), 40)]),
+    "latent_with_unit": U.model(61, 48, 1e-5, [U.latent(2, 16, 4, 8, 24, 0.4, 30, 200.0, 56)]),
+    "looped": U.model(61, 48, 1e-5, [U.attention(2, 1, 8, 8, 0.6, 9.0, 0.2, (4, 50.0), 24)], (0, 1, 3)),
+    "loop_at_the_end": U.model(61, 48, 1e-5, [U.latent(2, 8, 8, 8, 16, 0.5, 5, 90.0), U.latent(2, 8, 8, 8, 16, 0.5, 5, 90.0, 32)], (1, 2, 2)),
+}
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which", sorted(ALONE))
+def test_each_kind_of_layer_alone(model_root, which, dtype):
+    d = U.make_dir(model_root, which, ALONE[which], 11)
+    reqs = requests_for(ALONE[which], [1, 2, 37, 90])
+    ref = plain_logits(d, reqs, dtype)
+    for fam, steps in (("whole", R.whole_trace(reqs)), ("decode", R.decode_trace(reqs, tail=20)),
+                       ("chunks", R.chunk_trace(reqs, seed=2))):
+        s = session(d, dtype, R.live_token_peak(steps), 8)
+        ok, what = ref.holds(R.collect(s.step, steps))
+        assert ok, f"{which} {dtype} {fam}: {what}"
+
+
+@pytest.mark.parametrize("which", ["A", "D", "E"])
+def test_the_stream_after_every_run_of_a_layer(model_root, which):
+    from rust_llm_inference_server_b200.parts.block import ParallelBlock
+    d = U.make_dir(model_root, which)
+    cfg, w = U.read_config(d), U.plain_weights(d)
+    toks = requests_for(cfg, [45], seed=4)["r0"]
+    want = P.forward(cfg, w, toks)[1]
+    s = session(d, "float32", 64, 16)
+    seen = []
+    for blk in set(s.model.blocks):
+        assert isinstance(blk, ParallelBlock)
+
+        def tapped(*a, _inner=blk.forward, **k):
+            resid, pending = _inner(*a, **k)
+            seen.append(host(resid) + sum(host(p) for p in (pending if isinstance(pending, tuple) else (pending,))))
+            return resid, pending
+        blk.forward = tapped
+    s.step({"step": 0, "entries": [{"id": "x", "tokens": toks, "want": [len(toks) - 1]}], "end": ["x"]})
+    assert len(seen) == len(U.runs(cfg))
+    for i, (got, ref) in enumerate(zip(seen, want)):
+        np.testing.assert_allclose(got, ref, rtol=0, atol=2e-4 * max(1.0, np.abs(ref).max() / 10), err_msg=f"after run {i}")
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which,page,lens", [("A", 16, [1, 50, 97, 200, 64, 17, 2]), ("A", 8, [130, 33, 2, 71, 40]),
+                                             ("B", 16, [3, 150, 40, 2, 129, 1]), ("C", 16, [1, 70, 333, 2, 129, 64, 65]),
+                                             ("C", 64, [200, 65, 2, 30]), ("D", 16, [90, 1, 33, 150, 2]), ("D", 32, [260, 31, 5, 90]),
+                                             ("E", 16, [420, 3, 200, 77]), ("F", 16, [300, 5, 131, 64])])
+def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens, dtype):
+    from rust_llm_inference_server_b200 import ops
+    ops.launches_by_kernel.clear()
+    d = U.make_dir(model_root, which)
+    reqs = requests_for(U.CONFIGS[which], lens, seed=page)
+    ref = plain_logits(d, reqs, dtype)
+    families = {
+        "whole": (R.whole_trace(reqs), 4),
+        "decode": (R.decode_trace(reqs, tail=40), 4),
+        "chunks": (R.chunk_trace(reqs, seed=3), 4),
+        "mixed": (R.mixed_trace(reqs, seed=4), 4),
+        "mixed2": (R.mixed_trace(dict(reversed(list(reqs.items()))), seed=5, max_live=2), 2),
+    }
+    results = {}
+    for fam, (steps, live) in families.items():
+        s = session(d, dtype, R.live_token_peak(steps, max(64, page)), page, max_live=live)
+        for pool in s.storage.pools:                         # whatever a page held before must not matter
+            for t in (pool if isinstance(pool, tuple) else (pool,)):
+                t.fill_(30.0)
+        results[fam] = R.collect(s.step, steps)
+        assert s.cache.check_invariants() == ""
+        for g in range(len(s.storage.groups)):
+            assert s.cache.num_free_pages(g) == s.cache.group(g).num_pages, fam
+        ok, what = ref.holds(results[fam])
+        assert ok, f"{which} {dtype} {fam} vs plain: {what}"
+    for fam in ("decode", "chunks", "mixed", "mixed2"):
+        ok, what = ref.holds(results[fam], results["whole"], between=True)
+        assert ok, f"{which} {dtype}: {fam} differs from whole by {what}"
+    launched = ops.launches_by_kernel
+    needed = {"layer_norm", "layer_norm.rows", "qk_norm_store.rot", "latent_kv_store"}
+    if dtype == "float32":
+        needed |= {"attention_difference", "attention_latent"}
+    elif U.CONFIGS[which]["width"] % 8 == 0:
+        needed |= {"stream_gemm.scaled.centred.mixed", "stream_gemm.sink.centred.two", "embedding.sink"}
+        if U.CONFIGS[which].get("loop"):
+            needed |= {"stream_gemm.sink.centred"}
+        if which != "F":
+            needed |= {"attention_difference.decode.mma", "attention_difference.prefill.tcgen05"}
+        if which in ("C", "E"):
+            needed |= {"attention_latent.decode.mma", "attention_latent.prefill.mma", "gemm_tcgen05.glu4"}
+    assert needed <= set(launched), f"never launched {sorted(needed - set(launched))}"
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("which,n,tail", [("A", 230, 215), ("C", 260, 240)])
+def test_long_decoding_while_the_windows_pass_over_decoded_tokens(model_root, which, n, tail, dtype):
+    d = U.make_dir(model_root, which)
+    reqs = requests_for(U.CONFIGS[which], [n], seed=9)
+    ref = plain_logits(d, reqs, dtype)
+    steps = R.decode_trace(reqs, tail=tail)             # a page border every 8 tokens; steps replayed from a CUDA graph
+    s = session(d, dtype, R.live_token_peak(steps), 8)
+    ok, what = ref.holds(R.collect(s.step, steps))
+    assert ok, what
+    assert s.runner._graph_launches > 0
+
+
+def test_pages_behind_a_window_are_given_back(model_root):
+    d = U.make_dir(model_root, "A")
+    s = session(d, "bfloat16", 256, 8, max_live=1)
+    toks = requests_for(U.CONFIGS["A"], [180], seed=2)["r0"]
+    s.step({"step": 0, "entries": [{"id": "x", "tokens": toks[:100], "want": []}], "end": []})
+    for i in range(100, 180):
+        s.step({"step": i, "entries": [{"id": "x", "tokens": toks[i:i + 1], "want": []}], "end": []})
+    held = {(g.spec.window if hasattr(g, "spec") else None): s.cache.group(i).num_pages - s.cache.num_free_pages(i)
+            for i, g in enumerate(s.storage.groups)}
+    assert min(held.values()) <= 3 and max(held.values()) >= 180 // 8      # a window of 7 holds two or three pages of 8
+
+
+def plain_greedy(cfg, w, prompt, n):
+    toks = list(prompt)
+    for _ in range(n):
+        toks.append(int(np.argmax(P.forward(cfg, w, toks)[0][-1])))
+    return toks[len(prompt):]
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_greedy_generation_through_the_entry_point(model_root, dtype):
+    """Prompts of unequal length batched by the scheduler, portions of 16 tokens, decode steps from CUDA graphs and
+    launched ahead; two seats, so the later prompts take over pages."""
+    from rust_llm_inference_server_b200 import LLM, SamplingParams
+    d = U.make_dir(model_root, "A")
+    cfg, w = U.read_config(d), U.plain_weights(d)
+    prompts = list(requests_for(cfg, [1, 9, 40, 23, 3], seed=12).values())
+    llm = LLM(d, dtype=dtype, max_seq_len=128, num_blocks=60, block_size=8, max_num_seqs=2, max_batched_tokens=16)
+    outs = llm.generate(prompts, SamplingParams(max_tokens=12))
+    for p, o in zip(prompts, outs):
+        want = plain_greedy(cfg, w, p, 12)
+        assert o.finish_reason == "length" and len(o.token_ids) == 12
+        if o.token_ids != want:
+            i = next(k for k, (a, b) in enumerate(zip(o.token_ids, want)) if a != b)
+            lg = P.forward(cfg, w, p + want[:i])[0][-1]
+            gap = (lg[want[i]] - lg[o.token_ids[i]]) / lg.std()
+            assert dtype == "bfloat16" and gap < 0.15, f"parted at token {i} with a gap of {gap}"
+    assert llm.engine.cache.check_invariants() == ""
+    assert llm.engine.runner._graph_launches > 0
+
+
+def test_command_line_serves_the_design(tmp_path):
+    """random-weights and generate of the command line with a Dotivik folder."""
+    import json
+    import os
+    import subprocess
+    import sys
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+
+    def rlis(*args):
+        return subprocess.run([sys.executable, os.path.join(root, "bin", "rlis"), *args], capture_output=True,
+                              text=True, timeout=600)
+
+    cfg_file = tmp_path / "c.json"
+    cfg_file.write_text(json.dumps(U.CONFIGS["A"]))
+    d = str(tmp_path / "m")
+    r = rlis("random-weights", "--config", str(cfg_file), "--seed", "21", "--out", d)
+    assert r.returncode == 0, r.stderr[-2000:]
+    cfg, w = U.read_config(d), U.plain_weights(d)
+    assert cfg["architecture"] == "Dotivik" and set(w) == set(U.tensor_shapes(cfg))
+    prompt = [5, 9, 200, 31, 7]
+    r = rlis("generate", "--model", d, "--dtype", "f32", "--prompt-ids", ",".join(map(str, prompt)),
+             "--max-tokens", "8", "--max-seq-len", "64", "--kv-cache-gb", "0.001", "--block-size", "8",
+             "--max-num-seqs", "2")
+    assert r.returncode == 0, r.stderr[-2000:]
+    assert [int(t) for t in r.stdout.split()] == plain_greedy(cfg, w, prompt, 8)
