@@ -96,8 +96,9 @@ def rotate_halves(x, rot):
 
 
 def softmax(s):
-    e = np.exp(s - s.max())
-    return e / e.sum()
+    """Over the last axis; a hidden key has a score of minus infinity."""
+    e = np.exp(s - s.max(axis=-1, keepdims=True))
+    return e / e.sum(axis=-1, keepdims=True)
 
 
 def capped(s, cap):
@@ -107,12 +108,9 @@ def capped(s, cap):
 def softmax_attention(q, k, v, score, window=None):
     """One head: q, k [T, d], v [T, dv]; `score` turns raw products into scores; each row sees the keys up to itself,
     the last `window` of them where one is given."""
-    raw = q @ k.T
-    out = np.zeros((q.shape[0], v.shape[1]))
-    for i in range(q.shape[0]):
-        lo = 0 if window is None else max(0, i - int(window) + 1)
-        out[i] = kept(softmax(score(raw[i, lo:i + 1]))) @ v[lo:i + 1]
-    return out
+    i, j = np.arange(q.shape[0])[:, None], np.arange(k.shape[0])[None, :]
+    seen = (j <= i) if window is None else (j <= i) & (i - j < int(window))
+    return kept(softmax(np.where(seen, score(q @ k.T), -np.inf))) @ v
 
 
 def head_weight(w, p, diff):
