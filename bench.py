@@ -1150,6 +1150,133 @@ def workload_papulix(args, torch, np) -> dict:
                            papulix_kernel_rooflines, args, torch, np)
 
 
+def dotivik_config(width: int, vocab: int = 32000) -> dict:
+    """Four Dotivik layers at a real model's proportions, run as one pass (with the map in front of it).  Attention of two maps:
+    heads of 2 x 64 in groups of four with values of 128, half of a map rotated, scores capped at 50.  Latent attention: heads
+    of 128 with 64 rotated entries, a latent of 512, a window of 1,024.  Gated units of 8/3 widths beside every mixer."""
+    H = width // 128
+    attn = {"heads": H, "kv_heads": max(1, H // 4), "dim": 64, "vdim": 128, "scale": 0.125, "softcap": 50.0, "diff": 0.3,
+            "rot": {"dims": 32, "base": 50000.0}}
+    lat = {"heads": H, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "scale": (128 + 64) ** -0.5, "mask": {"size": 1024},
+           "rot": {"dims": 64, "base": 500000.0}}
+    mlp = {"kind": "dense", "ff": width * 8 // 3 // 128 * 128}
+    return {"architecture": "Dotivik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": {"start": 0, "stop": 4, "times": 1},
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in
+                       (("attention", attn), ("latent_attention", lat), ("attention", attn), ("latent_attention", lat))]}
+
+
+def dotivik_kernel_rooflines(width: int, B: int, ctx: int, T: int, pk: dict, torch, np) -> dict:
+    """The kernels that Dotivik adds or extends, alone, at the sizes of `dotivik_config(width)`, each beside the like kernel of
+    the closest models: {name: {"us", "ideal_us", "frac"}}.  Ideal: bytes that must move over the measured copy bandwidth
+    (single tokens, norms, stores), or FLOPs over the measured bfloat16 GEMM rate (over prompts); attention over prompts counts
+    what the scores and value sums of the visible keys need (two maps of d and two value sums of dv a head and key)."""
+    from rust_llm_inference_server_b200 import ops
+    from rust_llm_inference_server_b200.parts.spec import GELU_TANH
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    page, H, G, d, dv = 16, width // 128, max(1, width // 512), 64, 128
+    rank, rot, window, nh, nkv, hd = 512, 64, 1024, width // 64, max(1, width // 256), 64
+    dk, I = rank + rot, width * 8 // 3 // 128 * 128
+    bf, out = torch.bfloat16, {}
+    rnd = lambda *shape: torch.randn(*shape, device="cuda") * 0.3
+
+    def row(name, us, ideal_s):
+        out[name] = {"us": round(us, 1), "ideal_us": round(ideal_s * 1e6, 1), "frac": round(ideal_s * 1e6 / us, 3)}
+    timed = lambda fn: _graph_time_us(fn, torch)
+
+    for kind, reqs in (("decode", [(ctx - 1, 1)] * B), ("prefill", [(0, T)])):
+        st = _KernelStep(reqs, page, torch, np)
+        dec, n = kind == "decode", st.n_tokens
+        st.n_prefill_tokens = 0 if dec else st.n_prefill_tokens
+        keys = B * ctx if dec else T * (T + 1) // 2
+        seen = B * min(ctx, window) if dec else sum(min(p + 1, window) for p in range(T))
+        # two maps a head with cap, difference, norm and gate, beside the slope attention and Llama's (heads of 64)
+        kc, vc, q = rnd(st.n_pages, G, page, 2 * d).to(bf), rnd(st.n_pages, G, page, dv).to(bf), rnd(n, H * 2 * d).to(bf)
+        gate, o = rnd(n, H + 8).to(bf)[:, :H], torch.empty(n, H * dv, dtype=bf, device="cuda")
+        us = timed(lambda: ops.attention_difference(q, kc, vc, o, gate, st, 0, H, G, d, dv, page, 0.125, 50.0, 0.4, 0.7, 1e-5))
+        row(f"difference_attention_{kind}", us, keys * G * (2 * d + dv) * 2 / hbm if dec else 2 * H * keys * 2 * (d + dv) / tf)
+        kc2, vc2, q2 = rnd(st.n_pages, nkv, page, hd).to(bf), rnd(st.n_pages, nkv, page, hd).to(bf), rnd(n, nh * hd).to(bf)
+        o2, slopes = torch.empty_like(q2), torch.tensor([2.0 ** (-8.0 * (h + 1) / nh) for h in range(nh)], device="cuda")
+        attn = keys * nkv * hd * 2 * 2 / hbm if dec else 2 * nh * keys * 2 * hd / tf
+        row(f"slope_attention_{kind}", timed(lambda: ops.attention_biased(q2, kc2, vc2, o2, None, None, st, 0, nh, nkv, hd, hd, page, 0.125,
+                                                                          0, slopes=slopes)), attn)
+        row(f"gqa_attention_{kind}", timed(lambda: ops.attention(q2, kc2, vc2, o2, st, 0, nh, nkv, hd, page, 0.125, 0)), attn)
+        # latent attention with a window and a gate, beside Lasapel's over all keys
+        cache, qa, lat = rnd(st.n_pages, 1, page, dk).to(bf), rnd(n, H * dk).to(bf), torch.empty(n, H * rank, dtype=bf, device="cuda")
+        us = timed(lambda: ops.attention_latent(qa, cache, lat, st, 0, H, rank, page, 0.07, None, window, gate=gate))
+        row(f"latent_window_gate_attention_{kind}", us, max(seen * dk * 2 / hbm, 2 * H * seen * (dk + rank) / tf) if dec
+            else 2 * H * seen * (dk + rank) / tf)
+        us = timed(lambda: ops.attention_latent(qa, cache, lat, st, 0, H, rank, page, 0.07, None, 0))
+        row(f"latent_attention_{kind}", us, max(keys * dk * 2 / hbm, 2 * H * keys * (dk + rank) / tf) if dec
+            else 2 * H * keys * (dk + rank) / tf)
+        # rotation and paged write of two vectors a head, beside one with norms
+        N = 2 * H * d + 2 * G * d + G * dv + H
+        proj, slots = rnd(n, N + (-N % 8)).to(bf), torch.arange(n, device="cuda", dtype=torch.int32)
+        freq, one = torch.ones(16, device="cuda"), torch.ones(hd, device="cuda")
+        us = timed(lambda: ops.qk_norm_store(proj, 0, 2 * H * d, 2 * (H + G) * d, None, None, 1e-5, None, 0.0, q, kc, vc, slots, H, G, d, dv,
+                                             page, rotation=(freq, 32, 1.0), positions=st.positions, maps=2))
+        row(f"two_map_store_{kind}", us, 2 * n * (N - H) * 2 / hbm)
+        proj2 = rnd(n, (nh + 2 * nkv) * hd).to(bf)
+        us = timed(lambda: ops.qk_norm_store(proj2, 0, nh * hd, (nh + nkv) * hd, one, one, 1e-5, None, 0.0, q2, kc2, vc2, slots, nh, nkv, hd,
+                                             hd, page, rotation=(freq, 32, 1.0), positions=st.positions))
+        row(f"head_norm_store_{kind}", us, 2 * n * (nh + 2 * nkv) * hd * 2 / hbm)
+        # the layer norm that joins two sublayers, beside the RMS norm that joins one
+        resid, a, b, h = rnd(n, width).contiguous(), rnd(n, width).to(bf), rnd(n, width).to(bf), torch.empty(n, width, dtype=bf, device="cuda")
+        wv = torch.ones(width, device="cuda")
+        row(f"layer_norm_two_{kind}", timed(lambda: ops.layer_norm(resid, wv, 1e-5, h, (a, b))), n * width * (8 + 6) / hbm)
+        row(f"residual_rmsnorm_{kind}", timed(lambda: ops.rmsnorm(resid, wv, 1e-5, h, a)), n * width * (8 + 4) / hbm)
+        # the unit gated by gelu, beside silu
+        wgu, wdn = rnd(2 * I, width).to(bf), rnd(width, I).to(bf)
+        glu = (GELU_TANH["slope"], None, 0.0, GELU_TANH["cubic"])
+        ideal = 3 * I * width * 2 / hbm if dec else 2.0 * n * 3 * I * width / tf
+        if dec:
+            row("gelu_gated_ff_decode", timed(lambda: ops.linear(ops.stream_gemm(a, wgu, swiglu4=True, **GELU_TANH), wdn)), ideal)
+            row("silu_gated_ff_decode", timed(lambda: ops.linear(ops.stream_gemm(a, wgu, swiglu4=True), wdn)), ideal)
+        else:
+            row("gelu_gated_ff_prefill", timed(lambda: ops.linear(ops.gemm_tcgen05(a, wgu, "glu4", glu=glu), wdn)), ideal)
+            row("silu_gated_ff_prefill", timed(lambda: ops.linear(ops.gemm_tcgen05(a, wgu, "swiglu4"), wdn)), ideal)
+        # the map in front of a pass, beside the same product alone
+        wx, base = rnd(width, width).to(bf), rnd(n, width).contiguous()
+        ideal = width * width * 2 / hbm if dec else 2.0 * n * width * width / tf
+        if dec:
+            sink = ops.ResidualSink(resid, wv, 1e-5, centred=True, base=base, exact=True)
+            row("pass_input_decode", timed(lambda: ops.linear(a, wx, sink=sink)), ideal)
+            row("product_into_stream_decode", timed(lambda: ops.linear(a, wx, sink=ops.ResidualSink(resid, wv, 1e-5))), ideal)
+            # both products of a block, beside Llama's four: norm applied, gated second part; two sources, into the stream
+            Np = N + (-N % 8)
+            w_in, wo, act = rnd(Np + 2 * I, width).to(bf), rnd(width, H * dv).to(bf), rnd(n, I).to(bf)
+            rows = ops.linear(a, wx, sink=sink)
+            ideal = ((Np + 2 * I) * width + width * (H * dv + I)) * 2 / hbm
+            both = ops.ResidualSink(resid, wv, 1e-5, centred=True, exact=True)
+
+            def block():
+                ops.stream_gemm(rows, w_in, n_plain=Np, **GELU_TANH)
+                return ops.linear(o, wo, sink=both, second=(act, wdn))
+            row("block_products_decode", timed(block), ideal)
+            wq = rnd((nh + 2 * nkv) * hd, width).to(bf)
+            wo2 = rnd(width, nh * hd).to(bf)
+            rs = ops.ResidualSink(resid, wv, 1e-5)
+            r2 = ops.linear(a, wx, sink=rs)
+
+            def llama():
+                ops.linear(r2, wq)
+                x = ops.linear(o2, wo2, sink=rs)
+                return ops.linear(ops.stream_gemm(x, wgu, swiglu4=True), wdn, sink=rs)
+            row("llama_products_decode", timed(llama), ((nh + 2 * nkv) * hd * width + width * nh * hd + 3 * I * width) * 2 / hbm)
+        else:
+            row("pass_input_prefill", timed(lambda: ops.linear_add(a, wx, base)), ideal)
+            row("product_float32_prefill", timed(lambda: ops.linear(a, wx, out_dtype=torch.float32)), ideal)
+    return out
+
+
+def workload_dotivik(args, torch, np) -> dict:
+    """Prefill (one 2,048-token prompt) and decode (batch 8, context 4,096) of four Dotivik layers at two widths beside four
+    Lasapel layers (the closest model: latent attention) and four Llama layers of the same width, random bfloat16 weights;
+    then the stages of one step by CUDA-event spans (eager launches), and the kernels alone, replayed from CUDA graphs,
+    against their rooflines."""
+    return layers_workload("dotivik", (("dotivik", dotivik_config), ("lasapel", lasapel_config), ("llama", llama_config_like)),
+                           dotivik_kernel_rooflines, args, torch, np)
+
+
 def layers_workload(head: str, models, rooflines, args, torch, np) -> dict:
     """Prefill, decode and stages of four layers of every one of `models` (name, configuration by width) at two widths, and
     the kernels of the first alone."""
@@ -1229,7 +1356,8 @@ def print_timeline(records: list) -> None:
 
 
 WORKLOADS = {"3b": workload_3b, "8b": workload_8b, "1b-fp32": workload_1b_fp32, "lasapel": workload_lasapel,
-             "gavodra": workload_gavodra, "lanirax": workload_lanirax, "rumedra": workload_rumedra, "papulix": workload_papulix}
+             "gavodra": workload_gavodra, "lanirax": workload_lanirax, "rumedra": workload_rumedra, "papulix": workload_papulix,
+             "dotivik": workload_dotivik}
 
 
 def main() -> int:
