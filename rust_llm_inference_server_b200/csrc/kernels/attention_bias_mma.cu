@@ -18,7 +18,9 @@
 // Single tokens with two maps a head (attention_difference.cu): the same, with rows 0..7 of the products the query heads' first
 // maps and rows 8..15 their second ones (groups of up to 8).  A key row is [map 1 | map 2], each padded to 64 entries; a query
 // row is its map's vector and zeros over the other's entries, so one set of products gives both maps' scores and the values
-// are multiplied once.  The maps meet where the warps (or the pieces) are merged.
+// are multiplied once.  The maps meet where the warps (or the pieces) are merged: up to 16 pieces of a context are a
+// thread-block cluster, which merges through distributed shared memory (a CTA a head of the group, a warp a quarter of its
+// columns), more by a second kernel.
 #include "common.cuh"
 #include "mma_utils.cuh"
 #include <math.h>
@@ -570,6 +572,7 @@ __global__ __launch_bounds__(128) void attn_bias_decode_merge_kernel(
     }
 }
 
+constexpr int MAX_CLUSTER_PIECES = 16;
 struct DiffDecode {
     const bf16 *q, *k_cache, *v_cache;
     bf16* out;
@@ -578,6 +581,7 @@ struct DiffDecode {
     long long gate_stride;
     const int *dec_rows, *dec_seqs, *ctx_lens, *block_tables;
     int max_blocks, nh, nkv, d, dv, page_size, window, pieces;
+    int cluster;              // 1: the pieces are a cluster and merge themselves
     float scale, cap, lambda, out_scale, eps;
 };
 
@@ -600,10 +604,12 @@ __device__ __forceinline__ void store_difference(const float* base, int n, size_
     for (int mp = 0; mp < 2; ++mp) {
         const float* b = base + mp * map_stride;
         float m = -INFINITY, l = 0.f;
-        for (int p = 0; p < n; ++p) m = fmaxf(m, b[p * part_stride + mcol]);
+        for (int p = lane; p < n; p += 32) m = fmaxf(m, b[p * part_stride + mcol]);
+        m = warp_max(m);
         float a[NC];
 #pragma unroll
         for (int i = 0; i < NC; ++i) a[i] = 0.f;
+#pragma unroll 4
         for (int p = 0; p < n; ++p) {
             const float* r = b + p * part_stride;
             const float f = r[mcol] == -INFINITY ? 0.f : exp2f(r[mcol] - m);
@@ -808,6 +814,8 @@ __global__ __launch_bounds__(THREADS) void attn_difference_decode_kernel(const D
         }
         return;
     }
+    // (in a cluster: this CTA's merged rows [head][map][MW], behind the warps' rows)
+    float* mine = mg + (size_t)WARPS * 16 * MW;
     for (int idx = threadIdx.x; idx < 2 * nrep * DV; idx += THREADS) {
         const int u = idx / DV, col = idx - u * DV, r = u >> 1, mp = u & 1;
         const float* b = mg + (size_t)(mp * 8 + r) * MW;
@@ -821,10 +829,60 @@ __global__ __launch_bounds__(THREADS) void attn_difference_decode_kernel(const D
             l = fmaf(x[DV + 1], f, l);
             o = fmaf(x[col], f, o);
         }
-        float* dst = a.partial + ((((size_t)bi * a.nh + kvh * nrep + r) * 2 + mp) * a.pieces + piece) * MW;
+        float* dst = a.cluster ? mine + (size_t)u * MW : a.partial + ((((size_t)bi * a.nh + kvh * nrep + r) * 2 + mp) * a.pieces + piece) * MW;
         dst[col] = o;
         if (col == 0) { dst[DV] = m; dst[DV + 1] = l; }
     }
+    if (!a.cluster) return;
+    cluster_sync_all();
+    __shared__ float red[WARPS];
+    for (int r = piece; r < nrep; r += a.pieces) {         // the same for all threads of the CTA
+        // warp w takes columns w, w + 4, ... blocks of 32; every lane reads its columns from all pieces
+        constexpr int NC = DV / 32 / WARPS > 0 ? DV / 32 / WARPS : 1;
+        float o[NC];
+#pragma unroll
+        for (int i = 0; i < NC; ++i) o[i] = 0.f;
+#pragma unroll
+        for (int mp = 0; mp < 2; ++mp) {
+            const float* b = mine + (size_t)(2 * r + mp) * MW;
+            // lane p holds piece p's maximum and denominator (up to 16 pieces)
+            const float pm = lane < a.pieces ? ld_dsmem(b + DV, (uint32_t)lane) : -INFINITY;
+            const float pl = lane < a.pieces ? ld_dsmem(b + DV + 1, (uint32_t)lane) : 0.f;
+            const float m = warp_max(pm);
+            const float pf = pm == -INFINITY ? 0.f : exp2f(pm - m);
+            const float inv = (mp == 0 ? 1.0f : -a.lambda) / warp_sum(pl * pf);
+            float x[NC][16];
+#pragma unroll
+            for (int p = 0; p < 16; ++p)
+#pragma unroll
+                for (int i = 0; i < NC; ++i) {
+                    const int col = (warp + i * WARPS) * 32 + lane;
+                    x[i][p] = p < a.pieces && col < DV ? ld_dsmem(b + col, (uint32_t)p) : 0.f;
+                }
+#pragma unroll
+            for (int p = 0; p < 16; ++p) {
+                const float f = __shfl_sync(0xffffffffu, pf, p) * inv;
+#pragma unroll
+                for (int i = 0; i < NC; ++i) o[i] = fmaf(x[i][p], f, o[i]);
+            }
+        }
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NC; ++i) ss = fmaf(o[i], o[i], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) red[warp] = ss;
+        __syncthreads();
+        const int head = kvh * nrep + r;
+        float f = a.out_scale / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)dv + a.eps);
+        if (a.gate != nullptr) f /= 1.0f + expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + head]));
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+            const int col = (warp + i * WARPS) * 32 + lane;
+            if (col < dv) a.out[((size_t)row * a.nh + head) * dv + col] = __float2bfloat16_rn(o[i] * f);
+        }
+        __syncthreads();
+    }
+    cluster_sync_all();        // nobody leaves while its rows may still be read
 }
 
 // Pieces of a context into one result: one warp a (token, head), both maps.
@@ -921,7 +979,10 @@ extern "C" int rlis_attention_difference_decode_takes(int nh, int nkv, int d, in
 // Width of a value row in the partial sums (values are padded to it).
 extern "C" int rlis_attention_difference_decode_width(int dv) { return dv <= 64 ? 64 : 128; }
 
-// partial: float32, at least n_dec * nh * 2 * pieces * (width(dv) + 2) elements when pieces > 1; the rest as
+// Up to this many pieces of a context merge inside a cluster.
+extern "C" int rlis_attention_difference_decode_cluster() { return MAX_CLUSTER_PIECES; }
+
+// partial: float32, at least n_dec * nh * 2 * pieces * (width(dv) + 2) elements when the pieces do not merge in a cluster; the rest as
 // rlis_attention_difference.
 extern "C" int rlis_attention_difference_decode(const void* q, const void* k_cache, const void* v_cache, void* out, float* partial,
                                                 const void* gate, long long gate_stride, const int* dec_rows, const int* dec_seqs,
@@ -930,24 +991,27 @@ extern "C" int rlis_attention_difference_decode(const void* q, const void* k_cac
                                                 float lambda, float out_scale, float eps, cudaStream_t stream) {
     if (n_dec <= 0) return 0;
     if (!rlis_attention_difference_decode_takes(nh, nkv, d, dv) || pieces < 1 || pieces > 65535 || n_dec > 65535 || cap < 0.f ||
-        (pieces > 1 && partial == nullptr) ||
+        (pieces > MAX_CLUSTER_PIECES && partial == nullptr) ||
         ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) != 0)
         return RLIS_ERR_UNSUPPORTED;
     static bool done = false;
     if (!done) {
         cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<128, 64>());
         cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<128, 128>());
+        cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+        cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         done = true;
     }
     const DiffDecode a{(const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, partial, (const bf16*)gate, gate_stride,
-                       dec_rows, dec_seqs, ctx_lens, block_tables, max_blocks, nh, nkv, d, dv, page_size, window, pieces, scale, cap,
-                       lambda, out_scale, eps};
+                       dec_rows, dec_seqs, ctx_lens, block_tables, max_blocks, nh, nkv, d, dv, page_size, window, pieces,
+                       pieces > 1 && pieces <= MAX_CLUSTER_PIECES ? 1 : 0, scale, cap, lambda, out_scale, eps};
     const dim3 grid(nkv, n_dec, pieces);
     const bool narrow = rlis_attention_difference_decode_width(dv) == 64;
-    if (narrow) rlis_launch(attn_difference_decode_kernel<64>, grid, THREADS, decode_smem_bytes<128, 64>(), stream, a);
-    else rlis_launch(attn_difference_decode_kernel<128>, grid, THREADS, decode_smem_bytes<128, 128>(), stream, a);
+    const dim3 cluster(1, 1, a.cluster ? (unsigned)pieces : 1u);
+    if (narrow) rlis_launch_cluster(attn_difference_decode_kernel<64>, grid, THREADS, decode_smem_bytes<128, 64>(), stream, cluster, a);
+    else rlis_launch_cluster(attn_difference_decode_kernel<128>, grid, THREADS, decode_smem_bytes<128, 128>(), stream, cluster, a);
     const int err = RLIS_LAUNCH_CHECK();
-    if (err != 0 || pieces == 1) return err;
+    if (err != 0 || pieces == 1 || a.cluster) return err;
     const int units = n_dec * nh;
     if (narrow) rlis_launch(attn_difference_merge_kernel<64>, (units + 3) / 4, 128, 0, stream, a, units);
     else rlis_launch(attn_difference_merge_kernel<128>, (units + 3) / 4, 128, 0, stream, a, units);

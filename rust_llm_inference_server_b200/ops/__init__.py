@@ -1703,8 +1703,21 @@ def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, 
                 and _difference_decode_sizes(int(n_heads), int(n_kv_heads), int(dim), int(v_dim)))
 
 
+@functools.lru_cache(maxsize=4096)
+def _difference_decode_pieces(n_decode: int, n_kv_heads: int, seen: int, sms: int) -> int:
+    """Pieces a context is cut into: a CTA takes one key/value head of one request and two fit an SM, so the context is cut
+    until they about fill the SMs, in pieces of at least two tiles of 64 keys.  Up to 16 pieces merge in a cluster; more only
+    where that many would still leave every CTA a long way to go."""
+    tiles = -(-seen // 64) + 1
+    want = max(1, min(2 * sms // max(1, n_decode * n_kv_heads), tiles // 2, 64))
+    if want > 16 and tiles <= 16 * 16:
+        want = 16
+    return max(1, -(-tiles // -(-tiles // want)))
+
+
 def difference_decode_pieces(n_decode: int, n_kv_heads: int, max_ctx: int, window: int = 0) -> int:
-    return biased_decode_pieces(n_decode, n_kv_heads, min(int(max_ctx), int(window)) if window else max_ctx)
+    seen = min(int(max_ctx), int(window)) if window else int(max_ctx)
+    return _difference_decode_pieces(int(n_decode), int(n_kv_heads), max(1, seen), num_sms())
 
 
 def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_heads: int, n_kv_heads: int, dim: int,
@@ -1735,13 +1748,13 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
     if n_dec:
         pieces = difference_decode_pieces(n_dec, n_kv_heads, step.max_decode_ctx, window)
         scratch = step.buffer("attn_partial", (n_dec * n_heads * 2 * pieces * (lib().rlis_attention_difference_decode_width(v_dim) + 2),),
-                              torch.float32) if pieces > 1 else None
+                              torch.float32) if pieces > lib().rlis_attention_difference_decode_cluster() else None
         check(lib().rlis_attention_difference_decode(
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), scratch.data_ptr() if scratch is not None else None,
             gp, gs, step.dec_rows.data_ptr(), step.dec_seqs.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1],
             n_dec, n_heads, n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), pieces, float(lam),
             float(out_scale), float(eps), _stream()), "attention_difference_decode")
-        _count("attention_difference.decode.mma" + (".split" if pieces > 1 else ""))
+        _count("attention_difference.decode.mma" + (".split" if scratch is not None else ".cluster" if pieces > 1 else ""))
     if n_tiles:
         check(lib().rlis_attention_difference_prefill(
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), gp, gs, step.prefill_tiles.data_ptr(), n_tiles,

@@ -63,6 +63,7 @@ SIGNATURES = {
     "rlis_attention_difference_decode": [P, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, F, F, F, P],
     "rlis_attention_difference_decode_takes": [I, I, I, I],
     "rlis_attention_difference_decode_width": [I],
+    "rlis_attention_difference_decode_cluster": [],
     "rlis_moe_route": [P, P, P, P, P, P, I, I, I, I, F, P, I, I, I, I, I, P],
     "rlis_moe_align": [P, P, P, P, I, I, I, I, P],
     "rlis_moe_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, I, P],
