@@ -13,7 +13,9 @@
 //   decode : 16 heads of one token and one piece of its context a CTA of 4 warps, stages of 32 keys,
 //            so that two CTAs fit an SM at the widest rows.  Warp w forms the scores of 8 of a stage's
 //            keys and sums a QUARTER of the value columns over all 32; maxima and weights go through
-//            shared memory.  Several pieces of a context are merged by a second small kernel.
+//            shared memory.  Up to 16 pieces of a context are a thread-block cluster: their CTAs leave
+//            sums, maxima and denominators in shared memory, and CTA z merges heads z, z + pieces, ...
+//            of the tile through distributed shared memory.  More are merged by a second small kernel.
 // Queries arrive as bfloat16 (copied asynchronously) or as float32 (rounded once, into shared memory).
 #include "common.cuh"
 #include "mma_utils.cuh"
@@ -22,6 +24,7 @@
 namespace {
 constexpr int LF_BN_MAX = 64;             // the longest stage: pieces of a context are multiples of it
 constexpr float LOG2E = 1.4426950408889634f;
+constexpr int LATENT_CLUSTER_PIECES = 16;      // up to this many pieces of a context merge inside a cluster
 
 // Barrier over the two warps of pair `p` (named barriers 1..4; 0 is __syncthreads).
 __device__ __forceinline__ void pair_barrier(int p) { asm volatile("bar.sync %0, 64;" ::"r"(p + 1) : "memory"); }
@@ -41,6 +44,7 @@ struct LatentArgs {
     int max_blocks, nh, dk, page_size, window, pieces, piece_keys;
     float scale;
     int q_bf16;
+    int cluster;              // decode: 1: the pieces are a cluster and merge themselves
     const bf16* gate;         // logits, one a head: head h of token t at gate[t * gate_stride + h]; null: none
     long long gate_stride;
 };
@@ -317,6 +321,7 @@ template <int DV>
 __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) {
     pdl_wait();
     constexpr int BN = 32, NO = DV / 32, PS = BN + 8;   // keys a stage; output tiles a warp; row pitch of the weights
+    static_assert(16 * (DV + 2) * 4 <= 2 * BN * (DV + 8) * 2, "a cluster's rows lie in the stages of keys (rows of DV entries or more)");
     const int dk = a.dk, stride = dk + 8, ksteps = dk / 16, cpr = dk / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* qs = reinterpret_cast<bf16*>(smem_raw);              // [16][stride]
@@ -513,7 +518,9 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
                 *reinterpret_cast<uint32_t*>(o + n * 8 + 2 * c) = pack_bf16(oacc[n][2] * inv1, oacc[n][3] * inv1);
         }
     } else {
-        float* part = a.scratch + (((size_t)blockIdx.y * gridDim.x + blockIdx.x) * a.pieces + blockIdx.z) * 16 * (DV + 2);
+        if (a.cluster) __syncthreads();                 // everybody is done with the stages: the rows go there
+        float* rows = reinterpret_cast<float*>(kbuf);
+        float* part = a.cluster ? rows : a.scratch + (((size_t)blockIdx.y * gridDim.x + blockIdx.x) * a.pieces + blockIdx.z) * 16 * (DV + 2);
         float* p0 = part + g * (DV + 2);
         float* p1 = part + (g + 8) * (DV + 2);
         if (warp == 0 && c == 0) {
@@ -525,6 +532,41 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
             const int col = col0 + n * 8 + 2 * c;
             *reinterpret_cast<float2*>(p0 + col) = make_float2(oacc[n][0], oacc[n][1]);
             *reinterpret_cast<float2*>(p1 + col) = make_float2(oacc[n][2], oacc[n][3]);
+        }
+        if (a.cluster) {
+            cluster_sync_all();
+            const int heads = min(16, nh - head0);
+            for (int r = blockIdx.z; r < heads; r += a.pieces) {       // the same for all threads of the CTA
+                const float* b = rows + r * (DV + 2);
+                // lane p holds piece p's maximum and denominator
+                const float pm = lane < a.pieces ? ld_dsmem(b + DV, (uint32_t)lane) : -INFINITY;
+                const float pl = lane < a.pieces ? ld_dsmem(b + DV + 1, (uint32_t)lane) : 0.f;
+                const float m = warp_max(pm);
+                const float pf = pm == -INFINITY ? 0.f : exp2f(pm - m);
+                const float l = warp_sum(pl * pf);
+                const float inv = (l > 0.f ? 1.0f / l : 0.f) * latent_gate(a.gate, a.gate_stride, q_row0, head0 + r);
+                bf16* o = a.out + ((size_t)q_row0 * nh + head0 + r) * DV;
+#pragma unroll 1
+                for (int c0 = 0; c0 < DV; c0 += 256) {
+                    const int col = c0 + 2 * (int)threadIdx.x;
+                    const bool in = col < DV;
+                    float2 x[16];
+#pragma unroll
+                    for (int p = 0; p < 16; ++p) {
+                        x[p].x = in && p < a.pieces ? ld_dsmem(b + col, (uint32_t)p) : 0.f;
+                        x[p].y = in && p < a.pieces ? ld_dsmem(b + col + 1, (uint32_t)p) : 0.f;
+                    }
+                    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+                    for (int p = 0; p < 16; ++p) {
+                        const float f = __shfl_sync(0xffffffffu, pf, p);
+                        s0 = fmaf(x[p].x, f, s0);
+                        s1 = fmaf(x[p].y, f, s1);
+                    }
+                    if (in) *reinterpret_cast<uint32_t*>(o + col) = pack_bf16(s0 * inv, s1 * inv);
+                }
+            }
+            cluster_sync_all();        // nobody leaves while its rows may still be read
         }
     }
     pdl_trigger();
@@ -541,9 +583,10 @@ int launch_latent_decode(const LatentArgs& a, dim3 grid, cudaStream_t stream) {
     static size_t allowed = 0;
     if (smem > allowed) {
         cudaFuncSetAttribute(latent_decode_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(latent_decode_kernel<DV>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         allowed = smem;
     }
-    rlis_launch(latent_decode_kernel<DV>, grid, 128, smem, stream, a);
+    rlis_launch_cluster(latent_decode_kernel<DV>, grid, 128, smem, stream, dim3(1, 1, a.cluster ? grid.z : 1u), a);
     return RLIS_LAUNCH_CHECK();
 }
 
@@ -625,7 +668,7 @@ extern "C" int rlis_attention_latent_prefill(const void* qa, int q_bf16, const v
     if (n_tiles <= 0) return 0;
     if (!rlis_attention_latent_mma_takes(dk, dv) || n_tiles > 65535 || nh <= 0) return RLIS_ERR_UNSUPPORTED;
     LatentArgs a = {qa, (const bf16*)cache, (bf16*)out, sinks, tiles, cu_seqlens, ctx_lens, block_tables, nullptr,
-                    nullptr, nullptr, max_blocks, nh, dk, page_size, window, 1, 0, scale, q_bf16, (const bf16*)gate, gate_stride};
+                    nullptr, nullptr, max_blocks, nh, dk, page_size, window, 1, 0, scale, q_bf16, 0, (const bf16*)gate, gate_stride};
     dim3 grid(nh, n_tiles);
     switch (dv) {
         case 64: return launch_latent<64>(a, grid, stream);
@@ -635,7 +678,10 @@ extern "C" int rlis_attention_latent_prefill(const void* qa, int q_bf16, const v
     }
 }
 
-// pieces > 1: `scratch` holds n_dec * ceil(nh / 16) * pieces * 16 * (dv + 2) floats and the context
+// Up to this many pieces need no scratch.
+extern "C" int rlis_attention_latent_decode_cluster() { return LATENT_CLUSTER_PIECES; }
+
+// pieces beyond that: `scratch` holds n_dec * ceil(nh / 16) * pieces * 16 * (dv + 2) floats and the context
 // is cut into pieces of `piece_keys` keys (a multiple of 64).
 extern "C" int rlis_attention_latent_decode(const void* qa, int q_bf16, const void* cache, void* out, const float* sinks,
                                             float* scratch, const int* dec_rows, const int* dec_seqs,
@@ -645,12 +691,12 @@ extern "C" int rlis_attention_latent_decode(const void* qa, int q_bf16, const vo
                                             cudaStream_t stream) {
     if (n_dec <= 0) return 0;
     if (!rlis_attention_latent_mma_takes(dk, dv) || n_dec > 65535 || nh <= 0 || pieces < 1 || pieces > 4096 ||
-        (pieces > 1 && (scratch == nullptr || piece_keys <= 0 || piece_keys % LF_BN_MAX)))
+        (pieces > LATENT_CLUSTER_PIECES && scratch == nullptr) || (pieces > 1 && (piece_keys <= 0 || piece_keys % LF_BN_MAX)))
         return RLIS_ERR_UNSUPPORTED;
     if (pieces == 1) piece_keys = 0x40000000;
     LatentArgs a = {qa, (const bf16*)cache, (bf16*)out, sinks, nullptr, nullptr, ctx_lens, block_tables, dec_rows,
                     dec_seqs, scratch, max_blocks, nh, dk, page_size, window, pieces, piece_keys, scale, q_bf16,
-                    (const bf16*)gate, gate_stride};
+                    pieces > 1 && pieces <= LATENT_CLUSTER_PIECES ? 1 : 0, (const bf16*)gate, gate_stride};
     const int head_tiles = (nh + 15) / 16;
     dim3 grid(head_tiles, n_dec, pieces);
     int rc;
@@ -660,7 +706,7 @@ extern "C" int rlis_attention_latent_decode(const void* qa, int q_bf16, const vo
         case 256: rc = launch_latent_decode<256>(a, grid, stream); break;
         default: rc = launch_latent_decode<512>(a, grid, stream); break;
     }
-    if (rc != 0 || pieces == 1) return rc;
+    if (rc != 0 || pieces == 1 || a.cluster) return rc;
     dim3 mgrid(nh, n_dec);
     switch (dv) {
         case 64: rlis_launch(latent_merge_kernel<64>, mgrid, 32, (size_t)2 * pieces * sizeof(float), stream, (const float*)scratch, (bf16*)out, dec_rows, nh, head_tiles, pieces, (const bf16*)gate, gate_stride); break;

@@ -219,14 +219,26 @@ def gemm_f32_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> tor
     return out
 
 
+def _small_rows(a: torch.Tensor) -> bool:
+    """Whether the rows of a [T, H, K] can be read in vectors of 8."""
+    return a.shape[2] % 8 == 0 and a.stride(2) == 1 and a.stride(0) % 8 == 0 and a.stride(1) % 8 == 0 and a.data_ptr() % 16 == 0
+
+
 def per_head_linear(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
     """out[t, h, :] = w[h] @ a[t, h, :]: one small product a head (a [T, H, K] and out [T, H, N] may be
-    slices of wider rows, w [H, N, K]).  float32: this package's FFMA kernel; bfloat16 operands: the
+    slices of wider rows, w [H, N, K]).  float32: this package's FFMA kernel; bfloat16 operands: up to 16 rows
+    on 16-byte boundaries this package's kernel that reads every weight once (`rlis_per_head_small`), else the
     library's batched GEMM with float32 accumulation, into `out`'s element type."""
     if a.dtype == torch.float32:
         return gemm_f32_batched(a, w, out)
     if a.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or not a.is_cuda:
         raise KernelError(f"per_head_linear: expected float32 or bfloat16 operands on the device, got {a.dtype}, {w.dtype}")
+    if (a.shape[0] <= DECODE_GEMM_ROWS and out.dtype == torch.bfloat16 and w.is_contiguous() and _small_rows(a) and w.data_ptr() % 16 == 0
+            and out.stride(2) == 1):
+        check(lib().rlis_per_head_small(a.data_ptr(), a.stride(0), a.stride(1), w.data_ptr(), out.data_ptr(), out.stride(0),
+                                        out.stride(1), a.shape[0], w.shape[0], w.shape[1], w.shape[2], _stream()), "per_head_small")
+        _count("per_head_small")
+        return out
     # [H, T, N] view of `out` (rows H * width apart, heads one head's width apart): the library writes it in place
     if out.dtype != a.dtype:
         torch.bmm(a.transpose(0, 1), w.transpose(1, 2), out_dtype=out.dtype, out=out.transpose(0, 1))
@@ -641,6 +653,37 @@ def latent_q_rope(q: torch.Tensor, qa: torch.Tensor, inv_freq: torch.Tensor, rot
     return qa
 
 
+def latent_step_takes(q: torch.Tensor, qa_dtype, k_fold: torch.Tensor, n_heads: int, d_plain: int, rot: int) -> bool:
+    """Whether `latent_step` takes a step's queries [T, nh (d_plain + rot)] (a column slice of wider rows)."""
+    return (qa_dtype == torch.bfloat16 and q.dtype == torch.bfloat16 and q.shape[0] <= DECODE_GEMM_ROWS and k_fold.data_ptr() % 16 == 0
+            and _small_rows(q.unflatten(1, (n_heads, d_plain + rot))[:, :, :d_plain]))
+
+
+def latent_step(q: torch.Tensor, z: torch.Tensor, k_fold: torch.Tensor, weight: torch.Tensor, eps: float, inv_freq: torch.Tensor,
+                rot_dims: int, magnitude: float, positions: torch.Tensor, slots, cache: torch.Tensor, qa: torch.Tensor, n_heads: int,
+                d_plain: int, rank: int, page_size: int) -> torch.Tensor:
+    """`latent_kv_store` of z, the queries' plain parts through `k_fold` [nh, rank, d_plain], and `latent_q_rope`, in one launch
+    for up to 16 tokens of bfloat16 (see `latent_step_takes`).  q and z may be column slices of wider rows; qa [T, nh (rank +
+    rot)]; slots None: nothing is stored."""
+    T, rot = z.shape[0], z.shape[1] - rank
+    _req(k_fold, "k_fold", torch.bfloat16, (n_heads, rank, d_plain))
+    _req(weight, "weight", torch.float32, (rank,))
+    _req(inv_freq, "inv_freq", torch.float32, (rot_dims // 2,))
+    _req(positions, "positions", torch.int32, (T,))
+    _req(qa, "qa", torch.bfloat16, (T, n_heads * (rank + rot)))
+    _req(cache, "cache", torch.bfloat16, (None, 1, page_size, rank + rot))
+    if tuple(q.shape) != (T, n_heads * (d_plain + rot)) or q.dtype != torch.bfloat16 or z.dtype != torch.bfloat16 or q.stride(1) != 1 or z.stride(1) != 1:
+        raise KernelError("latent_step: q and z must be bfloat16 rows with unit stride")
+    if slots is not None:
+        _req(slots, "slots", torch.int32, (T,))
+    check(lib().rlis_latent_step(q.data_ptr(), q.stride(0), z.data_ptr(), z.stride(0), k_fold.data_ptr(), weight.data_ptr(),
+                                 inv_freq.data_ptr(), positions.data_ptr(), slots.data_ptr() if slots is not None else None,
+                                 cache.data_ptr(), qa.data_ptr(), T, n_heads, d_plain, rank, rot, int(rot_dims), float(magnitude),
+                                 float(eps), _stream()), "latent_step")
+    _count("latent_step")
+    return qa
+
+
 LATENT_DECODE_CTAS_PER_SM = 2   # debug switch "latent_ctas_per_sm": how full decode attention over latents fills the SMs
 LATENT_MMA = True          # debug switch "latent_mma": 0 takes the one-warp-a-row kernel for every size
 
@@ -723,7 +766,7 @@ def attention_latent(qa: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, s
         if n_dec:
             pieces, keys = latent_decode_pieces(n_dec, n_heads, step.max_decode_ctx, window)
             scratch = None
-            if pieces > 1:
+            if pieces > lib().rlis_attention_latent_decode_cluster():
                 scratch = step.buffer("latent_partial", (n_dec * ((n_heads + 15) // 16) * pieces * 16 * (rank + 2),),
                                       torch.float32)
             check(lib().rlis_attention_latent_decode(
@@ -732,7 +775,7 @@ def attention_latent(qa: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, s
                 step.dec_seqs.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1], n_dec,
                 n_heads, dk, rank, page_size, float(scale), int(window), pieces, keys, gp, gs, _stream()),
                 "attention_latent_decode")
-            _count("attention_latent.decode.mma" + (".split" if pieces > 1 else ""))
+            _count("attention_latent.decode.mma" + (".split" if scratch is not None else ".cluster" if pieces > 1 else ""))
         if n_tiles:
             check(lib().rlis_attention_latent_prefill(
                 qa.data_ptr(), q16, cache.data_ptr(), out.data_ptr(), sink_ptr, step.prefill_tiles.data_ptr(), n_tiles,

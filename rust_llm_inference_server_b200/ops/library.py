@@ -47,6 +47,9 @@ SIGNATURES = {
     "rlis_attention_latent_mma_takes": [I, I],
     "rlis_attention_latent_prefill": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, F, I, P, LL, P],
     "rlis_attention_latent_decode": [P, I, P, P, P, P, P, P, P, P, I, I, I, I, I, I, F, I, I, I, P, LL, P],
+    "rlis_attention_latent_decode_cluster": [],
+    "rlis_per_head_small": [P, LL, LL, P, P, LL, LL, I, I, I, I, P],
+    "rlis_latent_step": [P, LL, P, LL, P, P, P, P, P, P, P, I, I, I, I, I, I, F, F, P],
     "rlis_lightning_scan": [P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, I, P, I, P],
     "rlis_recurrence_inputs": [P, LL, I, I, I, P, I, I, I, I, P, I, P, F, I, P, P, I, P],
     "rlis_recurrence_scan_rows": [P, LL, I, I, I, P, P, P, P, P, P, I, I, I, I, P, I, F, P, P, I, P],

@@ -108,30 +108,18 @@ class LatentAttention(ProjectedMixer):
         T, H = proj.shape[0], s.n_heads
         dk = s.kv_rank + s.rot_dim
         stores = self.own_kv and writes_cache
-        cq = step.buffer("latent_cq", (T, s.q_rank), self.dtype) if self.q_latent else None
-        if stores:
-            # one launch: the kv latent's norm, the shared key part's rotation, the paged write, and the
-            # query latent's norm
-            q_args = dict(q_latent=proj[:, :s.q_rank], q_weight=self.q_norm, q_out=cq) if self.q_latent else {}
-            with span("latent norms + rope + cache write"):
-                ops.latent_kv_store(proj[:, self.kv_off:self.kv_off + dk], self.kv_norm, self.eps, self.inv_freq, self.rot_dims,
-                                    self.magnitude, step.positions, step.slots[cache.group], cache.k, s.kv_rank,
-                                    cache.page_size, **q_args)
-        elif self.q_latent:
-            with span("q latent norm"):
-                ops.act_norm(proj[:, :s.q_rank], self.q_norm, self.eps, cq)
-        q = proj[:, :self.kv_off]
-        if self.q_latent:
-            with span("q up proj"):
-                q = ops.linear(cq, self.w_q_up)
         # float32, or bfloat16 when the whole step goes to the tensor-core attention kernels
         qa_dtype = ops.latent_attention_queries_dtype(step, self.dtype, dk, s.kv_rank)
         qa = step.buffer("latent_qa" if qa_dtype == torch.float32 else "latent_qa16", (T, H * dk), qa_dtype)
-        with span("q fold + rope"):
-            ops.per_head_linear(q.unflatten(1, (H, s.dim + s.rot_dim))[:, :, :s.dim], self.w_k_fold,
-                                qa.view(T, H, dk)[:, :, :s.kv_rank])
-            ops.latent_q_rope(q, qa, self.inv_freq, self.rot_dims, self.magnitude, step.positions, H, s.dim,
-                              s.rot_dim, s.kv_rank)
+        z = proj[:, self.kv_off:self.kv_off + dk]
+        q = proj[:, :self.kv_off]
+        if not self.q_latent and self.own_kv and ops.latent_step_takes(q, qa_dtype, self.w_k_fold, H, s.dim, s.rot_dim):
+            with span("latent norm + rope + cache write, q fold + rope"):
+                ops.latent_step(q, z, self.w_k_fold, self.kv_norm, self.eps, self.inv_freq, self.rot_dims, self.magnitude,
+                                step.positions, step.slots[cache.group] if stores else None, cache.k, qa, H, s.dim, s.kv_rank,
+                                cache.page_size)
+        else:
+            self._queries(proj, q, z, qa, step, cache, stores)
         lat = step.buffer("latent_o", (T, H * s.kv_rank), self.dtype)
         gate = proj[:, self.g_off:self.g_off + H] if s.head_gate is not None else None
         with span("attention"):
@@ -141,6 +129,29 @@ class LatentAttention(ProjectedMixer):
         with span("v up proj"):
             ops.per_head_linear(lat.view(T, H, s.kv_rank), self.w_v_up, o.view(T, H, s.v_dim))
         return o
+
+    def _queries(self, proj, q, z, qa, step, cache, stores) -> None:
+        """The cached row of every token, and `qa`, operation by operation."""
+        s = self.spec
+        T, H = proj.shape[0], s.n_heads
+        cq = step.buffer("latent_cq", (T, s.q_rank), self.dtype) if self.q_latent else None
+        if stores:
+            # one launch: the kv latent's norm, the shared key part's rotation, the paged write, and the
+            # query latent's norm
+            q_args = dict(q_latent=q, q_weight=self.q_norm, q_out=cq) if self.q_latent else {}
+            with span("latent norms + rope + cache write"):
+                ops.latent_kv_store(z, self.kv_norm, self.eps, self.inv_freq, self.rot_dims, self.magnitude, step.positions,
+                                    step.slots[cache.group], cache.k, s.kv_rank, cache.page_size, **q_args)
+        elif self.q_latent:
+            with span("q latent norm"):
+                ops.act_norm(q, self.q_norm, self.eps, cq)
+        if self.q_latent:
+            with span("q up proj"):
+                q = ops.linear(cq, self.w_q_up)
+        with span("q fold + rope"):
+            ops.per_head_linear(q.unflatten(1, (H, s.dim + s.rot_dim))[:, :, :s.dim], self.w_k_fold,
+                                qa.view(T, H, -1)[:, :, :s.kv_rank])
+            ops.latent_q_rope(q, qa, self.inv_freq, self.rot_dims, self.magnitude, step.positions, H, s.dim, s.rot_dim, s.kv_rank)
 
 
 register_mixer("latent_attention", LatentAttention)

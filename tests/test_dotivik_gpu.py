@@ -263,9 +263,7 @@ def test_attention_of_two_maps_far_keys_page_borders_and_windows(dtype, H, G, d,
     if dtype == BF16 and ops.difference_prefill_takes_mma(dtype, d, dv, page):
         assert "attention_difference.prefill.tcgen05" in ran
     if dtype == BF16 and ops.difference_decode_takes_mma(dtype, H, G, d, dv):
-        assert ran & {"attention_difference.decode.mma", "attention_difference.decode.mma.split"}
-        if not window:
-            assert "attention_difference.decode.mma.split" in ran
+        assert "attention_difference.decode.mma" + (".cluster" if not window else "") in ran
     ops.check_device_errors()
 
 
@@ -326,8 +324,81 @@ def test_latent_attention_with_a_gate_at_window_edges(dtype, H, rank, rot, windo
     want *= P.sigmoid(host(gate))[:, :, None]
     np.testing.assert_allclose(host(out).reshape(T, H, rank), want, rtol=0, atol=3e-5 if dtype == torch.float32 else 0.04)
     if dtype == BF16 and ops.latent_attention_takes_mma(dtype, dk, rank):
-        split = window == 0 or window >= 256
-        assert ops.launches_by_kernel.get("attention_latent.decode.mma" + (".split" if split else ""))
+        assert ops.launches_by_kernel.get("attention_latent.decode.mma" + (".cluster" if window == 0 or window >= 256 else ""))
+
+
+@pytest.mark.parametrize("H,G,d,dv", [(2, 1, 64, 128), (1, 1, 40, 56)])
+def test_a_single_token_far_into_a_long_context(H, G, d, dv):
+    """More pieces than a cluster holds: they are merged by a second kernel."""
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(d)
+    page, ctx = 64, [20000, 300]
+    st = hand_step(ctx, [1, 1], page, 330, rng)
+    keys, vals = [rng.standard_normal((c, G, 2 * d)) for c in ctx], [rng.standard_normal((c, G, dv)) for c in ctx]
+    q = rng.standard_normal((2, H, 2, d))
+    for h in range(H):                                      # a key in the first piece and one in the middle
+        for m, j in ((0, 3), (1, 11111)):
+            k = keys[0][j, h // (H // G), m * d:(m + 1) * d]
+            q[0, h, m] = k * (11.0 / 0.1 / float(k @ k))
+    q = dev(q.reshape(2, -1), BF16)
+    kr, vr = [host(dev(k, BF16)) for k in keys], [host(dev(v, BF16)) for v in vals]
+    kc, vc = (torch.full((330, G, page, w), 50.0, dtype=BF16, device="cuda") for w in (2 * d, dv))
+    for b, (k, v) in enumerate(zip(kr, vr)):
+        for p in range(0, ctx[b], page):
+            for pool, x in ((kc, k), (vc, v)):
+                part = dev(x[p:p + page], BF16).transpose(0, 1)
+                pool[int(st.host_tables[b, p // page]), :, :part.shape[1]] = part
+    out = torch.full((2, H * dv), float("nan"), dtype=BF16, device="cuda")
+    ops.launches_by_kernel.clear()
+    ops.attention_difference(q, kc, vc, out, None, st, 0, H, G, d, dv, page, 0.1, 50.0, 0.5, 0.7, 1e-5)
+    want = plain_difference_rows(host(q).reshape(2, H, 2, d), [k.reshape(-1, G, 2, d) for k in kr], vr, 0.1, 50.0, 0, 0.5, 0.3, 1e-5,
+                                 np.full((2, H), 60.0), st, H, G)
+    np.testing.assert_allclose(host(out).reshape(2, H, dv), want, rtol=0, atol=0.05)
+    assert ops.launches_by_kernel == {"attention_difference.decode.mma.split": 1}
+
+
+@pytest.mark.parametrize("T,H,N,K", [(1, 3, 40, 16), (8, 6, 64, 32), (16, 16, 512, 128), (9, 2, 24, 512), (5, 16, 128, 512), (3, 1, 10, 264),
+                                     (16, 5, 72, 200)])
+def test_small_product_a_head(T, H, N, K):
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(N + K)
+    wide = dev(rng.standard_normal((T, H * (K + 8) + 16)), BF16)
+    a = wide[:, 8:8 + H * (K + 8)].unflatten(1, (H, K + 8))[:, :, :K]                # slices of wider rows
+    w = dev(rng.standard_normal((H, N, K)) / np.sqrt(K), BF16)
+    out = torch.full((T, H, N + 3), 7.0, dtype=BF16, device="cuda")
+    ops.launches_by_kernel.clear()
+    ops.per_head_linear(a, w, out[:, :, :N])
+    assert ops.launches_by_kernel == {"per_head_small": 1}
+    np.testing.assert_allclose(host(out[:, :, :N]), np.einsum("thk,hnk->thn", host(a), host(w)), rtol=1e-2, atol=0.02)
+    assert float((out[:, :, N:].float() - 7.0).abs().max()) == 0.0
+
+
+@pytest.mark.parametrize("T,H,d,rank,rot", [(1, 3, 16, 64, 16), (8, 16, 128, 512, 64), (16, 6, 32, 128, 32), (5, 2, 8, 64, 0)])
+def test_latent_rows_and_folded_queries_in_one_launch(T, H, d, rank, rot):
+    """Against the operations one by one: the same rows in the cache and nothing beside them, the same queries."""
+    from rust_llm_inference_server_b200 import ops
+    rng = np.random.default_rng(T + d)
+    page = 16
+    ctx = [int(c) for c in rng.integers(1, 60, size=T)]
+    st = hand_step(ctx, [1] * T, page, 4 * T + 2, rng)
+    n_q = H * (d + rot)
+    proj = dev(rng.standard_normal((T, n_q + rank + rot + 8)), BF16)
+    q, z = proj[:, :n_q], proj[:, n_q:n_q + rank + rot]
+    fold, w = dev(rng.standard_normal((H, rank, d)) / np.sqrt(d), BF16), dev(1 + 0.2 * rng.standard_normal(rank))
+    freq = dev(100.0 ** (-2.0 * np.arange(rot // 2) / max(rot, 1)))
+    caches = [torch.full((4 * T + 2, 1, page, rank + rot), 7.0, dtype=BF16, device="cuda") for _ in range(2)]
+    qas = [torch.empty((T, H * (rank + rot)), dtype=BF16, device="cuda") for _ in range(2)]
+    assert ops.latent_step_takes(q, BF16, fold, H, d, rot)
+    ops.latent_step(q, z, fold, w, 1e-5, freq, rot, 1.0, st.positions, st.slots[0], caches[0], qas[0], H, d, rank, page)
+    ops.latent_kv_store(z, w, 1e-5, freq, rot, 1.0, st.positions, st.slots[0], caches[1], rank, page)
+    torch.bmm(q.unflatten(1, (H, d + rot))[:, :, :d].transpose(0, 1), fold.transpose(1, 2), out=qas[1].view(T, H, -1)[:, :, :rank].transpose(0, 1))
+    if rot:
+        ops.latent_q_rope(q, qas[1], freq, rot, 1.0, st.positions, H, d, rot, rank)
+    assert torch.equal(caches[0], caches[1])
+    np.testing.assert_allclose(host(qas[0]), host(qas[1]), rtol=1e-2, atol=0.02)
+    before = caches[0].clone()
+    ops.latent_step(q, z, fold, w, 1e-5, freq, rot, 1.0, st.positions, None, caches[0], qas[0], H, d, rank, page)
+    assert torch.equal(caches[0], before)
 
 
 # ---- whole models ------------------------------------------------------------------------------
@@ -413,6 +484,7 @@ def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens
         assert ok, f"{which} {dtype}: {fam} differs from whole by {what}"
     launched = ops.launches_by_kernel
     needed = {"layer_norm", "layer_norm.rows", "qk_norm_store.rot", "latent_kv_store"}
+    assert max(lens) > 128
     if dtype == "float32":
         needed |= {"attention_difference", "attention_latent"}
     elif U.CONFIGS[which]["width"] % 8 == 0:
@@ -420,9 +492,9 @@ def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens
         if U.CONFIGS[which].get("loop"):
             needed |= {"stream_gemm.sink.centred"}
         if which != "F":
-            needed |= {"attention_difference.decode.mma", "attention_difference.prefill.tcgen05"}
+            needed |= {"attention_difference.decode.mma.cluster", "attention_difference.prefill.tcgen05"}
         if which in ("C", "E"):
-            needed |= {"attention_latent.decode.mma", "attention_latent.prefill.mma", "gemm_tcgen05.glu4"}
+            needed |= {"attention_latent.decode.mma", "attention_latent.prefill.mma", "gemm_tcgen05.glu4", "latent_step", "per_head_small"}
     assert needed <= set(launched), f"never launched {sorted(needed - set(launched))}"
 
 

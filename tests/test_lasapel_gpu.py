@@ -287,9 +287,9 @@ def test_tensor_core_attention_over_latents(H, rank, rot, window, use_sinks):
     ops.attention_latent(dev(qa.reshape(step.n_tokens, -1)), cache, out, step, 0, H, rank, page, 0.3,
                          dev(sinks) if use_sinks else None, window)
     # (a short window is one piece)
-    split = ops.latent_decode_pieces(step.n_decode, H, step.max_decode_ctx, window)[0] > 1
-    assert split or window and window < 256
-    assert ops.launches_by_kernel.get("attention_latent.decode.mma" + (".split" if split else ""))
+    pieces = ops.latent_decode_pieces(step.n_decode, H, step.max_decode_ctx, window)[0]
+    assert pieces > 1 or window and window < 256
+    assert ops.launches_by_kernel.get("attention_latent.decode.mma" + (".split" if pieces > 16 else ".cluster" if pieces > 1 else ""))
     assert ops.launches_by_kernel.get("attention_latent.prefill.mma")
     np.testing.assert_allclose(out.float().cpu().numpy().reshape(step.n_tokens, H, rank), want, rtol=0, atol=2e-2)
     # queries that are bfloat16 already (as the mixer hands them over) are copied as they are
