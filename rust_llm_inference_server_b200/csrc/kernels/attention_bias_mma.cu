@@ -573,6 +573,8 @@ __global__ __launch_bounds__(128) void attn_bias_decode_merge_kernel(
 }
 
 constexpr int MAX_CLUSTER_PIECES = 16;
+constexpr int TABLE_SLICE = 512;       // page numbers of a CTA's piece kept in shared memory (longer pieces look them up as they go)
+template <int DV> constexpr size_t difference_smem_bytes() { return decode_smem_bytes<128, DV>() + TABLE_SLICE * sizeof(int); }
 struct DiffDecode {
     const bf16 *q, *k_cache, *v_cache;
     bf16* out;
@@ -671,6 +673,14 @@ __global__ __launch_bounds__(THREADS) void attn_difference_decode_kernel(const D
     const int per = (t_all + a.pieces - 1) / a.pieces;
     const int kt0 = t_first + piece * per, kt1 = min(kt0 + per, t_first + t_all);
     const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
+    // a look-up in global memory before every copy is most of a tile's time: the piece's page numbers come to shared memory once
+    int* pages = reinterpret_cast<int*>(sbase + (size_t)DEC_STAGES * Stage<D, DV>::ELEMS);
+    const int p_first = kt0 * BN / page_size, p_count = kt1 > kt0 ? (min(kt1 * BN, k_hi) - 1) / page_size - p_first + 1 : 0;
+    const bool sliced = p_count <= TABLE_SLICE;
+    if (sliced) {
+        for (int i = threadIdx.x; i < p_count; i += THREADS) pages[i] = table[p_first + i];
+        __syncthreads();
+    }
 
     auto issue = [&](int kt, int stage) {
         bf16* ks_ = sbase + (size_t)stage * Stage<D, DV>::ELEMS;
@@ -688,7 +698,8 @@ __global__ __launch_bounds__(THREADS) void attn_difference_decode_kernel(const D
             size_t off = 0;
             if (valid) {
                 const int pi = page_shift >= 0 ? key >> page_shift : key / page_size;
-                const size_t r = ((size_t)table[pi] * a.nkv + kvh) * page_size + (key - pi * page_size);
+                const int page = sliced ? pages[pi - p_first] : table[pi];
+                const size_t r = ((size_t)page * a.nkv + kvh) * page_size + (key - pi * page_size);
                 off = is_v ? r * dv + col : (r * 2 + c16 / (CK / 2)) * d + col;
             }
             if (is_v) cp_async16(vs_ + kin * SV + c16 * 8, a.v_cache + off, valid);
@@ -979,6 +990,42 @@ extern "C" int rlis_attention_difference_decode_takes(int nh, int nkv, int d, in
 // Width of a value row in the partial sums (values are padded to it).
 extern "C" int rlis_attention_difference_decode_width(int dv) { return dv <= 64 ? 64 : 128; }
 
+static void raise_difference_limits() {
+    static bool done = false;
+    if (done) return;
+    cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)difference_smem_bytes<64>());
+    cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)difference_smem_bytes<128>());
+    cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    done = true;
+}
+
+// How many clusters of `pieces` CTAs the device holds at a time (0: none, or the query failed).
+extern "C" int rlis_attention_difference_decode_resident(int dv, int pieces) {
+    if (pieces < 1 || pieces > MAX_CLUSTER_PIECES) return 0;
+    raise_difference_limits();
+    const bool narrow = rlis_attention_difference_decode_width(dv) == 64;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(1, 1, (unsigned)pieces);
+    cfg.blockDim = THREADS;
+    cfg.dynamicSmemBytes = narrow ? difference_smem_bytes<64>() : difference_smem_bytes<128>();
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = 1;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = (unsigned)pieces;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    int n = 0;
+    const cudaError_t e = narrow ? cudaOccupancyMaxActiveClusters(&n, attn_difference_decode_kernel<64>, &cfg)
+                                 : cudaOccupancyMaxActiveClusters(&n, attn_difference_decode_kernel<128>, &cfg);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        return 0;
+    }
+    return n;
+}
+
 // Up to this many pieces of a context merge inside a cluster.
 extern "C" int rlis_attention_difference_decode_cluster() { return MAX_CLUSTER_PIECES; }
 
@@ -994,22 +1041,15 @@ extern "C" int rlis_attention_difference_decode(const void* q, const void* k_cac
         (pieces > MAX_CLUSTER_PIECES && partial == nullptr) ||
         ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) != 0)
         return RLIS_ERR_UNSUPPORTED;
-    static bool done = false;
-    if (!done) {
-        cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<128, 64>());
-        cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)decode_smem_bytes<128, 128>());
-        cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-        done = true;
-    }
+    raise_difference_limits();
     const DiffDecode a{(const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, partial, (const bf16*)gate, gate_stride,
                        dec_rows, dec_seqs, ctx_lens, block_tables, max_blocks, nh, nkv, d, dv, page_size, window, pieces,
                        pieces > 1 && pieces <= MAX_CLUSTER_PIECES ? 1 : 0, scale, cap, lambda, out_scale, eps};
     const dim3 grid(nkv, n_dec, pieces);
     const bool narrow = rlis_attention_difference_decode_width(dv) == 64;
     const dim3 cluster(1, 1, a.cluster ? (unsigned)pieces : 1u);
-    if (narrow) rlis_launch_cluster(attn_difference_decode_kernel<64>, grid, THREADS, decode_smem_bytes<128, 64>(), stream, cluster, a);
-    else rlis_launch_cluster(attn_difference_decode_kernel<128>, grid, THREADS, decode_smem_bytes<128, 128>(), stream, cluster, a);
+    if (narrow) rlis_launch_cluster(attn_difference_decode_kernel<64>, grid, THREADS, difference_smem_bytes<64>(), stream, cluster, a);
+    else rlis_launch_cluster(attn_difference_decode_kernel<128>, grid, THREADS, difference_smem_bytes<128>(), stream, cluster, a);
     const int err = RLIS_LAUNCH_CHECK();
     if (err != 0 || pieces == 1 || a.cluster) return err;
     const int units = n_dec * nh;

@@ -24,6 +24,7 @@
 namespace {
 constexpr int LF_BN_MAX = 64;             // the longest stage: pieces of a context are multiples of it
 constexpr float LOG2E = 1.4426950408889634f;
+constexpr int LATENT_TABLE_SLICE = 256;        // page numbers of a CTA's piece kept in shared memory
 constexpr int LATENT_CLUSTER_PIECES = 16;      // up to this many pieces of a context merge inside a cluster
 
 // Barrier over the two warps of pair `p` (named barriers 1..4; 0 is __syncthreads).
@@ -361,6 +362,15 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
         }
     }
     const int kt0 = k_lo / BN, kt1 = k_hi > k_lo ? (k_hi + BN - 1) / BN : kt0;
+    // the piece's page numbers come to shared memory once, if they fit: a look-up in global memory before every stage's
+    // copies is time in which nothing is in flight
+    __shared__ int pages[LATENT_TABLE_SLICE];
+    const int p_first = k_lo / page_size, p_count = k_hi > k_lo ? (k_hi - 1) / page_size - p_first + 1 : 0;
+    const bool sliced = p_count <= LATENT_TABLE_SLICE;
+    if (sliced) {
+        for (int i = threadIdx.x; i < p_count; i += 128) pages[i] = table[p_first + i];
+        __syncthreads();
+    }
     auto issue = [&](int kt, int stage) {      // a warp copies 8 keys' rows, in runs of 512 contiguous bytes
         const int key0 = kt * BN + warp * 8;
         long long my_off = -1;
@@ -368,7 +378,7 @@ __global__ __launch_bounds__(128) void latent_decode_kernel(const LatentArgs a) 
             const int key = key0 + lane;
             if (key < k_hi && key >= k_lo) {
                 const int pi = key / page_size;
-                my_off = ((long long)table[pi] * page_size + (key - pi * page_size)) * dk;
+                my_off = ((long long)(sliced ? pages[pi - p_first] : table[pi]) * page_size + (key - pi * page_size)) * dk;
             }
         }
         bf16* dst0 = kbuf + ((size_t)stage * BN + warp * 8) * stride;

@@ -1746,21 +1746,31 @@ def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, 
                 and _difference_decode_sizes(int(n_heads), int(n_kv_heads), int(dim), int(v_dim)))
 
 
+@functools.lru_cache(maxsize=None)
+def _difference_clusters(v_dim: int, pieces: int) -> int:
+    return int(lib().rlis_attention_difference_decode_resident(v_dim, pieces))
+
+
 @functools.lru_cache(maxsize=4096)
-def _difference_decode_pieces(n_decode: int, n_kv_heads: int, seen: int, sms: int) -> int:
-    """Pieces a context is cut into: a CTA takes one key/value head of one request and two fit an SM, so the context is cut
-    until they about fill the SMs, in pieces of at least two tiles of 64 keys.  Up to 16 pieces merge in a cluster; more only
-    where that many would still leave every CTA a long way to go."""
-    tiles = -(-seen // 64) + 1
-    want = max(1, min(2 * sms // max(1, n_decode * n_kv_heads), tiles // 2, 64))
-    if want > 16 and tiles <= 16 * 16:
-        want = 16
-    return max(1, -(-tiles // -(-tiles // want)))
+def _difference_decode_pieces(n_decode: int, n_kv_heads: int, v_dim: int, seen: int, sms: int) -> int:
+    """Pieces a context is cut into, at least two tiles of 64 keys each: a CTA takes one key/value head of one request and the
+    pieces of up to 16 merge in a cluster, so the context is cut as finely as clusters of that size are all resident at once
+    (one that does not fit waits for a whole round: 8 requests with four heads, 35 us in clusters of 8 and 60 us in clusters of
+    9).  More pieces and a second kernel only where 16 would leave every CTA a long way to go."""
+    tiles, ctas = -(-seen // 64), max(1, n_decode * n_kv_heads)
+    most = max(1, min(2 * sms // ctas, tiles // 2))
+    if most > 16 and tiles > 16 * 16:
+        return -(-tiles // -(-tiles // min(most, 64)))
+    for want in range(min(most, 16), 1, -1):
+        pieces = -(-tiles // -(-tiles // want))
+        if ctas <= _difference_clusters(v_dim, pieces):
+            return pieces
+    return 1
 
 
-def difference_decode_pieces(n_decode: int, n_kv_heads: int, max_ctx: int, window: int = 0) -> int:
+def difference_decode_pieces(n_decode: int, n_kv_heads: int, v_dim: int, max_ctx: int, window: int = 0) -> int:
     seen = min(int(max_ctx), int(window)) if window else int(max_ctx)
-    return _difference_decode_pieces(int(n_decode), int(n_kv_heads), max(1, seen), num_sms())
+    return _difference_decode_pieces(int(n_decode), int(n_kv_heads), int(v_dim), max(1, seen), num_sms())
 
 
 def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_heads: int, n_kv_heads: int, dim: int,
@@ -1789,7 +1799,7 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
     n_dec = step.n_decode if difference_decode_takes_mma(q.dtype, n_heads, n_kv_heads, dim, v_dim) else 0
     n_tiles = step.n_prefill_tiles if difference_prefill_takes_mma(q.dtype, dim, v_dim, page_size) else 0
     if n_dec:
-        pieces = difference_decode_pieces(n_dec, n_kv_heads, step.max_decode_ctx, window)
+        pieces = difference_decode_pieces(n_dec, n_kv_heads, v_dim, step.max_decode_ctx, window)
         scratch = step.buffer("attn_partial", (n_dec * n_heads * 2 * pieces * (lib().rlis_attention_difference_decode_width(v_dim) + 2),),
                               torch.float32) if pieces > lib().rlis_attention_difference_decode_cluster() else None
         check(lib().rlis_attention_difference_decode(

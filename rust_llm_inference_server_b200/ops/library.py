@@ -67,6 +67,7 @@ SIGNATURES = {
     "rlis_attention_difference_decode_takes": [I, I, I, I],
     "rlis_attention_difference_decode_width": [I],
     "rlis_attention_difference_decode_cluster": [],
+    "rlis_attention_difference_decode_resident": [I, I],
     "rlis_moe_route": [P, P, P, P, P, P, I, I, I, I, F, P, I, I, I, I, I, P],
     "rlis_moe_align": [P, P, P, P, I, I, I, I, P],
     "rlis_moe_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, F, F, F, LL, I, I, P],

@@ -79,7 +79,7 @@ class DifferenceAttention(ProjectedMixer):
         s = self.spec
         if not step.n_decode or not ops.difference_decode_takes_mma(self.dtype, s.n_heads, s.n_kv_heads, s.dim, s.v_dim):
             return None
-        return ops.difference_decode_pieces(step.n_decode, s.n_kv_heads, step.max_decode_ctx, self.window)
+        return ops.difference_decode_pieces(step.n_decode, s.n_kv_heads, s.v_dim, step.max_decode_ctx, self.window)
 
     def mix(self, proj, step, cache, state, writes_cache=True):
         s = self.spec
