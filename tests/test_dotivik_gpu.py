@@ -484,7 +484,6 @@ def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens
         assert ok, f"{which} {dtype}: {fam} differs from whole by {what}"
     launched = ops.launches_by_kernel
     needed = {"layer_norm", "layer_norm.rows", "qk_norm_store.rot", "latent_kv_store"}
-    assert max(lens) > 128
     if dtype == "float32":
         needed |= {"attention_difference", "attention_latent"}
     elif U.CONFIGS[which]["width"] % 8 == 0:
@@ -492,7 +491,8 @@ def test_all_ways_of_cutting_give_the_plain_logits(model_root, which, page, lens
         if U.CONFIGS[which].get("loop"):
             needed |= {"stream_gemm.sink.centred"}
         if which != "F":
-            needed |= {"attention_difference.decode.mma.cluster", "attention_difference.prefill.tcgen05"}
+            needed |= {"attention_difference.decode.mma.cluster" if max(lens) > 190 else "attention_difference.decode.mma",
+                       "attention_difference.prefill.tcgen05"}
         if which in ("C", "E"):
             needed |= {"attention_latent.decode.mma", "attention_latent.prefill.mma", "gemm_tcgen05.glu4", "latent_step", "per_head_small"}
     assert needed <= set(launched), f"never launched {sorted(needed - set(launched))}"
