@@ -1208,6 +1208,25 @@ def dotivik_kernel_rooflines(width: int, B: int, ctx: int, T: int, pk: dict, tor
         us = timed(lambda: ops.attention_latent(qa, cache, lat, st, 0, H, rank, page, 0.07, None, 0))
         row(f"latent_attention_{kind}", us, max(keys * dk * 2 / hbm, 2 * H * keys * (dk + rank) / tf) if dec
             else 2 * H * keys * (dk + rank) / tf)
+        # single tokens: folded queries, rotations and the cached row in one launch, beside the operations one by one, and the
+        # value map, beside the library's batched product
+        if dec:
+            z = rnd(n, H * 192 + dk + 8).to(bf)
+            qz, zz, ones, f64 = z[:, :H * 192], z[:, H * 192:H * 192 + dk], torch.ones(rank, device="cuda"), torch.ones(rot // 2, device="cuda")
+            fold, wv, slots = rnd(H, rank, 128).to(bf), rnd(H, 128, rank).to(bf), torch.arange(n, device="cuda", dtype=torch.int32)
+            ov = torch.empty(n, H * 128, dtype=bf, device="cuda")
+
+            def one_by_one():
+                ops.latent_kv_store(zz, ones, 1e-5, f64, rot, 1.0, st.positions, slots, cache, rank, page)
+                torch.bmm(qz.unflatten(1, (H, 192))[:, :, :128].transpose(0, 1), fold.transpose(1, 2),
+                          out=qa.view(n, H, dk)[:, :, :rank].transpose(0, 1))
+                ops.latent_q_rope(qz, qa, f64, rot, 1.0, st.positions, H, 128, rot, rank)
+            row("latent_step_decode", timed(lambda: ops.latent_step(qz, zz, fold, ones, 1e-5, f64, rot, 1.0, st.positions, slots, cache, qa,
+                                                                    H, 128, rank, page)), H * rank * 128 * 2 / hbm)
+            row("latent_one_by_one_decode", timed(one_by_one), H * rank * 128 * 2 / hbm)
+            row("value_map_decode", timed(lambda: ops.per_head_linear(lat.view(n, H, rank), wv, ov.view(n, H, 128))), H * rank * 128 * 2 / hbm)
+            row("value_map_library_decode", timed(lambda: torch.bmm(lat.view(n, H, rank).transpose(0, 1), wv.transpose(1, 2),
+                                                                    out=ov.view(n, H, 128).transpose(0, 1))), H * rank * 128 * 2 / hbm)
         # rotation and paged write of two vectors a head, beside one with norms
         N = 2 * H * d + 2 * G * d + G * dv + H
         proj, slots = rnd(n, N + (-N % 8)).to(bf), torch.arange(n, device="cuda", dtype=torch.int32)

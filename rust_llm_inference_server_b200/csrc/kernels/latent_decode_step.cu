@@ -8,8 +8,8 @@
 //                    product does not mind in which order it sums, as long as both sides agree).  The weights do not depend on
 //                    the kernel before and are requested before the wait for it.
 //   latent_step    : the folding of the key map into the queries, the rotation of the queries' other part, and the row that the
-//                    cache keeps of every token (norm of the latent, rotation of the shared key part), in one launch: the last
-//                    CTAs of the grid take a token each.
+//                    cache keeps of every token (norm of the latent, rotation of the shared key part), in one launch: behind the
+//                    CTAs that fold come one a token for its row and some for the queries' rotations, a pair a thread.
 //
 // Sums are float32.  Rotation and norm are those of attention_latent.cu.
 #include "common.cuh"
@@ -121,6 +121,7 @@ struct LatentStep {
     bf16* cache;
     int rank, rot, rot_dims;
     float mag, eps;
+    int units;                  // of a head's rotated part: its pairs, and the entries that pass
 };
 
 __device__ __forceinline__ float turned(const bf16* x, int i, int rot_dims, const float* inv_freq, float pos, float mag) {
@@ -141,6 +142,25 @@ __global__ __launch_bounds__(128) void latent_step_kernel(const LatentStep s) {
         return;
     }
     pdl_wait_and_trigger();
+    if ((int)blockIdx.x >= s.fold_ctas + s.fold.T) {
+        const int idx = (blockIdx.x - s.fold_ctas - s.fold.T) * 128 + threadIdx.x, u = idx % s.units, th = idx / s.units;
+        if (th >= s.fold.T * s.fold.H) return;
+        const int t = th / s.fold.H, h = th - t * s.fold.H, half = s.rot_dims / 2;
+        const bf16* x = s.q_rot + (size_t)t * s.fold.a_row + (size_t)h * s.fold.a_head;
+        bf16* o = s.fold.out + (size_t)t * s.fold.o_row + (size_t)h * s.fold.o_head + s.rank;
+        if (u >= half) {
+            o[half + u] = x[half + u];
+            return;
+        }
+        float sn, cs;
+        sincosf((float)s.positions[t] * s.inv_freq[u], &sn, &cs);
+        sn *= s.mag;
+        cs *= s.mag;
+        const float a = __bfloat162float(x[u]), b = __bfloat162float(x[u + half]);
+        o[u] = __float2bfloat16_rn(rope_first(a, b, cs, sn));
+        o[u + half] = __float2bfloat16_rn(rope_second(a, b, cs, sn));
+        return;
+    }
     __shared__ float scratch[33];
     const int t = blockIdx.x - s.fold_ctas;
     const float pos = (float)s.positions[t];
@@ -158,11 +178,6 @@ __global__ __launch_bounds__(128) void latent_step_kernel(const LatentStep s) {
         for (int i = threadIdx.x; i < s.rank; i += 128) row[i] = __float2bfloat16_rn(__bfloat162float(zr[i]) * r * s.w[i]);
         for (int i = threadIdx.x; i < s.rot; i += 128)
             row[s.rank + i] = __float2bfloat16_rn(turned(zr + s.rank, i, s.rot_dims, s.inv_freq, pos, s.mag));
-    }
-    for (int idx = threadIdx.x; idx < s.fold.H * s.rot; idx += 128) {
-        const int h = idx / s.rot, i = idx - h * s.rot;
-        s.fold.out[(size_t)t * s.fold.o_row + (size_t)h * s.fold.o_head + s.rank + i] = __float2bfloat16_rn(
-            turned(s.q_rot + (size_t)t * s.fold.a_row + (size_t)h * s.fold.a_head, i, s.rot_dims, s.inv_freq, pos, s.mag));
     }
 }
 
@@ -212,6 +227,7 @@ extern "C" int rlis_latent_step(const void* q, long long q_row, const void* z, l
     s.rot_dims = rot_dims;
     s.mag = mag;
     s.eps = eps;
-    rlis_launch(latent_step_kernel, (unsigned)(s.fold_ctas + T), 128, 0, stream, s);
+    s.units = rot_dims / 2 + (rot - rot_dims);
+    rlis_launch(latent_step_kernel, (unsigned)(s.fold_ctas + T + (T * H * s.units + 127) / 128), 128, 0, stream, s);
     return RLIS_LAUNCH_CHECK();
 }
