@@ -14,13 +14,6 @@
 // heads of the group are the 16 rows of the products, so keys and values are read once a group.
 // Each of the 4 warps takes 16 of a tile's 64 keys with a running softmax of its own; the warps are
 // merged through shared memory at the end, pieces of a context by a second kernel.
-//
-// Single tokens with two maps a head (attention_difference.cu): the same, with rows 0..7 of the products the query heads' first
-// maps and rows 8..15 their second ones (groups of up to 8).  A key row is [map 1 | map 2], each padded to 64 entries; a query
-// row is its map's vector and zeros over the other's entries, so one set of products gives both maps' scores and the values
-// are multiplied once.  The maps meet where the warps (or the pieces) are merged: up to 16 pieces of a context are a
-// thread-block cluster, which merges through distributed shared memory (a CTA a head of the group, a warp a quarter of its
-// columns), more by a second kernel.
 #include "common.cuh"
 #include "mma_utils.cuh"
 #include <math.h>
@@ -572,343 +565,6 @@ __global__ __launch_bounds__(128) void attn_bias_decode_merge_kernel(
     }
 }
 
-constexpr int MAX_CLUSTER_PIECES = 16;
-constexpr int TABLE_SLICE = 512;       // page numbers of a CTA's piece kept in shared memory (longer pieces look them up as they go)
-template <int DV> constexpr size_t difference_smem_bytes() { return decode_smem_bytes<128, DV>() + TABLE_SLICE * sizeof(int); }
-struct DiffDecode {
-    const bf16 *q, *k_cache, *v_cache;
-    bf16* out;
-    float* partial;           // several pieces: [n_dec][nh][map][pieces][DV + 2]
-    const bf16* gate;         // logits, one a head, or null
-    long long gate_stride;
-    const int *dec_rows, *dec_seqs, *ctx_lens, *block_tables;
-    int max_blocks, nh, nkv, d, dv, page_size, window, pieces;
-    int cluster;              // 1: the pieces are a cluster and merge themselves
-    float scale, cap, lambda, out_scale, eps;
-};
-
-// log2(e) cap tanh(s scale / cap), or log2(e) s scale without a cap.
-__device__ __forceinline__ float capped_log2(float s, float scale, float cap) {
-    if (cap <= 0.f) return s * scale * LOG2E;
-    const float e = ex2(s * (2.0f * LOG2E * scale / cap)), top = cap * LOG2E;         // e^{2u}: tanh(u) = 1 - 2 / (1 + e^{2u})
-    return fmaf(-2.0f * top, __fdividef(1.0f, 1.0f + fminf(e, 1e30f)), top);
-}
-
-// One head's result from its maps' sums (unnormalised, over `n` parts of MW floats each, maximum and denominator at the end of a
-// part; part p of map m at base + (m * n + p) * part_stride): a warp a head.
-template <int NC>
-__device__ __forceinline__ void store_difference(const float* base, int n, size_t part_stride, size_t map_stride, int mcol, int dv,
-                                                 float lambda, float out_scale, float eps, const bf16* gate, bf16* out, int lane) {
-    float o[NC];
-#pragma unroll
-    for (int i = 0; i < NC; ++i) o[i] = 0.f;
-#pragma unroll
-    for (int mp = 0; mp < 2; ++mp) {
-        const float* b = base + mp * map_stride;
-        float m = -INFINITY, l = 0.f;
-        for (int p = lane; p < n; p += 32) m = fmaxf(m, b[p * part_stride + mcol]);
-        m = warp_max(m);
-        float a[NC];
-#pragma unroll
-        for (int i = 0; i < NC; ++i) a[i] = 0.f;
-#pragma unroll 4
-        for (int p = 0; p < n; ++p) {
-            const float* r = b + p * part_stride;
-            const float f = r[mcol] == -INFINITY ? 0.f : exp2f(r[mcol] - m);
-            l = fmaf(r[mcol + 1], f, l);
-#pragma unroll
-            for (int i = 0; i < NC; ++i)
-                if (lane + 32 * i < dv) a[i] = fmaf(r[lane + 32 * i], f, a[i]);
-        }
-        const float inv = (mp == 0 ? 1.0f : -lambda) / l;
-#pragma unroll
-        for (int i = 0; i < NC; ++i) o[i] = fmaf(a[i], inv, o[i]);
-    }
-    float ss = 0.f;
-#pragma unroll
-    for (int i = 0; i < NC; ++i) ss = fmaf(o[i], o[i], ss);
-    ss = warp_sum(ss);
-    float r = out_scale / sqrtf(ss / (float)dv + eps);
-    if (gate != nullptr) r /= 1.0f + expf(-__bfloat162float(*gate));
-#pragma unroll
-    for (int i = 0; i < NC; ++i)
-        if (lane + 32 * i < dv) out[lane + 32 * i] = __float2bfloat16_rn(o[i] * r);
-}
-
-template <int DV>
-__global__ __launch_bounds__(THREADS) void attn_difference_decode_kernel(const DiffDecode a) {
-    pdl_wait();
-    constexpr int D = 128, SK = D + 8, SV = DV + 8, KS = D / 16, ND = DV / 8;
-    extern __shared__ __align__(16) unsigned char smem_raw[];
-    bf16* sbase = reinterpret_cast<bf16*>(smem_raw);
-
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int g = lane >> 2, c = lane & 3;
-    const int kvh = blockIdx.x, bi = blockIdx.y, piece = blockIdx.z;
-    const int nrep = a.nh / a.nkv;
-    const int row = a.dec_rows[bi], seq = a.dec_seqs[bi];
-    const int ctx = a.ctx_lens[seq];
-    const int* table = a.block_tables + (size_t)seq * a.max_blocks;
-    const bool live = g < nrep;                            // this lane's two rows: both maps of head kvh * nrep + g
-    const int d = a.d, dv = a.dv, page_size = a.page_size;
-
-    uint32_t qa[KS][4];
-    {
-        const bf16* q0 = a.q + ((size_t)row * a.nh + kvh * nrep + (live ? g : 0)) * 2 * d;
-#pragma unroll
-        for (int ks = 0; ks < KS; ++ks) {
-            const int mp = ks / (KS / 2), col = (ks % (KS / 2)) * 16 + 2 * c;
-            const bool in0 = live && col < d, in8 = live && col + 8 < d;
-            const uint32_t x0 = in0 ? *reinterpret_cast<const uint32_t*>(q0 + mp * d + col) : 0u;
-            const uint32_t x8 = in8 ? *reinterpret_cast<const uint32_t*>(q0 + mp * d + col + 8) : 0u;
-            qa[ks][0] = mp == 0 ? x0 : 0u;
-            qa[ks][1] = mp == 0 ? 0u : x0;
-            qa[ks][2] = mp == 0 ? x8 : 0u;
-            qa[ks][3] = mp == 0 ? 0u : x8;
-        }
-    }
-    const int k_lo = a.window > 0 ? max(0, ctx - a.window) : 0;
-    const int k_hi = ctx;
-    const int t_first = k_lo / BN, t_all = (k_hi + BN - 1) / BN - t_first;
-    const int per = (t_all + a.pieces - 1) / a.pieces;
-    const int kt0 = t_first + piece * per, kt1 = min(kt0 + per, t_first + t_all);
-    const int page_shift = (page_size & (page_size - 1)) == 0 ? 31 - __clz(page_size) : -1;
-    // a look-up in global memory before every copy is most of a tile's time: the piece's page numbers come to shared memory once
-    int* pages = reinterpret_cast<int*>(sbase + (size_t)DEC_STAGES * Stage<D, DV>::ELEMS);
-    const int p_first = kt0 * BN / page_size, p_count = kt1 > kt0 ? (min(kt1 * BN, k_hi) - 1) / page_size - p_first + 1 : 0;
-    const bool sliced = p_count <= TABLE_SLICE;
-    if (sliced) {
-        for (int i = threadIdx.x; i < p_count; i += THREADS) pages[i] = table[p_first + i];
-        __syncthreads();
-    }
-
-    auto issue = [&](int kt, int stage) {
-        bf16* ks_ = sbase + (size_t)stage * Stage<D, DV>::ELEMS;
-        bf16* vs_ = ks_ + BN * SK;
-        constexpr int CK = D / 8, CV = DV / 8;
-#pragma unroll
-        for (int i = 0; i < BN * (CK + CV) / THREADS; ++i) {
-            const bool is_v = i >= BN * CK / THREADS;
-            const int idx = threadIdx.x + (is_v ? i - BN * CK / THREADS : i) * THREADS;
-            const int chunks = is_v ? CV : CK;
-            const int kin = idx / chunks, c16 = idx % chunks;
-            const int key = kt * BN + kin;
-            const int col = is_v ? c16 * 8 : (c16 % (CK / 2)) * 8;
-            const bool valid = key < k_hi && key >= k_lo && col < (is_v ? dv : d);
-            size_t off = 0;
-            if (valid) {
-                const int pi = page_shift >= 0 ? key >> page_shift : key / page_size;
-                const int page = sliced ? pages[pi - p_first] : table[pi];
-                const size_t r = ((size_t)page * a.nkv + kvh) * page_size + (key - pi * page_size);
-                off = is_v ? r * dv + col : (r * 2 + c16 / (CK / 2)) * d + col;
-            }
-            if (is_v) cp_async16(vs_ + kin * SV + c16 * 8, a.v_cache + off, valid);
-            else cp_async16(ks_ + kin * SK + c16 * 8, a.k_cache + off, valid);
-        }
-        cp_async_commit();
-    };
-
-    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
-    float oacc[ND][4];
-#pragma unroll
-    for (int nd = 0; nd < ND; ++nd)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) oacc[nd][e] = 0.f;
-#pragma unroll
-    for (int s = 0; s < DEC_STAGES - 1; ++s) {
-        if (kt0 + s < kt1) issue(kt0 + s, s);
-        else cp_async_commit();                      // an empty group keeps the count of groups in step
-    }
-    for (int kt = kt0; kt < kt1; ++kt) {
-        const int stage = (kt - kt0) % DEC_STAGES;
-        cp_async_wait<DEC_STAGES - 2>();
-        __syncthreads();                             // tile kt has landed, and everyone is done with the stage of tile kt - 1
-        if (kt + DEC_STAGES - 1 < kt1) issue(kt + DEC_STAGES - 1, (kt - kt0 + DEC_STAGES - 1) % DEC_STAGES);
-        else cp_async_commit();
-        const bf16* ks_ = sbase + (size_t)stage * Stage<D, DV>::ELEMS;
-        const bf16* vs_ = ks_ + BN * SK;
-        const int key0 = kt * BN + warp * 16;              // this warp's 16 keys of the tile
-        if (key0 < k_hi && key0 + 15 >= k_lo) {
-            float sacc[2][4];
-#pragma unroll
-            for (int nt = 0; nt < 2; ++nt) {
-#pragma unroll
-                for (int e = 0; e < 4; ++e) sacc[nt][e] = 0.f;
-#pragma unroll
-                for (int ks2 = 0; ks2 < KS / 2; ++ks2) {
-                    uint32_t kb[4];
-                    ldmatrix_x4(kb, ks_ + (warp * 16 + nt * 8 + (lane & 7)) * SK + ks2 * 32 + (lane >> 3) * 8);
-                    mma_bf16_16816(sacc[nt], qa[2 * ks2], kb[0], kb[1]);
-                    mma_bf16_16816(sacc[nt], qa[2 * ks2 + 1], kb[2], kb[3]);
-                }
-            }
-            float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-            for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    const int key = key0 + nt * 8 + 2 * c + (e & 1);
-                    const bool seen = key < k_hi && key >= k_lo;
-                    sacc[nt][e] = seen ? capped_log2(sacc[nt][e], a.scale, a.cap) : -INFINITY;
-                    mx[e >> 1] = fmaxf(mx[e >> 1], sacc[nt][e]);
-                }
-            float ms[2], corr[2], ls[2] = {0.f, 0.f};
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
-                mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
-                const float mn = fmaxf(m_run[r], mx[r]);
-                ms[r] = mn == -INFINITY ? 0.f : mn;
-                corr[r] = exp2f(m_run[r] - ms[r]);
-                m_run[r] = mn;
-            }
-#pragma unroll
-            for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    sacc[nt][e] = exp2f(sacc[nt][e] - ms[e >> 1]);
-                    ls[e >> 1] += sacc[nt][e];
-                }
-#pragma unroll
-            for (int r = 0; r < 2; ++r) {
-                ls[r] += __shfl_xor_sync(0xffffffffu, ls[r], 1);
-                ls[r] += __shfl_xor_sync(0xffffffffu, ls[r], 2);
-                l_run[r] = l_run[r] * corr[r] + ls[r];
-            }
-#pragma unroll
-            for (int nd = 0; nd < ND; ++nd)
-#pragma unroll
-                for (int e = 0; e < 4; ++e) oacc[nd][e] *= corr[e >> 1];
-            uint32_t pa[4];
-            pa[0] = pack_bf16(sacc[0][0], sacc[0][1]);
-            pa[1] = pack_bf16(sacc[0][2], sacc[0][3]);
-            pa[2] = pack_bf16(sacc[1][0], sacc[1][1]);
-            pa[3] = pack_bf16(sacc[1][2], sacc[1][3]);
-#pragma unroll
-            for (int nd2 = 0; nd2 < ND / 2; ++nd2) {
-                uint32_t vb[4];
-                const int mat = lane >> 3;
-                ldmatrix_x4_trans(vb, vs_ + (warp * 16 + (mat & 1) * 8 + (lane & 7)) * SV + (nd2 * 2 + (mat >> 1)) * 8);
-                mma_bf16_16816(oacc[2 * nd2], pa, vb[0], vb[1]);
-                mma_bf16_16816(oacc[2 * nd2 + 1], pa, vb[2], vb[3]);
-            }
-        }
-    }
-    cp_async_wait<0>();
-    __syncthreads();
-    pdl_trigger();
-    // the four warps' states meet in shared memory (the stages are free now): [warp][row][DV + 2]
-    constexpr int MW = DV + 2;
-    float* mg = reinterpret_cast<float*>(smem_raw);
-    {
-        float* a0 = mg + ((size_t)warp * 16 + g) * MW;
-        float* a1 = a0 + 8 * MW;
-#pragma unroll
-        for (int nd = 0; nd < ND; ++nd) {
-            a0[nd * 8 + 2 * c] = oacc[nd][0];
-            a0[nd * 8 + 2 * c + 1] = oacc[nd][1];
-            a1[nd * 8 + 2 * c] = oacc[nd][2];
-            a1[nd * 8 + 2 * c + 1] = oacc[nd][3];
-        }
-        if (c == 0) {
-            a0[DV] = m_run[0]; a0[DV + 1] = l_run[0];
-            a1[DV] = m_run[1]; a1[DV + 1] = l_run[1];
-        }
-    }
-    __syncthreads();
-    if (a.pieces == 1) {
-        for (int r = warp; r < nrep; r += WARPS) {
-            const int head = kvh * nrep + r;
-            store_difference<DV / 32>(mg + (size_t)r * MW, WARPS, (size_t)16 * MW, (size_t)8 * MW, DV, dv, a.lambda, a.out_scale, a.eps,
-                                      a.gate != nullptr ? a.gate + (size_t)row * a.gate_stride + head : nullptr,
-                                      a.out + ((size_t)row * a.nh + head) * dv, lane);
-        }
-        return;
-    }
-    // (in a cluster: this CTA's merged rows [head][map][MW], behind the warps' rows)
-    float* mine = mg + (size_t)WARPS * 16 * MW;
-    for (int idx = threadIdx.x; idx < 2 * nrep * DV; idx += THREADS) {
-        const int u = idx / DV, col = idx - u * DV, r = u >> 1, mp = u & 1;
-        const float* b = mg + (size_t)(mp * 8 + r) * MW;
-        float m = -INFINITY, l = 0.f, o = 0.f;
-#pragma unroll
-        for (int w = 0; w < WARPS; ++w) m = fmaxf(m, b[(size_t)w * 16 * MW + DV]);
-#pragma unroll
-        for (int w = 0; w < WARPS; ++w) {
-            const float* x = b + (size_t)w * 16 * MW;
-            const float f = x[DV] == -INFINITY ? 0.f : exp2f(x[DV] - m);
-            l = fmaf(x[DV + 1], f, l);
-            o = fmaf(x[col], f, o);
-        }
-        float* dst = a.cluster ? mine + (size_t)u * MW : a.partial + ((((size_t)bi * a.nh + kvh * nrep + r) * 2 + mp) * a.pieces + piece) * MW;
-        dst[col] = o;
-        if (col == 0) { dst[DV] = m; dst[DV + 1] = l; }
-    }
-    if (!a.cluster) return;
-    cluster_sync_all();
-    __shared__ float red[WARPS];
-    for (int r = piece; r < nrep; r += a.pieces) {         // the same for all threads of the CTA
-        // warp w takes columns w, w + 4, ... blocks of 32; every lane reads its columns from all pieces
-        constexpr int NC = DV / 32 / WARPS > 0 ? DV / 32 / WARPS : 1;
-        float o[NC];
-#pragma unroll
-        for (int i = 0; i < NC; ++i) o[i] = 0.f;
-#pragma unroll
-        for (int mp = 0; mp < 2; ++mp) {
-            const float* b = mine + (size_t)(2 * r + mp) * MW;
-            // lane p holds piece p's maximum and denominator (up to 16 pieces)
-            const float pm = lane < a.pieces ? ld_dsmem(b + DV, (uint32_t)lane) : -INFINITY;
-            const float pl = lane < a.pieces ? ld_dsmem(b + DV + 1, (uint32_t)lane) : 0.f;
-            const float m = warp_max(pm);
-            const float pf = pm == -INFINITY ? 0.f : exp2f(pm - m);
-            const float inv = (mp == 0 ? 1.0f : -a.lambda) / warp_sum(pl * pf);
-            float x[NC][16];
-#pragma unroll
-            for (int p = 0; p < 16; ++p)
-#pragma unroll
-                for (int i = 0; i < NC; ++i) {
-                    const int col = (warp + i * WARPS) * 32 + lane;
-                    x[i][p] = p < a.pieces && col < DV ? ld_dsmem(b + col, (uint32_t)p) : 0.f;
-                }
-#pragma unroll
-            for (int p = 0; p < 16; ++p) {
-                const float f = __shfl_sync(0xffffffffu, pf, p) * inv;
-#pragma unroll
-                for (int i = 0; i < NC; ++i) o[i] = fmaf(x[i][p], f, o[i]);
-            }
-        }
-        float ss = 0.f;
-#pragma unroll
-        for (int i = 0; i < NC; ++i) ss = fmaf(o[i], o[i], ss);
-        ss = warp_sum(ss);
-        if (lane == 0) red[warp] = ss;
-        __syncthreads();
-        const int head = kvh * nrep + r;
-        float f = a.out_scale / sqrtf(((red[0] + red[1]) + (red[2] + red[3])) / (float)dv + a.eps);
-        if (a.gate != nullptr) f /= 1.0f + expf(-__bfloat162float(a.gate[(size_t)row * a.gate_stride + head]));
-#pragma unroll
-        for (int i = 0; i < NC; ++i) {
-            const int col = (warp + i * WARPS) * 32 + lane;
-            if (col < dv) a.out[((size_t)row * a.nh + head) * dv + col] = __float2bfloat16_rn(o[i] * f);
-        }
-        __syncthreads();
-    }
-    cluster_sync_all();        // nobody leaves while its rows may still be read
-}
-
-// Pieces of a context into one result: one warp a (token, head), both maps.
-template <int DV>
-__global__ __launch_bounds__(128) void attn_difference_merge_kernel(const DiffDecode a, int n_units) {
-    pdl_wait_and_trigger();
-    const int unit = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (unit >= n_units) return;
-    const int bi = unit / a.nh, head = unit - bi * a.nh, row = a.dec_rows[bi];
-    constexpr int MW = DV + 2;
-    store_difference<DV / 32>(a.partial + (size_t)unit * 2 * a.pieces * MW, a.pieces, MW, (size_t)a.pieces * MW, DV, a.dv, a.lambda,
-                              a.out_scale, a.eps, a.gate != nullptr ? a.gate + (size_t)row * a.gate_stride + head : nullptr,
-                              a.out + ((size_t)row * a.nh + head) * a.dv, lane);
-}
-
 bool sizes_taken(int d, int dv) { return (d == 64 || d == 128) && (dv == 32 || dv == 64 || dv == 128); }
 
 template <int D, int DV> void raise_smem_limits() {
@@ -980,80 +636,5 @@ extern "C" int rlis_attention_bias_decode(const void* q, const void* k_cache, co
     const int units = n_dec * nh;
     rlis_launch(attn_bias_decode_merge_kernel, (units + 3) / 4, 128, 0, stream, (const float*)partial, (bf16*)out,
                 (const bf16*)gate, gate_stride, dec_rows, units, nh, dv, pieces, sinks, gate_cols);
-    return RLIS_LAUNCH_CHECK();
-}
-
-// Whether the kernel for single tokens with two maps a head takes these sizes (bfloat16).
-extern "C" int rlis_attention_difference_decode_takes(int nh, int nkv, int d, int dv) {
-    return nkv > 0 && nh % nkv == 0 && nh / nkv <= 8 && d > 0 && d <= 64 && d % 8 == 0 && dv > 0 && dv <= 128 && dv % 8 == 0;
-}
-// Width of a value row in the partial sums (values are padded to it).
-extern "C" int rlis_attention_difference_decode_width(int dv) { return dv <= 64 ? 64 : 128; }
-
-static void raise_difference_limits() {
-    static bool done = false;
-    if (done) return;
-    cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)difference_smem_bytes<64>());
-    cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)difference_smem_bytes<128>());
-    cudaFuncSetAttribute(attn_difference_decode_kernel<64>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-    cudaFuncSetAttribute(attn_difference_decode_kernel<128>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
-    done = true;
-}
-
-// How many clusters of `pieces` CTAs the device holds at a time (0: none, or the query failed).
-extern "C" int rlis_attention_difference_decode_resident(int dv, int pieces) {
-    if (pieces < 1 || pieces > MAX_CLUSTER_PIECES) return 0;
-    raise_difference_limits();
-    const bool narrow = rlis_attention_difference_decode_width(dv) == 64;
-    cudaLaunchConfig_t cfg = {};
-    cfg.gridDim = dim3(1, 1, (unsigned)pieces);
-    cfg.blockDim = THREADS;
-    cfg.dynamicSmemBytes = narrow ? difference_smem_bytes<64>() : difference_smem_bytes<128>();
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeClusterDimension;
-    attr[0].val.clusterDim.x = 1;
-    attr[0].val.clusterDim.y = 1;
-    attr[0].val.clusterDim.z = (unsigned)pieces;
-    cfg.attrs = attr;
-    cfg.numAttrs = 1;
-    int n = 0;
-    const cudaError_t e = narrow ? cudaOccupancyMaxActiveClusters(&n, attn_difference_decode_kernel<64>, &cfg)
-                                 : cudaOccupancyMaxActiveClusters(&n, attn_difference_decode_kernel<128>, &cfg);
-    if (e != cudaSuccess) {
-        cudaGetLastError();
-        return 0;
-    }
-    return n;
-}
-
-// Up to this many pieces of a context merge inside a cluster.
-extern "C" int rlis_attention_difference_decode_cluster() { return MAX_CLUSTER_PIECES; }
-
-// partial: float32, at least n_dec * nh * 2 * pieces * (width(dv) + 2) elements when the pieces do not merge in a cluster; the rest as
-// rlis_attention_difference.
-extern "C" int rlis_attention_difference_decode(const void* q, const void* k_cache, const void* v_cache, void* out, float* partial,
-                                                const void* gate, long long gate_stride, const int* dec_rows, const int* dec_seqs,
-                                                const int* ctx_lens, const int* block_tables, int max_blocks, int n_dec, int nh,
-                                                int nkv, int d, int dv, int page_size, float scale, float cap, int window, int pieces,
-                                                float lambda, float out_scale, float eps, cudaStream_t stream) {
-    if (n_dec <= 0) return 0;
-    if (!rlis_attention_difference_decode_takes(nh, nkv, d, dv) || pieces < 1 || pieces > 65535 || n_dec > 65535 || cap < 0.f ||
-        (pieces > MAX_CLUSTER_PIECES && partial == nullptr) ||
-        ((reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k_cache) | reinterpret_cast<uintptr_t>(v_cache)) & 15) != 0)
-        return RLIS_ERR_UNSUPPORTED;
-    raise_difference_limits();
-    const DiffDecode a{(const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, partial, (const bf16*)gate, gate_stride,
-                       dec_rows, dec_seqs, ctx_lens, block_tables, max_blocks, nh, nkv, d, dv, page_size, window, pieces,
-                       pieces > 1 && pieces <= MAX_CLUSTER_PIECES ? 1 : 0, scale, cap, lambda, out_scale, eps};
-    const dim3 grid(nkv, n_dec, pieces);
-    const bool narrow = rlis_attention_difference_decode_width(dv) == 64;
-    const dim3 cluster(1, 1, a.cluster ? (unsigned)pieces : 1u);
-    if (narrow) rlis_launch_cluster(attn_difference_decode_kernel<64>, grid, THREADS, difference_smem_bytes<64>(), stream, cluster, a);
-    else rlis_launch_cluster(attn_difference_decode_kernel<128>, grid, THREADS, difference_smem_bytes<128>(), stream, cluster, a);
-    const int err = RLIS_LAUNCH_CHECK();
-    if (err != 0 || pieces == 1 || a.cluster) return err;
-    const int units = n_dec * nh;
-    if (narrow) rlis_launch(attn_difference_merge_kernel<64>, (units + 3) / 4, 128, 0, stream, a, units);
-    else rlis_launch(attn_difference_merge_kernel<128>, (units + 3) / 4, 128, 0, stream, a, units);
     return RLIS_LAUNCH_CHECK();
 }

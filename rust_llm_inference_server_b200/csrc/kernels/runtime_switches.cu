@@ -56,15 +56,17 @@ extern "C" int* rlis_gemm_tcgen05_error_addr(void);
 extern "C" int* rlis_stream_gemm_error_addr(void);
 extern "C" int* rlis_attention_prefill_tc_error_addr(void);
 extern "C" int* rlis_attention_decode_error_addr(void);
+extern "C" int* rlis_attention_difference_decode_error_addr(void);
 
 namespace {
-struct ErrorWords { int* w[4]; };
+constexpr int kWords = 5;
+struct ErrorWords { int* w[kWords]; };
 
 __global__ void take_errors_kernel(ErrorWords words, int* __restrict__ out) {
     pdl_wait_and_trigger();
     int v = 0;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) v |= atomicExch(words.w[i], 0);
+    for (int i = 0; i < kWords; ++i) v |= atomicExch(words.w[i], 0);
     *out = v;
 }
 
@@ -79,8 +81,9 @@ extern "C" int rlis_take_errors(int* out, cudaStream_t stream) {
     if (cudaGetDevice(&dev) != cudaSuccess || dev < 0 || dev >= kMaxDevices) return RLIS_ERR_UNSUPPORTED;
     if (!g_words_known[dev]) {
         ErrorWords w = {{rlis_gemm_tcgen05_error_addr(), rlis_stream_gemm_error_addr(),
-                         rlis_attention_prefill_tc_error_addr(), rlis_attention_decode_error_addr()}};
-        for (int i = 0; i < 4; ++i)
+                         rlis_attention_prefill_tc_error_addr(), rlis_attention_decode_error_addr(),
+                         rlis_attention_difference_decode_error_addr()}};
+        for (int i = 0; i < kWords; ++i)
             if (w.w[i] == nullptr) return RLIS_ERR_UNSUPPORTED;
         g_words[dev] = w;
         g_words_known[dev] = true;

@@ -1169,7 +1169,7 @@ def check_device_errors() -> None:
     """Raises if a bounded wait inside a kernel ever ran out on this device (the kernel then
     finished without its data; results since are not to be trusted).  Synchronises the device."""
     code = (lib().rlis_gemm_tcgen05_error() or lib().rlis_stream_gemm_error() or lib().rlis_attention_prefill_tc_error()
-            or lib().rlis_attention_decode_error())
+            or lib().rlis_attention_decode_error() or lib().rlis_attention_difference_decode_error())
     if code != 0:
         raise KernelError(f"a bounded mbarrier wait of a tcgen05 kernel ran out on the device (code {code})")
 
@@ -1731,8 +1731,8 @@ def _difference_prefill_sizes(dim: int, v_dim: int, page_size: int) -> bool:
 
 
 @functools.lru_cache(maxsize=None)
-def _difference_decode_sizes(n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
-    return bool(lib().rlis_attention_difference_decode_takes(n_heads, n_kv_heads, dim, v_dim))
+def _difference_decode_sizes(n_heads: int, n_kv_heads: int, dim: int, v_dim: int, page_size: int) -> bool:
+    return bool(lib().rlis_attention_difference_decode_takes(n_heads, n_kv_heads, dim, v_dim, page_size))
 
 
 def difference_prefill_takes_mma(dtype, dim: int, v_dim: int, page_size: int = 16) -> bool:
@@ -1740,10 +1740,10 @@ def difference_prefill_takes_mma(dtype, dim: int, v_dim: int, page_size: int = 1
     return bool(DIFFERENCE_MMA and dtype == torch.bfloat16 and _difference_prefill_sizes(int(dim), int(v_dim), int(page_size)))
 
 
-def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, v_dim: int) -> bool:
+def difference_decode_takes_mma(dtype, n_heads: int, n_kv_heads: int, dim: int, v_dim: int, page_size: int = 16) -> bool:
     """The same for single tokens."""
     return bool(DIFFERENCE_MMA and dtype == torch.bfloat16
-                and _difference_decode_sizes(int(n_heads), int(n_kv_heads), int(dim), int(v_dim)))
+                and _difference_decode_sizes(int(n_heads), int(n_kv_heads), int(dim), int(v_dim), int(page_size)))
 
 
 @functools.lru_cache(maxsize=None)
@@ -1796,7 +1796,7 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
             raise KernelError("attention_difference: the gate must be [T, nh] rows with unit stride in q's type")
         gp, gs = gate.data_ptr(), gate.stride(0)
     tables = step.block_tables[group]
-    n_dec = step.n_decode if difference_decode_takes_mma(q.dtype, n_heads, n_kv_heads, dim, v_dim) else 0
+    n_dec = step.n_decode if difference_decode_takes_mma(q.dtype, n_heads, n_kv_heads, dim, v_dim, page_size) else 0
     n_tiles = step.n_prefill_tiles if difference_prefill_takes_mma(q.dtype, dim, v_dim, page_size) else 0
     if n_dec:
         pieces = difference_decode_pieces(n_dec, n_kv_heads, v_dim, step.max_decode_ctx, window)
@@ -1805,7 +1805,7 @@ def attention_difference(q, k_cache, v_cache, out, gate, step, group: int, n_hea
         check(lib().rlis_attention_difference_decode(
             q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), scratch.data_ptr() if scratch is not None else None,
             gp, gs, step.dec_rows.data_ptr(), step.dec_seqs.data_ptr(), step.ctx_lens.data_ptr(), tables.data_ptr(), tables.shape[1],
-            n_dec, n_heads, n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), pieces, float(lam),
+            n_dec, k_cache.shape[0], n_heads, n_kv_heads, dim, v_dim, page_size, float(scale), float(cap), int(window), pieces, float(lam),
             float(out_scale), float(eps), _stream()), "attention_difference_decode")
         _count("attention_difference.decode.mma" + (".split" if scratch is not None else ".cluster" if pieces > 1 else ""))
     if n_tiles:

@@ -63,8 +63,8 @@ SIGNATURES = {
     "rlis_attention_difference": [P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, F, F, F, I, P],
     "rlis_attention_difference_prefill": [P, P, P, P, P, LL, P, I, P, P, P, I, I, I, I, I, I, I, I, F, F, I, F, F, F, P],
     "rlis_attention_difference_prefill_takes": [I, I, I],
-    "rlis_attention_difference_decode": [P, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, F, F, I, I, F, F, F, P],
-    "rlis_attention_difference_decode_takes": [I, I, I, I],
+    "rlis_attention_difference_decode": [P, P, P, P, P, P, LL, P, P, P, P, I, I, I, I, I, I, I, I, F, F, I, I, F, F, F, P],
+    "rlis_attention_difference_decode_takes": [I, I, I, I, I],
     "rlis_attention_difference_decode_width": [I],
     "rlis_attention_difference_decode_cluster": [],
     "rlis_attention_difference_decode_resident": [I, I],
@@ -138,7 +138,7 @@ def lib():
             fn.argtypes = args
             fn.restype = c_int
         for name in ("rlis_gemm_tcgen05_error", "rlis_stream_gemm_error", "rlis_attention_prefill_tc_error",
-                     "rlis_attention_decode_error"):
+                     "rlis_attention_decode_error", "rlis_attention_difference_decode_error"):
             fn = getattr(handle, name)
             fn.argtypes = []
             fn.restype = c_int
