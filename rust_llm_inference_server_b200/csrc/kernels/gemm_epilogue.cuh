@@ -2,6 +2,7 @@
 #pragma once
 #include "common.cuh"
 #include "mma_utils.cuh"
+#include <math.h>
 
 namespace tc {
 
@@ -46,6 +47,16 @@ __device__ __forceinline__ void store_sums32(const uint32_t (&r)[32], void* __re
     } else if (EPI == 1 || EPI == 3) {
         bf16* o = reinterpret_cast<bf16*>(y) + (size_t)row * (N >> 1) + (col >> 1);
         float res[16];
+        if (EPI == 3 && gp.cubic != 0.f && gp.limit == INFINITY && gp.shift == 0.f) {
+            // a gate of the gelu kind, without the branches of the general one: its result is rounded to bfloat16, so the
+            // fast exponential and division serve
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+                const float g = __uint_as_float(r[(i >> 2) * 8 + (i & 3)]), u = __uint_as_float(r[(i >> 2) * 8 + 4 + (i & 3)]);
+                const float z = fmaf(gp.cubic * g * g, g, g);
+                res[i] = __fdividef(g, 1.0f + __expf(-gp.slope * z)) * u;
+            }
+        } else
 #pragma unroll
         for (int tt = 0; tt < 4; ++tt)
 #pragma unroll
