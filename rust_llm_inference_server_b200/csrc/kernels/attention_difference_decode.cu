@@ -1,4 +1,4 @@
-// Single decoded tokens of attention with two maps a head (attention_difference.cu has the contract), on mma.sync m16n8k16 with
+// Single decoded tokens of attention with two maps a head (attention_difference.cu has the formulas), on mma.sync m16n8k16 with
 // float32 sums.  One CTA of four warps = one key/value head x one request x one piece of its context.  Rows 0..7 of the products
 // are the group's query heads' first maps, rows 8..15 their second ones; a cached key row is [map 1 | map 2], each padded to 64
 // entries, and a query row is its map's vector with zeros over the other's entries, so one set of products gives both maps'

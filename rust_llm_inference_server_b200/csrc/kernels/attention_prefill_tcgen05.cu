@@ -87,7 +87,7 @@
 // badly), and as two ordinary CTAs that leave their rows in a scratch buffer for the one that takes
 // the tile's last ticket, 57 -> 78 us; at 4096 tokens and more nothing is shared and nothing changes.)
 //
-// Two maps a head (DIFF; the contract of attention_difference.cu): the same kernel at its head size of 128, with one query
+// Two maps a head (DIFF; the formulas are in attention_difference.cu): the same kernel at its head size of 128, with one query
 // head a CTA.  A cached key row is [map 1 | map 2], up to 64 entries each, in the two sub-tiles of a row of K; the 128 rows of
 // the instruction are (map 1, tokens 0..63) and (map 2, tokens 0..63), and a row of Q is its map's vector in that map's
 // sub-tile and zeros in the other, so one product over both sub-tiles gives both maps' scores (the zeros double the score

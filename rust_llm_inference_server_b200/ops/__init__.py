@@ -1755,7 +1755,7 @@ def _difference_clusters(v_dim: int, pieces: int) -> int:
 def _difference_decode_pieces(n_decode: int, n_kv_heads: int, v_dim: int, seen: int, sms: int) -> int:
     """Pieces a context is cut into, at least two tiles of 64 keys each: a CTA takes one key/value head of one request and the
     pieces of up to 16 merge in a cluster, so the context is cut as finely as clusters of that size are all resident at once
-    (one that does not fit waits for a whole round: 8 requests with four heads, 35 us in clusters of 8 and 60 us in clusters of
+    (one that does not fit waits for a whole wave: 8 requests with four heads, 35 us in clusters of 8 and 60 us in clusters of
     9).  More pieces and a second kernel only where 16 would leave every CTA a long way to go."""
     tiles, ctas = -(-seen // 64), max(1, n_decode * n_kv_heads)
     most = max(1, min(2 * sms // ctas, tiles // 2))
